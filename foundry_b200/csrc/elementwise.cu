@@ -2,7 +2,7 @@
 // residual add fused with RMS normalisation, SiLU(gate) * up, row gather.
 //
 // Formulas (reference file:line, by its path in stratorys/foundry):
-//   embedding  x[t,:] = E[ids[t],:]; an id outside the table gives a zero row
+//   embedding  x[t,:] = E[ids[t],:] (times a constant); an id outside the table gives a zero row
 //              (src/nn/linear.rs:54-69, src/metal/kernels/index_select.metal:23-26)
 //   RMS norm   r = 1/sqrt(sum(x^2) * (1/H) + eps); y = x * r * w, in 32-bit
 //              (src/nn/norm.rs:31-51)
@@ -30,7 +30,7 @@ __device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
 // ------------------------------------------------------------------ embedding
 template <typename T>
 __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                    float* __restrict__ out, int H, int V) {
+                                    float* __restrict__ out, int H, int V, float scale) {
   fb_pdl_launch();  // a few small blocks: the norm behind them may be placed at once
   fb_pdl_wait();
   const int t = blockIdx.x;
@@ -54,21 +54,23 @@ __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __re
 #pragma unroll
       for (int a = 0; a < AHEAD; ++a) {
         const int i = i0 + a * blockDim.x * 4;
-        if (i < H) *reinterpret_cast<float4*>(dst + i) = v[a];
+        if (i < H)
+          *reinterpret_cast<float4*>(dst + i) =
+              make_float4(v[a].x * scale, v[a].y * scale, v[a].z * scale, v[a].w * scale);
       }
     }
     return;
   }
-  for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = fb_to_float<T>(src[i]);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = fb_to_float<T>(src[i]) * scale;
 }
 
 FB_API int fb_embed_gather(const void* table, int table_dtype, const int* ids, float* out, int T,
-                           int H, int V, cudaStream_t stream) {
+                           int H, int V, float scale, cudaStream_t stream) {
   FB_REQUIRE(T >= 0 && H > 0 && V > 0, "embed_gather: bad sizes T=%d H=%d V=%d", T, H, V);
   if (T == 0) return 0;
   const int threads = H >= 1024 ? 256 : 128;
   FB_DISPATCH_DTYPE(table_dtype, E, (fb_launch(embed_gather_kernel<E>, dim3(T), dim3(threads), 0, stream, 
-                                        (const E*)table, ids, out, H, V)));
+                                        (const E*)table, ids, out, H, V, scale)));
   return fb_check_launch("embed_gather");
 }
 

@@ -5,8 +5,10 @@
 //   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // RWKV-style time mixing with a bonus for the current token (per head):
 //   o = (S + diag(b) k v^T)^T r;  S <- diag(w) S + k v^T
-// State-space duality (Mamba-2) with one decay a head, a step size and a skip (per head):
-//   S <- g S + k (step v)^T;  o = S^T q + skip v
+// Linear recurrence with a decay a head or a key channel, optionally a step size and a skip
+// (per head); with one decay a head, step size and skip it is state-space duality (Mamba-2),
+// with a decay a channel and neither it is gated linear attention:
+//   S <- diag(g) S + k (step v)^T;  o = scale S^T q + skip v
 //
 // Both recurrences act on the columns of S independently, so a thread owns a
 // slice of one column in registers (16 consecutive key rows at most, a column
@@ -15,6 +17,12 @@
 // lanes of a column. The state is 32-bit and lives in the sequence's state row
 // between steps; every sequence of the step is walked by its own blocks from
 // `cu_tokens`, so a step may bring any number of tokens per sequence.
+//
+// The linear recurrences (the last two) may also run a prompt's chunks of tokens side by
+// side, in three launches: every chunk's own contribution to the state, from a zero state,
+// with the product of its decays; one pass over the chunks that turns these into each
+// chunk's starting state, S_(c+1) = diag(G_c) S_c + dS_c; and every chunk's outputs from
+// its starting state. All of it is the same 32-bit arithmetic, reordered at chunk ends.
 //
 // Around them, per token: the mix with the previous token's input (token
 // shift), a short causal convolution with SiLU and unit-length heads, the
@@ -205,13 +213,19 @@ struct ScanArgs {
   const float* v; long long v_ld;   // values: head h at h * vdim
   const float* g; long long g_ld;   // decays: head h at h * dim, or one per head at h (g_scalar)
   const float* beta; long long beta_ld;  // delta: raw step size per head (sigmoid applied here);
-                                    // ssd: the step size per head as it is
-  const float* bonus;               // wkv: [H, dim]; ssd: the skip, [H]
+                                    // linear: the step size per head as it is, or null (1)
+  const float* bonus;               // wkv: [H, dim]; linear: the skip, [H], or null
   float* state; long long state_stride; long long s_offset;
   float* out;                       // [T, H * vdim]
   const int* cu_tokens; const int* slots;
   int H, rep, dim, vdim;
   int g_scalar;                     // one decay a head instead of one a key channel
+  float out_scale;                  // linear: o = out_scale * S^T q + skip v
+  // chunks side by side: blockIdx.x = seq * n_chunks + chunk, chunks of `chunk` tokens.
+  // ws [n_seqs, n_chunks, H, dim, vdim]: a chunk's contribution, then its starting state;
+  // wg [n_seqs, n_chunks, H, dim]: the product of a chunk's decays. n_chunks 1: off.
+  int n_chunks, chunk;
+  float* ws; float* wg;
 };
 
 __device__ __forceinline__ void cp_async4(float* dst, const float* src) {
@@ -231,15 +245,23 @@ __device__ __forceinline__ void cp_async_wait_but_one() {
 // consecutive rows part * rp .. (a multiple of 4: they are read as float4).
 // RP: key rows a lane holds (4 or 8, or 16 for heads of more than 256 key channels);
 // MINE: elements of a token's record a thread copies at most.
+// MODE 0: delta rule; 1: wkv; 2: linear; 3: a chunk's contribution to the state of 1 or 2.
 template <int MODE, int KP, int RP, int MINE>
 __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
   constexpr int rp = RP;
   fb_pdl_wait();
   constexpr int COLS_W = 32 / KP;  // columns a warp holds
   extern __shared__ __align__(16) float sbuf[];
-  const int seq = blockIdx.x, h = blockIdx.y;
-  const int start = a.cu_tokens[seq], n = a.cu_tokens[seq + 1] - start;
-  if (n <= 0) return;
+  const int seq = blockIdx.x / a.n_chunks, h = blockIdx.y;
+  const int chunk = blockIdx.x - seq * a.n_chunks;
+  int start = a.cu_tokens[seq], n = a.cu_tokens[seq + 1] - start;
+  const bool last_chunk = a.n_chunks == 1 || (chunk + 1) * a.chunk >= n;
+  if (a.n_chunks > 1) {
+    start += chunk * a.chunk;
+    n = min(n - chunk * a.chunk, a.chunk);
+  }
+  // (nothing starts from the last chunk's contribution: it is not worked out)
+  if (n <= 0 || (MODE == 3 && last_chunk)) return;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   const int part = lane / COLS_W;
   const int cols_blk = nwarps * COLS_W;
@@ -251,6 +273,8 @@ __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
   const int dimp = KP * rp;
   float* S = a.state + (long long)a.slots[seq] * a.state_stride + a.s_offset +
              (long long)h * dim * vdim;
+  const long long unit = ((long long)blockIdx.x * a.H + h) * dim;  // this chunk's place in wg, ws
+  float* S_chunk = a.n_chunks > 1 ? a.ws + unit * vdim : nullptr;
   const long long qoff = (long long)(h / a.rep) * dim, goff = (long long)h * dim;
   const int per_tok = (3 * dimp + cols_blk + 1 + 3) / 4 * 4;
   const int row0 = part * rp;  // this thread's first key row
@@ -272,7 +296,7 @@ __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
     long long step = 0;
     if (c < 3 * dimp) {
       const int which = c / dimp, row = c - which * dimp;
-      if (row < dim) {
+      if (row < dim && !(MODE == 3 && which == 0)) {
         src = which == 0 ? a.q + qoff + row : which == 1 ? a.k + qoff + row
                          : a.g_scalar ? a.g + h : a.g + goff + row;
         step = which == 0 ? a.q_ld : which == 1 ? a.k_ld : a.g_ld;
@@ -282,7 +306,7 @@ __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
         src = a.v + (size_t)h * vdim + col0 + (c - 3 * dimp);
         step = a.v_ld;
       }
-    } else if (MODE != 1 && c == 3 * dimp + cols_blk) {
+    } else if (MODE != 1 && a.beta != nullptr && c == 3 * dimp + cols_blk) {
       src = a.beta + h;
       step = a.beta_ld;
     }
@@ -307,14 +331,17 @@ __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
     }
   };
 
-  const float skip = MODE == 2 ? a.bonus[h] : 0.f;
+  const float skip = (MODE == 2 && a.bonus != nullptr) ? a.bonus[h] : 0.f;
+  const bool stepped = MODE >= 2 && a.beta != nullptr;
+  const float* S0 = (MODE != 3 && a.n_chunks > 1) ? S_chunk : S;  // where the state starts
   float s[RP], bonus[RP];
 #pragma unroll
   for (int i = 0; i < RP; ++i) {
     const int row = row0 + i;
     const bool ok = row < dim;
-    s[i] = (col && ok) ? S[(size_t)row * vdim + j] : 0.f;
-    bonus[i] = (MODE == 1 && ok) ? a.bonus[goff + row] : 0.f;
+    s[i] = (MODE != 3 && col && ok) ? __ldcg(S0 + (size_t)row * vdim + j) : 0.f;
+    // (mode 3: the running product of the row's decays)
+    bonus[i] = MODE == 3 ? 1.f : (MODE == 1 && ok) ? a.bonus[goff + row] : 0.f;
   }
   stage(0, min(tc, n));
   cp_async_commit();
@@ -356,8 +383,17 @@ __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
             o4[2] = fmaf(s[i + 2], q.z, o4[2]); o4[3] = fmaf(s[i + 3], q.w, o4[3]);
           }
         }
+      } else if (MODE == 3) {
+        const float u = stepped ? tok[3 * dimp + cols_blk] * v : v;
+#pragma unroll
+        for (int i = 0; i < RP; i += 4) {
+          const float4 g = g4[i / 4], k = k4[i / 4];
+          s[i] = fmaf(k.x, u, g.x * s[i]); s[i + 1] = fmaf(k.y, u, g.y * s[i + 1]);
+          s[i + 2] = fmaf(k.z, u, g.z * s[i + 2]); s[i + 3] = fmaf(k.w, u, g.w * s[i + 3]);
+          bonus[i] *= g.x; bonus[i + 1] *= g.y; bonus[i + 2] *= g.z; bonus[i + 3] *= g.w;
+        }
       } else if (MODE == 2) {
-        const float u = tok[3 * dimp + cols_blk] * v;  // step size times the value
+        const float u = stepped ? tok[3 * dimp + cols_blk] * v : v;  // step size times the value
 #pragma unroll
         for (int i = 0; i < RP; i += 4) {
           {
@@ -383,23 +419,70 @@ __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
           }
         }
       }
-      opart[r * 32 + lane] = (o4[0] + o4[1]) + (o4[2] + o4[3]);
+      if (MODE != 3) opart[r * 32 + lane] = (o4[0] + o4[1]) + (o4[2] + o4[3]);
     }
     __syncwarp();
-    for (int r = part; r < nt; r += KP) {
+    for (int r = part; MODE != 3 && r < nt; r += KP) {
       float o = 0.f;
 #pragma unroll
       for (int p = 0; p < KP; ++p) o += opart[r * 32 + p * COLS_W + (lane % COLS_W)];
       if (MODE == 2)  // the skip: the token's own value straight to its output
-        o = fmaf(skip, sbuf[(size_t)buf * tc * per_tok + (size_t)r * per_tok + 3 * dimp + jl], o);
+        o = fmaf(skip, sbuf[(size_t)buf * tc * per_tok + (size_t)r * per_tok + 3 * dimp + jl],
+                 a.out_scale * o);
       if (col) a.out[(size_t)(start + c0 + r) * a.H * vdim + (size_t)h * vdim + j] = o;
     }
     __syncthreads();  // the buffers are refilled by the next iteration
   }
+  if (MODE == 3) {
+#pragma unroll
+    for (int i = 0; i < RP; ++i) {
+      const int row = row0 + i;
+      if (col && row < dim) {
+        S_chunk[(size_t)row * vdim + j] = s[i];
+        if (j == 0) a.wg[unit + row] = bonus[i];
+      }
+    }
+    return;
+  }
+  if (!last_chunk) return;  // the next chunk's starting state is known already
 #pragma unroll
   for (int i = 0; i < RP; ++i) {
     const int row = row0 + i;
     if (col && row < dim) S[(size_t)row * vdim + j] = s[i];
+  }
+}
+
+// From the chunks' contributions to their starting states, in place: one thread an element
+// of a head's state, walking the sequence's chunks; a few chunks' loads are in flight at once.
+__global__ void scan_chunk_starts_kernel(ScanArgs a) {
+  fb_pdl_wait();
+  const int seq = blockIdx.x, h = blockIdx.y;
+  const int n = a.cu_tokens[seq + 1] - a.cu_tokens[seq];
+  const int elements = a.dim * a.vdim;
+  const int i = blockIdx.z * blockDim.x + threadIdx.x;
+  if (n <= 0 || i >= elements) return;
+  const int chunks = (n + a.chunk - 1) / a.chunk;
+  float s = __ldcg(a.state + (long long)a.slots[seq] * a.state_stride + a.s_offset +
+                   (long long)h * elements + i);
+  const long long first = ((long long)seq * a.n_chunks * a.H + h) * a.dim;
+  const long long step = (long long)a.H * a.dim;
+  float* ws = a.ws + first * a.vdim + i;
+  const float* wg = a.wg + first + i / a.vdim;
+  constexpr int AHEAD = 8;
+  for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+    float d[AHEAD], g[AHEAD];
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      const bool there = c0 + u + 1 < chunks;  // (the last chunk has no contribution)
+      d[u] = there ? __ldcg(ws + (c0 + u) * step * a.vdim) : 0.f;
+      g[u] = there ? __ldcg(wg + (c0 + u) * step) : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      if (c0 + u >= chunks) break;
+      ws[(c0 + u) * step * a.vdim] = s;
+      s = fmaf(g[u], s, d[u]);
+    }
   }
 }
 
@@ -472,6 +555,46 @@ __global__ void head_norm_gate_kernel(const float* o, const float* __restrict__ 
   }
 }
 
+// ------------------------------------- decays from a low-rank projection, per key channel
+// out[t, c] = sigmoid(z)^(1 / tau),  z = sum_r low[t, r] w[c, r] + bias[c]
+// as exp(-softplus(-z) / tau). A block takes `tokens` token rows, a thread a channel: its
+// weight row is read once for all of them. low: float32 rows of stride ld, staged in
+// shared memory; w in the stored type; bias float32.
+constexpr int LR_TOKENS = 8;
+template <typename T>
+__global__ void low_rank_decay_kernel(const float* low, long long ld, const T* __restrict__ w,
+                                      const float* __restrict__ bias, float inv_tau,
+                                      float* __restrict__ out, int T_, int rank, int n) {
+  fb_pdl_launch();
+  fb_pdl_wait();
+  extern __shared__ float rows[];  // [rank][LR_TOKENS]
+  const int t0 = blockIdx.x * LR_TOKENS;
+  for (int i = threadIdx.x; i < rank * LR_TOKENS; i += blockDim.x) {
+    const int t = i / rank, r = i - t * rank;
+    rows[r * LR_TOKENS + t] = t0 + t < T_ ? __ldcg(low + (size_t)(t0 + t) * ld + r) : 0.f;
+  }
+  __syncthreads();
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= n) return;
+  float z[LR_TOKENS];
+#pragma unroll
+  for (int t = 0; t < LR_TOKENS; ++t) z[t] = bias[c];
+  const T* wr = w + (size_t)c * rank;
+  for (int r = 0; r < rank; ++r) {
+    const float v = fb_to_float<T>(wr[r]);
+    const float4* x = reinterpret_cast<const float4*>(rows + r * LR_TOKENS);
+    const float4 lo = x[0], hi = x[1];
+    z[0] = fmaf(lo.x, v, z[0]); z[1] = fmaf(lo.y, v, z[1]);
+    z[2] = fmaf(lo.z, v, z[2]); z[3] = fmaf(lo.w, v, z[3]);
+    z[4] = fmaf(hi.x, v, z[4]); z[5] = fmaf(hi.y, v, z[5]);
+    z[6] = fmaf(hi.z, v, z[6]); z[7] = fmaf(hi.w, v, z[7]);
+  }
+#pragma unroll
+  for (int t = 0; t < LR_TOKENS; ++t)
+    if (t0 + t < T_)
+      out[(size_t)(t0 + t) * n + c] = expf((fminf(z[t], 0.f) - log1pf(expf(-fabsf(z[t])))) * inv_tau);
+}
+
 // out = act(in) rounded to the activation type; act: 0 identity, 1 tanh, 2 the square of relu
 template <typename T>
 __global__ void unary_cast_kernel(const float* in, long long ld, T* __restrict__ out, int n,
@@ -510,6 +633,19 @@ FB_API int fb_sigmoid_gate(void* x, int dtype, long long ldx, const float* gate,
   FB_DISPATCH_DTYPE(dtype, E, (fb_launch(sigmoid_gate_kernel<E>, dim3(T, parts), dim3(256), 0, stream,
       (E*)x, ldx, gate, ldg, n)));
   return fb_check_launch("sigmoid_gate");
+}
+
+FB_API int fb_low_rank_decay(const float* low, long long ld, const void* w, int w_dtype,
+                             const float* bias, float tau, float* out, int T, int rank, int n,
+                             cudaStream_t stream) {
+  FB_REQUIRE(T >= 0 && rank > 0 && n > 0 && ld >= rank && tau > 0.f, "low_rank_decay: bad arguments");
+  const size_t smem = (size_t)rank * LR_TOKENS * 4;
+  FB_REQUIRE(smem <= 48 * 1024, "low_rank_decay: rank %d exceeds %d", rank, 48 * 1024 / (LR_TOKENS * 4));
+  if (T == 0) return 0;
+  const dim3 grid((T + LR_TOKENS - 1) / LR_TOKENS, (n + 127) / 128);
+  FB_DISPATCH_DTYPE(w_dtype, E, (fb_launch(low_rank_decay_kernel<E>, grid, dim3(128), smem, stream,
+      low, ld, (const E*)w, bias, 1.0f / tau, out, T, rank, n)));
+  return fb_check_launch("low_rank_decay");
 }
 
 FB_API int fb_token_shift_mix(const void* h, int dtype, float* state, long long state_stride,
@@ -596,18 +732,22 @@ FB_API int fb_state_scan(int mode, const float* q, long long q_ld, const float* 
                          const float* beta, long long beta_ld, const float* bonus, float* state,
                          long long state_stride, long long s_offset, float* out,
                          const int* cu_tokens, const int* slots, int n_seqs, int H, int rep,
-                         int dim, int vdim, int g_scalar, int serial_launch, cudaStream_t stream) {
+                         int dim, int vdim, int g_scalar, float out_scale, int n_chunks, int chunk,
+                         float* ws, float* wg, int serial_launch, cudaStream_t stream) {
   const bool serial = serial_launch != 0;
   FB_REQUIRE(mode >= 0 && mode <= 2, "state_scan: unknown recurrence %d", mode);
-  FB_REQUIRE(mode != 2 || g_scalar, "state_scan: the state-space recurrence takes one decay a head");
+  FB_REQUIRE(mode == 2 || out_scale == 1.0f, "state_scan: a constant on the outputs goes with mode 2");
+  FB_REQUIRE(n_chunks >= 1 && (n_chunks == 1 || (mode != 0 && chunk > 0 && ws && wg)),
+             "state_scan: %d chunks side by side of %d tokens in mode %d", n_chunks, chunk, mode);
   FB_REQUIRE(n_seqs >= 0 && H > 0 && rep > 0 && H % rep == 0 && dim > 0 && vdim > 0,
              "state_scan: bad sizes");
   FB_REQUIRE(dim <= R * 32, "state_scan: %d key channels exceed %d", dim, R * 32);
-  FB_REQUIRE((mode == 1 || beta != nullptr) && (mode == 0 || bonus != nullptr),
+  FB_REQUIRE((mode != 0 || beta != nullptr) && (mode != 1 || bonus != nullptr),
              "state_scan: a missing input");
   if (n_seqs == 0) return 0;
   ScanArgs a{q, q_ld, k, k_ld, v, v_ld, g, g_ld, beta, beta_ld, bonus, state, state_stride,
-             s_offset, out, cu_tokens, slots, H, rep, dim, vdim, g_scalar ? 1 : 0};
+             s_offset, out, cu_tokens, slots, H, rep, dim, vdim, g_scalar ? 1 : 0, out_scale,
+             n_chunks, chunk, ws, wg};
   // a column is shared by kp lanes: eight key rows a lane where the head allows it
   // (a token's step is a chain of dependent instructions; fewer rows a lane shorten it)
   int kp = 1;
@@ -619,14 +759,14 @@ FB_API int fb_state_scan(int mode, const float* q, long long q_ld, const float* 
     if (cudaGetDevice(&device) == cudaSuccess)
       cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
     const int cols_blk8 = 4 * (32 / kp);
-    const long long blocks = (long long)n_seqs * H * ((vdim + cols_blk8 - 1) / cols_blk8);
+    const long long blocks = (long long)n_seqs * n_chunks * H * ((vdim + cols_blk8 - 1) / cols_blk8);
     if (blocks < 2LL * sms && kp < 32 && (dim + 2 * kp - 1) / (2 * kp) <= 4) kp *= 2;
   }
   const int cols_w = 32 / kp;
   const int warps_needed = (vdim + cols_w - 1) / cols_w;
   const int most = kp >= 16 ? 8 : 4;  // (a wide head's record takes more threads to copy)
   const int warps = warps_needed < most ? warps_needed : most;
-  dim3 grid(n_seqs, H, (warps_needed + warps - 1) / warps);
+  dim3 grid(n_seqs * n_chunks, H, (warps_needed + warps - 1) / warps);
   // key rows a lane holds: 4 or 8, or 16 for heads of more than 256 key channels
   const int rows = (dim + kp - 1) / kp;
   const int rp = rows <= 4 ? 4 : rows <= 8 ? 8 : 16;
@@ -647,20 +787,34 @@ FB_API int fb_state_scan(int mode, const float* q, long long q_ld, const float* 
     if (mine <= 2) FB_SCAN_LAUNCH(M_, KP_, RP_, 2);      \
     else FB_SCAN_LAUNCH(M_, KP_, RP_, 8);                \
   } while (0)
+#define FB_SCAN_MODE(KP_, RP_)                             \
+  do {                                                     \
+    if (as_mode == 0) FB_SCAN_MINE(0, KP_, RP_);           \
+    else if (as_mode == 1) FB_SCAN_MINE(1, KP_, RP_);      \
+    else if (as_mode == 2) FB_SCAN_MINE(2, KP_, RP_);      \
+    else FB_SCAN_MINE(3, KP_, RP_);                        \
+  } while (0)
 #define FB_SCAN(KP_)                                                \
   case KP_:                                                         \
-    if (rp == 4) { if (mode == 0) FB_SCAN_MINE(0, KP_, 4); else if (mode == 1) FB_SCAN_MINE(1, KP_, 4); else FB_SCAN_MINE(2, KP_, 4); } \
-    else { if (mode == 0) FB_SCAN_MINE(0, KP_, 8); else if (mode == 1) FB_SCAN_MINE(1, KP_, 8); else FB_SCAN_MINE(2, KP_, 8); }         \
+    if (rp == 4) FB_SCAN_MODE(KP_, 4);                              \
+    else FB_SCAN_MODE(KP_, 8);                                      \
     break;
-  if (kp == 32 && rp == 16) {
-    if (mode == 0) FB_SCAN_MINE(0, 32, 16); else if (mode == 1) FB_SCAN_MINE(1, 32, 16); else FB_SCAN_MINE(2, 32, 16);
-  } else {
-    switch (kp) {
-      FB_SCAN(1) FB_SCAN(2) FB_SCAN(4) FB_SCAN(8) FB_SCAN(16) FB_SCAN(32)
-      default: return fb_fail(1, "state_scan: no kernel for %d lanes a column", kp);
+  // chunks side by side: their contributions, their starting states, then the outputs
+  for (int as_mode = n_chunks > 1 ? 3 : mode;; as_mode = mode) {
+    if (kp == 32 && rp == 16) {
+      FB_SCAN_MODE(32, 16);
+    } else {
+      switch (kp) {
+        FB_SCAN(1) FB_SCAN(2) FB_SCAN(4) FB_SCAN(8) FB_SCAN(16) FB_SCAN(32)
+        default: return fb_fail(1, "state_scan: no kernel for %d lanes a column", kp);
+      }
     }
+    if (as_mode == mode) break;
+    fb_launch(scan_chunk_starts_kernel, dim3(n_seqs, H, (dim * vdim + 255) / 256), dim3(256), 0,
+              stream, a);
   }
 #undef FB_SCAN
+#undef FB_SCAN_MODE
 #undef FB_SCAN_MINE
 #undef FB_SCAN_LAUNCH
   return fb_check_launch("state_scan");

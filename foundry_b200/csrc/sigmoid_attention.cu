@@ -1,9 +1,11 @@
 // Grouped-query attention whose weights are sigmoids, not a softmax, over the
 // keys of the query's own chunk of the sequence; and the kernel in front of it.
 //
+//   (q | k | v rows first plus a bias vector, where given)
 //   q, k: per head  x / sqrt(mean(x^2) + eps) * w   (w [dim], the same for every head;
 //         absent: no weight), then rotated on the first `rot` elements of a head:
-//         (x_i, x_{i + rot/2}) at position p turn by the angle p * f_i
+//         (x_i, x_{i + rot/2}) at position p turn by the angle p * f_i, cosine and sine
+//         times `rot_factor`
 //   v:    per head  x / sqrt(mean(x^2) + eps)  where `value_norm`; cached so
 //   s_ij = (q_i . k_j) * scale + bias[head]
 //   j visible to i  iff  j <= i and floor(i / chunk) == floor(j / chunk)   (chunk 0: j <= i)
@@ -51,12 +53,14 @@ __device__ __forceinline__ void sg_load8<__nv_bfloat16>(const __nv_bfloat16* p, 
 // 1 turns elements (2i, 2i + 1) instead of (i, i + rot / 2); G may be 0 (a mixer that
 // reads another's keys and values has queries only).
 template <typename T>
-__global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld, T* __restrict__ q_out,
+__global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld,
+                                            const float* __restrict__ bias, T* __restrict__ q_out,
                                             const float* __restrict__ wq,
                                             const float* __restrict__ wk, float eps,
                                             int qk_norm, int value_norm,
                                             const double* __restrict__ freq, int rot,
-                                            int interleaved, const int* __restrict__ positions,
+                                            int interleaved, float rot_factor,
+                                            const int* __restrict__ positions,
                                             const int* __restrict__ seq_of_token,
                                             const int* __restrict__ page_table, int max_pages,
                                             T* __restrict__ k_cache, T* __restrict__ v_cache,
@@ -73,8 +77,8 @@ __global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld, T* _
   float* cs = sg_smem;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     const double angle = (double)pos * freq[i];
-    cs[i] = (float)cos(angle);
-    cs[half + i] = (float)sin(angle);
+    cs[i] = (float)cos(angle) * rot_factor;
+    cs[half + i] = (float)sin(angle) * rot_factor;
   }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
@@ -95,9 +99,10 @@ __global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld, T* _
     const float* src = is_q ? row + (size_t)g * dim
                             : is_k ? row + (size_t)H * dim + (size_t)g * dim
                                    : row + (size_t)(H + G) * dim + (size_t)g * vdim;
+    const float* badd = bias != nullptr ? bias + (src - row) : nullptr;
     float ss = 0.f;
     for (int d = lane; d < n; d += 32) {
-      const float x = __ldcg(src + d);
+      const float x = __ldcg(src + d) + (badd != nullptr ? badd[d] : 0.f);
       buf[d] = x;
       ss = fmaf(x, x, ss);
     }
@@ -432,10 +437,12 @@ __global__ void attention_sigmoid_runs_kernel(const float* partial, int runs, T*
 }
 }  // namespace
 
-FB_API int fb_head_norm_rope_cache_write(const float* qkv, long long ld, void* q_out, int dtype,
+FB_API int fb_head_norm_rope_cache_write(const float* qkv, long long ld, const float* bias,
+                                         void* q_out, int dtype,
                                          const float* wq, const float* wk, float eps,
                                          int qk_norm, int value_norm, const double* freq,
-                                         int rot, int interleaved, const int* positions,
+                                         int rot, int interleaved, float rot_factor,
+                                         const int* positions,
                                          const int* seq_of_token,
                                          const int* page_table, int max_pages, void* k_cache,
                                          void* v_cache, long long k_page, long long k_head,
@@ -455,9 +462,8 @@ FB_API int fb_head_norm_rope_cache_write(const float* qkv, long long ld, void* q
   FB_REQUIRE(smem <= 48 * 1024, "head_norm_rope_cache_write: heads of %d do not fit", head_floats);
   const int parts = T <= 256 ? (heads + warps - 1) / warps : 1;  // few tokens: more blocks
   FB_DISPATCH_DTYPE(dtype, E, (fb_launch(head_norm_rope_cache_kernel<E>, dim3(T, parts), dim3(warps * 32),
-      smem, stream, qkv, ld, (E*)q_out, wq, wk, eps, qk_norm, value_norm, freq, rot, interleaved,
-      positions,
-      seq_of_token, page_table, max_pages, (E*)k_cache, (E*)v_cache, k_page, k_head, v_page,
+      smem, stream, qkv, ld, bias, (E*)q_out, wq, wk, eps, qk_norm, value_norm, freq, rot, interleaved,
+      rot_factor, positions, seq_of_token, page_table, max_pages, (E*)k_cache, (E*)v_cache, k_page, k_head, v_page,
       v_head, H, G, dim, vdim, write_cache, head_floats)));
   return fb_check_launch("head_norm_rope_cache_write");
 }

@@ -188,12 +188,10 @@ class Model:
         rows = torch.empty((n, spec.hidden_size), dtype=torch.float32, device=self.device)
         ops.gather_rows(resid, ctx.want_rows, rows)
         rows_delta = None
-        if isinstance(delta, ops.NormedDelta):
+        if isinstance(delta, (ops.NormedDelta, ops.PostNormed)):
             # a last output whose own norm is still to come: that norm works row by row,
             # so it is applied to the wanted rows only, by the final norm's pass
-            values = torch.empty((n, spec.hidden_size), dtype=delta.values.dtype, device=self.device)
-            ops.gather_rows(delta.values, ctx.want_rows, values)
-            rows_delta, delta = ops.NormedDelta(values, delta.weight, delta.bias, delta.eps), None
+            rows_delta, delta = delta.take(ctx.want_rows, n), None
         scale = None
         if isinstance(delta, ops.ScaledDelta):  # joins the residual times a constant
             delta, scale = delta.values, delta.scale

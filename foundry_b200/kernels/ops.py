@@ -26,7 +26,11 @@ c_void_p, c_int, c_ll, c_float, c_ull = (ctypes.c_void_p, ctypes.c_int, ctypes.c
                                          ctypes.c_float, ctypes.c_ulonglong)
 
 _SIGNATURES = {
-    "fb_embed_gather": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "fb_embed_gather": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
+                        c_void_p],
+    "fb_post_norm_add": [c_void_p, c_int, c_ll, c_void_p, c_int, c_ll, c_void_p, c_void_p, c_float,
+                         c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
+                         c_void_p],
     "fb_add_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_ll, c_void_p, c_float, c_void_p, c_int,
                        c_int, c_int, c_float, c_void_p],
     "fb_silu_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -93,8 +97,9 @@ _SIGNATURES = {
                      c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int,
                      c_void_p],
     "fb_softcap": [c_void_p, c_ll, c_float, c_void_p],
-    "fb_head_norm_rope_cache_write": [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_void_p, c_float,
-                                      c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
+    "fb_head_norm_rope_cache_write": [c_void_p, c_ll, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                                      c_float, c_int, c_int, c_void_p, c_int, c_int, c_float,
+                                      c_void_p, c_void_p,
                                       c_void_p, c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll,
                                       c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "fb_attention_sigmoid": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p,
@@ -155,7 +160,10 @@ _SIGNATURES = {
                       c_void_p, c_void_p],
     "fb_state_scan": [c_int, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll,
                       c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_ll, c_void_p, c_void_p, c_void_p,
-                      c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                      c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
+                      c_void_p, c_int, c_void_p],
+    "fb_low_rank_decay": [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int,
+                          c_int, c_int, c_void_p],
     "fb_head_norm_gate": [c_void_p, c_void_p, c_int, c_void_p, c_ll, c_int, c_float, c_void_p,
                           c_ll, c_float, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "fb_unary_cast": [c_void_p, c_ll, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -444,14 +452,16 @@ def plain(x):
 
 
 # ------------------------------------------------------------------ embedding
-def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """out[t,:] = table[ids[t],:] as float32; `out` is [T, H] float32."""
+def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor,
+                 scale: float = 1.0) -> torch.Tensor:
+    """out[t,:] = table[ids[t],:] * scale as float32; `out` is [T, H] float32."""
     V, H = table.shape
     T = ids.numel()
     if out.shape != (T, H):
         raise KernelError(f"embed_gather: out is {tuple(out.shape)}, expected {(T, H)}")
     _call("fb_embed_gather", _dev(table, "table"), code_of(table.dtype),
-          _dev(ids, "ids", torch.int32), _dev(out, "out", torch.float32), T, H, V, _stream())
+          _dev(ids, "ids", torch.int32), _dev(out, "out", torch.float32), T, H, V, float(scale),
+          _stream())
     return out
 
 
@@ -1680,6 +1690,96 @@ class NormedDelta:
         ln_add_ln(resid, self, None, None, self.eps, None)
         return None
 
+    def take(self, rows: torch.Tensor, n: int) -> "NormedDelta":
+        """The same for `n` rows of the step only (the norm works row by row)."""
+        return NormedDelta(_taken(self.values, rows, n), self.weight, self.bias, self.eps, self.scale)
+
+
+def _taken(values, rows: torch.Tensor, n: int) -> torch.Tensor:
+    if isinstance(values, Planes):
+        values = values.sum(torch.float32)
+    out = torch.empty((n, values.shape[1]), dtype=values.dtype, device=values.device)
+    return gather_rows(values, rows, out)
+
+
+class NormedPair:
+    """Two parts' outputs side by side, each still to pass an RMS norm of its own:
+    scale * (a / rms(a) * weight_a + b / rms(b) * weight_b). Float32 rows or split-K
+    `Planes`; the norm behind the pair makes it in its own pass (`post_norm_add`)."""
+
+    def __init__(self, a, weight_a: torch.Tensor, b, weight_b: torch.Tensor, eps: float,
+                 scale: float):
+        self.a, self.weight_a, self.b, self.weight_b = a, weight_a, b, weight_b
+        self.eps, self.scale = float(eps), float(scale)
+
+    @property
+    def shape(self):
+        return self.a.shape
+
+
+class PostNormed:
+    """The output of a part that still has to pass an RMS norm of its own before it joins
+    the residual: resid += y / rms(y) * weight, y being `values` (float32 rows, split-K
+    `Planes` or a `NormedPair` with the same eps). Whatever reads the stream next makes
+    that sum in its own pass (`post_norm_add`); `settle` makes it alone."""
+
+    def __init__(self, values, weight: torch.Tensor, eps: float):
+        self.values, self.weight, self.eps = values, weight, float(eps)
+
+    def settle(self, resid: torch.Tensor) -> None:
+        post_norm_add(resid, self, None, self.eps, None)
+        return None
+
+    def take(self, rows: torch.Tensor, n: int) -> "PostNormed":
+        """The same for `n` rows of the step only (the norms work row by row)."""
+        y = self.values
+        if isinstance(y, NormedPair):
+            y = NormedPair(_taken(y.a, rows, n), y.weight_a, _taken(y.b, rows, n), y.weight_b, y.eps,
+                           y.scale)
+        else:
+            y = _taken(y, rows, n)
+        return PostNormed(y, self.weight, self.eps)
+
+
+def _float_planes(y, shape, name: str):
+    """(pointer, planes, elements from plane to plane) of float32 rows or `Planes`."""
+    if y is None:
+        return 0, 1, 0
+    count, stride = 1, 0
+    if isinstance(y, Planes):
+        count, stride, y = y.count, shape[0] * shape[1], y.tensor
+    if tuple(y.shape[-2:]) != tuple(shape):
+        raise KernelError(f"post_norm_add: {name} is {tuple(y.shape)}, resid {tuple(shape)}")
+    return _dev(y, name, torch.float32), count, stride
+
+
+def post_norm_add(resid: torch.Tensor, pending: Optional[PostNormed], weight: Optional[torch.Tensor],
+                  eps: float, out: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+    """resid += the pending output behind its norm (None: nothing to add), in place, float32;
+    out = resid in out's type, or resid / rms(resid) * weight where a weight is given; with
+    `out=None` only the sum is made. One pass over the rows takes one eps."""
+    T, W = resid.shape
+    a = b = wa = wb = w1 = None
+    scale = 1.0
+    if pending is not None:
+        a, w1 = pending.values, pending.weight
+        if pending.eps != float(eps) or (isinstance(a, NormedPair) and a.eps != float(eps)):
+            raise KernelError(f"post_norm_add: norms with eps {pending.eps} in a pass with {eps}")
+        if isinstance(a, NormedPair):
+            a, wa, b, wb, scale = a.a, a.weight_a, a.b, a.weight_b, a.scale
+    for name, w in (("weight_a", wa), ("weight_b", wb), ("post weight", w1), ("weight", weight)):
+        if w is not None and tuple(w.shape) != (W,):
+            raise KernelError(f"post_norm_add: {name} is {tuple(w.shape)}, expected {(W,)}")
+    if out is not None and tuple(out.shape) != (T, W):
+        raise KernelError(f"post_norm_add: out is {tuple(out.shape)}, resid {(T, W)}")
+    f32 = lambda t, n: 0 if t is None else _dev(t, n, torch.float32)
+    _call("fb_post_norm_add", *_float_planes(a, (T, W), "values"), *_float_planes(b, (T, W), "b"),
+          f32(wa, "weight_a"), f32(wb, "weight_b"), scale, f32(w1, "post weight"),
+          f32(weight, "weight"), _dev(resid, "resid", torch.float32),
+          0 if out is None else _dev(out, "out"), F32 if out is None else code_of(out.dtype), T, W,
+          float(eps), _stream())
+    return out
+
 
 class DepthMix:
     """A stream that is still to be replaced by a weighted sum over the streams
@@ -2089,12 +2189,16 @@ def head_norm_rope_cache_write(qkv: torch.Tensor, q_out: torch.Tensor,
                                value_norm: bool, freq: Optional[torch.Tensor], positions,
                                seq_of_token, page_table, k_cache, v_cache, H: int, G: int,
                                dim: int, vdim: int, write_cache: bool = True,
-                               qk_norm: bool = True, pairing: str = "half") -> torch.Tensor:
+                               qk_norm: bool = True, pairing: str = "half",
+                               bias: Optional[torch.Tensor] = None,
+                               rot_factor: float = 1.0) -> torch.Tensor:
     """Per-head RMS norms of queries and keys (weights [dim] shared by the heads, or
     none; `qk_norm` False: queries and keys stay as they are), the rotation of their first
     2 * len(freq) elements (`pairing` "half": element i with element i + len(freq);
     "interleaved": 2i with 2i + 1; `freq` float64), the values' RMS norm without weight
     where `value_norm`; queries to `q_out`, keys and values into the token's cache row.
+    `bias` (float32 [H * dim + G * (dim + vdim)]) is added to the rows first; `rot_factor`
+    multiplies the rotation's cosines and sines.
     `qkv`: float32 rows [q | k | v]; with G = 0 rows of queries only (nothing is cached)."""
     T = qkv.shape[0]
     kp = vp = 0
@@ -2107,12 +2211,15 @@ def head_norm_rope_cache_write(qkv: torch.Tensor, q_out: torch.Tensor,
     for name, w in (("wq", wq), ("wk", wk)):
         if w is not None and tuple(w.shape) != (dim,):
             raise KernelError(f"head_norm_rope_cache_write: {name} {tuple(w.shape)} for heads of {dim}")
+    if bias is not None and bias.numel() != H * dim + G * (dim + vdim):
+        raise KernelError(f"head_norm_rope_cache_write: {bias.numel()} biases for {H} + {G} heads")
     _call("fb_head_norm_rope_cache_write", _dev(qkv, "qkv", torch.float32, contiguous=False),
-          _rows(qkv, "qkv"), _dev(q_out, "q_out"), code_of(q_out.dtype),
-          0 if wq is None else _dev(wq, "wq", torch.float32),
+          _rows(qkv, "qkv"), 0 if bias is None else _dev(bias, "bias", torch.float32),
+          _dev(q_out, "q_out"), code_of(q_out.dtype), 0 if wq is None else _dev(wq, "wq", torch.float32),
           0 if wk is None else _dev(wk, "wk", torch.float32), float(eps), 1 if qk_norm else 0,
           1 if value_norm else 0, 0 if freq is None else _dev(freq, "freq", torch.float64), rot,
-          _pairing_code(pairing), _dev(positions, "positions", torch.int32), _dev(seq_of_token, "seq_of_token", torch.int32),
+          _pairing_code(pairing), float(rot_factor), _dev(positions, "positions", torch.int32),
+          _dev(seq_of_token, "seq_of_token", torch.int32),
           _dev(page_table, "page_table", torch.int32), page_table.shape[1], kp, vp, *ks, *vs,
           T, H, G, dim, vdim, 1 if write_cache else 0, _stream())
     return q_out
@@ -2277,22 +2384,61 @@ def decay_gate(x: torch.Tensor, per_head: int, bias: torch.Tensor, A: Optional[t
     return out
 
 
-SCAN_DELTA, SCAN_WKV, SCAN_SSD = 0, 1, 2
+SCAN_DELTA, SCAN_WKV, SCAN_LINEAR = 0, 1, 2
+SCAN_SSD = SCAN_LINEAR  # with one decay a head, a step size and a skip
+# Chunks of a prompt that a scan works side by side (not the delta rule, whose update reads
+# the state): at least this many tokens a chunk, and about this many warps in all.
+SCAN_CHUNK_TOKENS = int(_os.environ.get("FOUNDRY_B200_SCAN_CHUNK_TOKENS", "64"))  # 0: one by one
+SCAN_CHUNK_WARPS = 148 * 64
+
+
+def scan_chunks(ctx, mode: int, H: int, dim: int, vdim: int):
+    """(chunks a sequence, tokens a chunk) of a step's scan. A chunked scan walks every token
+    twice, so it takes at least four chunks, and enough idle warps, to be worth it."""
+    longest, least = ctx.max_q_len, SCAN_CHUNK_TOKENS
+    if mode == SCAN_DELTA or ctx.is_decode or least <= 0 or longest < 4 * least:
+        return 1, 0
+    warps = max(1, ctx.n_seqs * H * ((vdim * ((dim + 7) // 8) + 31) // 32))
+    count = min((longest + least - 1) // least, SCAN_CHUNK_WARPS // warps)
+    if count < 4:
+        return 1, 0
+    chunk = ((longest + count - 1) // count + 15) // 16 * 16
+    return (longest + chunk - 1) // chunk, chunk
+
+
+def low_rank_decay(low: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, tau: float,
+                   out: torch.Tensor) -> torch.Tensor:
+    """out[t, c] = sigmoid(low[t] . weight[c] + bias[c])^(1 / tau), in 32-bit: `low` float32 rows
+    [T, rank] (possibly strided), `weight` [n, rank] as stored, `bias` and `out` float32."""
+    T, rank = low.shape
+    n = weight.shape[0]
+    if tuple(weight.shape) != (n, rank) or bias.numel() != n or tuple(out.shape) != (T, n):
+        raise KernelError(f"low_rank_decay: {tuple(low.shape)} x {tuple(weight.shape)}")
+    _call("fb_low_rank_decay", _dev(low, "low", torch.float32, contiguous=False), _rows(low, "low"),
+          _dev(weight, "weight"), code_of(weight.dtype), _dev(bias, "bias", torch.float32),
+          float(tau), _dev(out, "out", torch.float32), T, rank, n, _stream())
+    return out
 
 
 def state_scan(ctx, mode: int, q, k, v, g, state: StateRows, field: str, out: torch.Tensor,
                H: int, rep: int, dim: int, vdim: int, beta=None, bonus=None,
-               decay_per_head: bool = False) -> torch.Tensor:
+               decay_per_head: bool = False, out_scale: float = 1.0) -> torch.Tensor:
     """The recurrence of csrc/sequence_mix.cu over every sequence of the step.
     q, k: float32 views [T, >= (H / rep) * dim]; v [T, >= H * vdim]; g [T, H * dim], or
     [T, H] with `decay_per_head` (one decay for all key channels of a head);
     beta (delta) a float32 view [T, >= H]; bonus (wkv) [H, dim]; out float32 [T, H * vdim].
-    `SCAN_SSD`: S <- g S + k (beta v)^T; out = S^T q + bonus v, with one decay a head, `beta`
-    the step size as it is ([T, >= H]) and `bonus` the skip ([H])."""
+    `SCAN_LINEAR`: S <- diag(g) S + k (beta v)^T; out = out_scale S^T q + bonus v, with `beta`
+    the step size as it is ([T, >= H]; None: 1) and `bonus` the skip ([H]; None: 0).
+    Long prompts work their chunks of tokens side by side where the recurrence allows it."""
     T = out.shape[0]
     if out.shape != (T, H * vdim) or out.dtype != torch.float32 or not out.is_contiguous():
         raise KernelError("state_scan: out must be contiguous float32 [T, heads * vdim]")
     f32 = torch.float32
+    n_chunks, chunk = scan_chunks(ctx, mode, H, dim, vdim)
+    starts = decays = None
+    if n_chunks > 1:
+        starts = torch.empty((ctx.n_seqs, n_chunks, H, dim * vdim), dtype=f32, device=out.device)
+        decays = torch.empty((ctx.n_seqs, n_chunks, H, dim), dtype=f32, device=out.device)
     _call("fb_state_scan", mode, _dev(q, "q", f32, contiguous=False), _rows(q, "q"),
           _dev(k, "k", f32, contiguous=False), _rows(k, "k"),
           _dev(v, "v", f32, contiguous=False), _rows(v, "v"),
@@ -2302,7 +2448,9 @@ def state_scan(ctx, mode: int, q, k, v, g, state: StateRows, field: str, out: to
           0 if bonus is None else _dev(bonus, "bonus", f32), state.rows.data_ptr(), state.stride,
           state.offset[field], out.data_ptr(), _dev(ctx.cu_tokens, "cu_tokens", torch.int32),
           _dev(ctx.slots, "slots", torch.int32), ctx.n_seqs, H, rep, dim, vdim,
-          1 if decay_per_head else 0, 0 if ctx.is_decode else 1, _stream())
+          1 if decay_per_head else 0, float(out_scale), n_chunks, chunk,
+          0 if starts is None else starts.data_ptr(), 0 if decays is None else decays.data_ptr(),
+          0 if ctx.is_decode else 1, _stream())
     return out
 
 

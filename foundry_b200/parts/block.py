@@ -189,6 +189,88 @@ class SandwichNormBlock(Part):
                             self.depth)
 
 
+@register_block("post_norm_residual")
+class PostNormBlock(Part):
+    """A norm BEHIND each part and none in front, the parts reading the stream itself:
+
+        x <- x + post1(mixer(x));  x <- x + post2(feed_forward(x))
+
+    the second line only where the layer has a feed-forward. A part's output leaves with
+    its norm still to be applied (the post-norm's `pending`), and the next reader of the
+    stream makes the norm, the sum and its own input in one pass over the row. What stands
+    in front of the parts is the layer's `mixer_norm` / `feed_forward_norm`, normally
+    `stream_input`."""
+    replay_safe = True
+
+    def __init__(self, layer: LayerSpec, *, dtype: torch.dtype, device: torch.device):
+        ctx = dict(dtype=dtype, device=device)
+        if layer.mixer_post_norm is None:
+            raise ValueError("post_norm_residual needs a norm behind the mixer")
+        self.prefix = layer.prefix
+        self.names = dict(layer.names)
+        self.mixer = MIXERS.build(layer.mixer, **ctx)
+        self.mixer_norm = NORMS.build(layer.mixer_norm, **ctx)
+        self.mixer_post_norm = NORMS.build(layer.mixer_post_norm, **ctx)
+        self.feed_forward = self.feed_forward_norm = self.feed_forward_post_norm = None
+        if layer.feed_forward is not None:
+            if layer.feed_forward_norm is None or layer.feed_forward_post_norm is None:
+                raise ValueError("post_norm_residual: a feed-forward needs its norm")
+            self.feed_forward = FEED_FORWARDS.build(layer.feed_forward, **ctx)
+            self.feed_forward_norm = NORMS.build(layer.feed_forward_norm, **ctx)
+            self.feed_forward_post_norm = NORMS.build(layer.feed_forward_post_norm, **ctx)
+
+    def _named(self):
+        p, n = self.prefix, self.names
+        named = [(self.mixer_norm, f"{p}.{n.get('mixer_norm', '')}"),
+                 (self.mixer, f"{p}.{n['mixer']}"),
+                 (self.mixer_post_norm, f"{p}.{n['mixer_post_norm']}")]
+        if self.feed_forward is not None:
+            named += [(self.feed_forward_norm, f"{p}.{n.get('feed_forward_norm', '')}"),
+                      (self.feed_forward, f"{p}.{n['feed_forward']}"),
+                      (self.feed_forward_post_norm, f"{p}.{n['feed_forward_post_norm']}")]
+        return named
+
+    def parts(self):
+        return [part for part, _ in self._named()]
+
+    def expected_tensors(self, prefix: str = "") -> Dict[str, ExpectedTensor]:
+        out: Dict[str, ExpectedTensor] = {}
+        for part, name in self._named():
+            out.update(part.expected_tensors(name))
+        return out
+
+    def load(self, prefix: str, fetch: Fetch) -> None:
+        for part, name in self._named():
+            part.load(name, fetch)
+
+    def cache_request(self):
+        return self.mixer.cache_request()
+
+    def first_weight(self):
+        return first_weight_of(self.mixer)
+
+    def forward(self, ctx, resid: torch.Tensor, delta, cache):
+        after_block = getattr(ctx, "reads_after_part", None)
+        ctx.residual_sink = None  # the norm behind a part needs its whole row: no product makes the sum
+        x = self.mixer_norm.add_norm(resid, delta)
+        if self.feed_forward is None:
+            ctx.reads_after_part = after_block
+            return self.mixer_post_norm.pending(_as_float_planes(self.mixer.forward(ctx, x, cache)))
+        ctx.reads_after_part = first_weight_of(self.feed_forward)
+        mixed = self.mixer_post_norm.pending(_as_float_planes(self.mixer.forward(ctx, x, cache)))
+        x = self.feed_forward_norm.add_norm(resid, mixed)
+        ctx.reads_after_part = after_block
+        return self.feed_forward_post_norm.pending(
+            _as_float_planes(self.feed_forward.forward(ctx, x)))
+
+
+def _as_float_planes(y):
+    """A part's output as a norm behind it takes it: split-K planes and pairs as they are,
+    16-bit rows widened."""
+    from ..kernels import ops
+    return y if isinstance(y, (ops.Planes, ops.NormedPair)) else _as_float_rows(y)
+
+
 # keys of `ctx.shared`: the stream as the embedding left it (the model puts it there for
 # blocks that say `needs_embedding_output`), and the blocks' kept results [depth, T, W]
 EMBEDDING_OUTPUT = "embedding_output"

@@ -1,6 +1,7 @@
 """From token ids to the first residual rows.
 
-`lookup` is the plain table gather (src/nn/linear.rs:54-69). `scaled_sinusoidal`
+`lookup` is the plain table gather (src/nn/linear.rs:54-69), times a constant
+where one is given. `scaled_sinusoidal`
 multiplies the table row by a constant and adds a sinusoidal position vector:
 
     x[2i] = E[token][2i] * scale + sin(p * base^(-2i / width)),  x[2i+1] = ... + cos(same)
@@ -29,12 +30,13 @@ register_embedding = EMBEDDINGS.register
 class Lookup(Part):
     replay_safe = True
 
-    def __init__(self, *, dtype: torch.dtype, device: torch.device):
+    def __init__(self, scale: float = 1.0, *, dtype: torch.dtype, device: torch.device):
+        self.scale = float(scale)
         self.dtype, self.device = dtype, device
 
     def forward(self, ctx, table: torch.Tensor, out: torch.Tensor,
                 copy: Optional[torch.Tensor] = None) -> torch.Tensor:
-        ops.embed_gather(table, ctx.token_ids, out)
+        ops.embed_gather(table, ctx.token_ids, out, self.scale)
         if copy is not None:
             copy.copy_(out)
         return out

@@ -53,7 +53,7 @@ class LoopInput(Part):
         new un-added output (None)."""
         if not 0 <= number < self.times:
             raise ValueError(f"pass {number} of a loop of {self.times}")
-        if isinstance(delta, ops.NormedDelta):
+        if isinstance(delta, (ops.NormedDelta, ops.PostNormed)):
             delta = delta.settle(resid)
         elif delta is not None:
             delta = ops.NormedDelta(ops.plain(delta), None, None, 1.0).settle(resid)

@@ -23,7 +23,9 @@ class SwiGLU(Part):
 
     def __init__(self, hidden_size: int, intermediate_size: int, *, dtype: torch.dtype,
                  device: torch.device, names=("gate_proj", "up_proj", "down_proj"),
-                 suffix: str = ".weight", activation: str = "silu"):
+                 suffix: str = ".weight", activation: str = "silu", float_out: bool = False):
+        # the down product's 32-bit sums leave unrounded (a norm of the output stands behind)
+        self.out_dtype = torch.float32 if float_out else None
         if activation not in ops.GLU_ACTIVATIONS:
             raise ValueError(f"activation {activation!r}; known: {sorted(ops.GLU_ACTIVATIONS)}")
         self.activation = activation
@@ -66,7 +68,7 @@ class SwiGLU(Part):
 
     def forward(self, ctx, x):
         hidden = self.hidden(x)
-        return self.down.forward(hidden, allow_planes=True,
+        return self.down.forward(hidden, out_dtype=self.out_dtype, allow_planes=True,
                                  then_reads=getattr(ctx, "reads_after_part", None),
                                  residual=getattr(ctx, "residual_sink", None))
 

@@ -23,6 +23,14 @@ def product_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return y if isinstance(y, torch.Tensor) else out
 
 
+def product_planes(x: torch.Tensor, w: torch.Tensor, then_reads=None):
+    """`product_f32` for a consumer that sums split-K planes while it reads: float32 rows or
+    `ops.Planes`."""
+    if x.shape[0] == 0 or x.dtype == torch.float32 or x.shape[1] < SMALL_K:
+        return product_f32(x, w)
+    return matmul_nt(x, w, out_dtype=torch.float32, allow_planes=True, then_reads=then_reads)
+
+
 def product_to_residual(ctx, x: torch.Tensor, w: torch.Tensor):
     """A part's last product, whose result joins the residual: float32 as
     `product_f32` gives it, or, where the block offers the next norm's sink

@@ -38,6 +38,13 @@
     out = Wo [ rms_parts(y * silu(z)) * norm ]   (the gate first; the row normalised in
     `norm_groups` equal parts, each by its own root mean square)
 
+`gated_linear_attention`: a linear recurrence with a decay per key channel.
+
+    q = Wq h, k = Wk h  (heads x dim),  v = Wv h  (heads x vdim), no convolution;
+    a = sigmoid(Wa2 (Wa1 h) + b)^(1 / tau)  per head and key channel
+    S <- diag(a) S + k v^T;  o = S^T q * dim^-1/2
+    out = Wo [ o / rms(o) * norm * silu(Wg h) ]      (norm [vdim], shared by heads)
+
 The state S is float32 and, with the inputs that the next step needs from this
 one (the convolution's last taps - 1 inputs; the last h), one float32 row per
 sequence in the cache's state storage. Decays, step sizes, gates, unit norms
@@ -193,6 +200,79 @@ class GatedDelta(Part):
         y = torch.empty((T, H * v), dtype=x.dtype, device=x.device)
         ops.head_norm_gate(o, self.norm, False, p[:, C:at], self.gate, self.eps, y, H, v)
         return product_to_residual(ctx, y, self.o)
+
+
+@register_mixer("gated_linear_attention")
+class GatedLinearAttention(Part):
+    """Linear attention with a decay per key channel (see the module's notes). Tensor names
+    under the prefix: `q k v g a1 a2 a2.b norm o`."""
+    replay_safe = True
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, decay_rank: int, tau: float,
+                 eps: float, gate: str = "silu", *, dtype: torch.dtype, device: torch.device):
+        if dim > 512:
+            raise ValueError(f"{dim} key channels a head: the recurrence kernel holds at most 512")
+        if gate not in ("silu", "sigmoid"):
+            raise ValueError(f"output gate {gate!r}; known: silu, sigmoid")
+        if tau <= 0:
+            raise ValueError(f"the decays' root {tau} must be positive")
+        self.width, self.heads, self.dim, self.vdim = width, heads, dim, vdim
+        self.decay_rank, self.tau, self.eps, self.gate = decay_rank, float(tau), float(eps), gate
+        self.dtype, self.device = dtype, device
+        self.fields = [("S", heads * dim * vdim)]
+
+    def _shapes(self):
+        W, n, m = self.width, self.heads * self.dim, self.heads * self.vdim
+        return {"q": (n, W), "k": (n, W), "v": (m, W), "g": (m, W), "a1": (self.decay_rank, W),
+                "a2": (n, self.decay_rank), "a2.b": (n,), "norm": (self.vdim,), "o": (W, m)}
+
+    def expected_tensors(self, prefix: str) -> Dict[str, ExpectedTensor]:
+        return {f"{prefix}.{n}": ExpectedTensor(s) for n, s in self._shapes().items()}
+
+    def load(self, prefix: str, fetch: Fetch) -> None:
+        f = lambda n: fetch(f"{prefix}.{n}")
+        # every projection of h in one product: q | k | v | gate | decay low rank
+        self.w_in = torch.cat([f("q"), f("k"), f("v"), f("g"), f("a1")], 0).contiguous()
+        self.a2, self.o = f("a2").contiguous(), f("o").contiguous()
+        self.decay_bias, self.norm = _f32(f("a2.b")), _f32(f("norm"))
+
+    def cache_request(self) -> StateRequest:
+        return StateRequest((sum(n for _, n in self.fields),), torch.float32)
+
+    def first_weight(self):
+        return self.w_in
+
+    # the pieces of a mixer that may stand beside another one (parts/parallel.py)
+    def input_weight(self) -> torch.Tensor:
+        return self.w_in
+
+    def output_weight(self) -> torch.Tensor:
+        return self.o
+
+    @property
+    def inner_size(self) -> int:
+        return self.heads * self.vdim
+
+    def between(self, ctx, p: torch.Tensor, cache: StateView, out: torch.Tensor,
+                out_scale: float = 1.0) -> torch.Tensor:
+        """From the input projection `p` (float32 rows [q | k | v | gate | low rank]) to the
+        normalised, gated rows in `out` (rows may lie further apart), times `out_scale`."""
+        T, H, d, v = p.shape[0], self.heads, self.dim, self.vdim
+        n, m = H * d, H * v
+        f32 = dict(dtype=torch.float32, device=p.device)
+        state = ops.StateRows(cache.rows, self.fields)
+        decay = ops.low_rank_decay(p[:, 2 * n + 2 * m:2 * n + 2 * m + self.decay_rank], self.a2,
+                                   self.decay_bias, self.tau, torch.empty((T, n), **f32))
+        o = torch.empty((T, m), **f32)
+        ops.state_scan(ctx, ops.SCAN_LINEAR, p, p[:, n:], p[:, 2 * n:], decay, state, "S", o, H, 1,
+                       d, v, out_scale=d ** -0.5)
+        return ops.head_norm_gate(o, self.norm, False, p[:, 2 * n + m:], self.gate, self.eps, out,
+                                  H, v, out_scale=out_scale)
+
+    def forward(self, ctx, x, cache: StateView):
+        y = torch.empty((x.shape[0], self.inner_size), dtype=x.dtype, device=x.device)
+        self.between(ctx, product_f32(x, self.w_in), cache, y)
+        return product_f32(y, self.o)
 
 
 @register_mixer("wkv_time_mix")

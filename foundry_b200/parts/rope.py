@@ -69,6 +69,24 @@ def banded_frequencies(dims: int, base: float, factor: float = 1.0, low: float =
                     np.where(wavelength > original / low, f / factor, mixed))
 
 
+def yarn_frequencies(dims: int, base: float, factor: float, original: float, fast: float,
+                     slow: float):
+    """(float64 frequencies f_i, i < dims / 2; the factor on cosines and sines) of YaRN's
+    scaling. An element whose wavelength makes t turns in `original` positions is number
+    e(t) = dims ln(original / (2 pi t)) / (2 ln base). Elements in front of e(fast) (rounded
+    down) keep base^(-2i / dims), those behind e(slow) (rounded up) are divided by `factor`,
+    and between the two the frequencies are blended linearly in i."""
+    f = banded_frequencies(dims, base)
+
+    def element(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    first = max(math.floor(element(fast)), 0)
+    last = min(math.ceil(element(slow)), dims - 1)
+    ramp = np.clip((np.arange(dims // 2) - first) / max(last - first, 0.001), 0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 class _Rotary(Part):
     attention_factor = 1.0
     pairing = "half"  # src/models/llama/rotary_emb.rs:76-85 (rotate_half)
