@@ -127,7 +127,28 @@ def _kutepel(layers, width, heads, kv_heads, dim, ff, vocab, kv_rank, experts=16
             "residual_mult": 0.7, "layers": stack}
 
 
+def _tokovik(layers, width, heads, kv_heads, dim, ff, vocab, window=1024, state=128,
+             rank=32) -> Dict:
+    """A Tokovik stack of real layer sizes: every layer the two mixers side by side
+    (attention in a window of `window` positions with every head rotated whole, stretched
+    fourfold from 8,192 positions; gated linear attention whose heads hold `state` x
+    `state` numbers and together span the width) and a dense feed-forward."""
+    mixer = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim,
+                      "scale": dim ** -0.5, "mask": {"size": window},
+                      "rot": {"dims": dim, "base": 500000.0,
+                              "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0,
+                                          "slow": 1.0}}},
+             "right": {"heads": width // state, "dim": state, "vdim": state, "tau": 16.0,
+                       "decay_rank": rank}}
+    return {"architecture": "Tokovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 8.0}, "logit_scale": 0.5,
+            "layers": [{"type": "parallel", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}}
+                       for _ in range(layers)]}
+
+
 PRESETS: Dict[str, Dict] = {
+    "tokovik-1b-layers": _tokovik(6, 2048, 32, 8, 64, 8192, 32000),
+    "tokovik-3b-layers": _tokovik(6, 3072, 24, 8, 128, 8192, 32000),
     "kutepel-1b-layers": _kutepel(6, 2048, 32, 8, 64, 8192, 32000, 256),
     "kutepel-3b-layers": _kutepel(6, 3072, 24, 8, 128, 8192, 32000, 512),
     "vikarax-1b-layers": _vikarax(6, 2048, 32, 8, 64, 8192, 32000),

@@ -132,8 +132,8 @@ struct AttnParams {
   const void* next;      // constant data to bring into L2 for the kernel after this one
   long long next_bytes;  // 0 = none
   int trigger_next;      // 1: let the next kernel's blocks be placed once a CTA's pages are in
-  // prompts, masked form only: a key j is seen from position i iff j <= i and
-  // (window == 0 or i - j < window or j < keep_first); scores lose
+  // a key j is seen from position i iff j <= i and (window == 0 or i - j < window or
+  // j < keep_first); single tokens take the window, the masked prompt form all of this: scores lose
   // 2^(-steep (head + 1) / A) per token of distance (steep 0: no bias); with `sink`
   // the softmax's sum has one more term exp(0), which adds nothing to the output
   // (`sink_logits`, float32 per query head: the term is exp(sink_logits[head]) instead)
@@ -496,8 +496,10 @@ attn_decode_kernel(const AttnParams p) {
   const int token = p.cu_tokens[seq];
   const int kv_len = p.kv_lens[seq];
   const int n_pages = (kv_len + FB_PAGE - 1) / FB_PAGE;
-  const int per = (n_pages + p.splits - 1) / p.splits;  // a range: 1/splits of the pages
-  const int pg0 = split * per;
+  const int lo = p.window > 0 ? max(0, kv_len - p.window) : 0;  // the token's first visible key
+  const int first = lo / FB_PAGE;
+  const int per = (n_pages - first + p.splits - 1) / p.splits;  // a range: 1/splits of the pages
+  const int pg0 = first + split * per;
   const int pg1 = min(n_pages, pg0 + per);
   const int fresh = max(kv_len - (p.cu_tokens[seq + 1] - token), 0) / FB_PAGE;
 
@@ -606,7 +608,7 @@ attn_decode_kernel(const AttnParams p) {
       }
     }
     const int key0 = pg * FB_PAGE + warp * 16;  // this warp's 16 keys of the page
-    if (key0 < kv_len) {
+    if (key0 < kv_len && key0 + 16 > lo) {
       const __nv_bfloat16* tK = sK + st * 64 * D;
       const __nv_bfloat16* tV = sV + st * 64 * D;
       if constexpr (NARROW) {
@@ -632,7 +634,8 @@ attn_decode_kernel(const AttnParams p) {
 #pragma unroll
           for (int i = 1; i < NS; ++i) v += sp[i][e];
           v *= p.scale_log2;
-          if (key0 + g + (e >> 1) * 8 >= kv_len) v = -INFINITY;
+          const int key = key0 + g + (e >> 1) * 8;
+          if (key >= kv_len || key < lo) v = -INFINITY;
           s[e] = v;
           mx[e & 1] = fmaxf(mx[e & 1], v);
         }
@@ -642,7 +645,7 @@ attn_decode_kernel(const AttnParams p) {
           mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 8));
           mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 16));
         }
-        // key0 < kv_len: the warp's first key is visible, so mx is finite
+        // one of the warp's keys is visible, so mx is finite
         float corr[2], sum[2] = {0.f, 0.f};
 #pragma unroll
         for (int r = 0; r < 2; ++r) corr[r] = exp2f(m[r] - mx[r]);
@@ -694,7 +697,8 @@ attn_decode_kernel(const AttnParams p) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float v = s[n][e] * p.scale_log2;
-            if (key0 + n * 8 + 2 * t + (e & 1) >= kv_len) v = -INFINITY;
+            const int key = key0 + n * 8 + 2 * t + (e & 1);
+            if (key >= kv_len || key < lo) v = -INFINITY;
             s[n][e] = v;
             mx[e >> 1] = fmaxf(mx[e >> 1], v);
           }
@@ -956,14 +960,15 @@ FB_API int fb_attention_prefill_masked(const void* q, long long q_stride, void* 
 // n_seqs*Kh ints that are zero when the call starts (the kernel leaves them zero
 // again); with one part per pair they are not used and may be null. `stages`
 // (2 or 3) is the number of page buffers per CTA. A sequence with kv_lens == 0
-// is padding: its output rows are zeros. `trigger_next`: see AttnParams (it pays in
+// is padding: its output rows are zeros. `window` > 0: the last `window` keys only, and only
+// their pages are walked. `trigger_next`: see AttnParams (it pays in
 // front of the tcgen05 products and costs a third of the step in front of the
 // weight-streaming one, whose blocks then crowd in beside the attention's).
 FB_API int fb_attention_decode(const void* q, long long q_stride, void* out, long long out_stride,
                                const int* cu_tokens, const int* kv_lens, const int* page_table,
                                int max_pages, const void* k_cache, const void* v_cache,
                                long long page_stride, long long head_stride, int n_seqs, int A,
-                               int Kh, int D, float scale, int splits, int stages, int cluster,
+                               int Kh, int D, float scale, int window, int splits, int stages, int cluster,
                                float* ws_o, float* ws_ml, int* counters,
                                const void* next, long long next_bytes, int trigger_next,
                                const float* sink_logits, cudaStream_t stream) {
@@ -973,6 +978,7 @@ FB_API int fb_attention_decode(const void* q, long long q_stride, void* out, lon
                         v_cache, page_stride, head_stride);
   if (rc) return rc;
   FB_REQUIRE(splits >= 1 && splits <= 65535, "attention_decode: bad split count %d", splits);
+  FB_REQUIRE(window >= 0, "attention_decode: bad window %d", window);
   if (cluster < 1) cluster = 1;
   FB_REQUIRE(cluster <= MAX_CLUSTER && splits % cluster == 0,
              "attention_decode: clusters of %d do not divide %d splits (or exceed %d)", cluster,
@@ -992,6 +998,7 @@ FB_API int fb_attention_decode(const void* q, long long q_stride, void* out, lon
   p.ws_o = ws_o; p.ws_ml = ws_ml; p.counters = counters;
   p.next = next; p.next_bytes = next_bytes;
   p.trigger_next = trigger_next ? 1 : 0;
+  p.window = window;
   p.sink_logits = sink_logits;
   FB_REQUIRE(stages == 2 || stages == 3, "attention_decode: %d page buffers (2 or 3)", stages);
   if (stages == 2) {
@@ -1079,6 +1086,6 @@ FB_API int fb_attention_decode_static(const void* q, long long q_stride, void* o
   float* ws_ml = ws_o + units * 16 * D;
   return fb_attention_decode(q, q_stride, out, out_stride, cu_tokens, kv_lens, page_table,
                              max_pages, k_cache, v_cache, page_stride, head_stride, n_seqs, A, Kh,
-                             D, scale, splits, 3, 1, ws_o, ws_ml, counters, nullptr, 0, 0, nullptr,
+                             D, scale, 0, splits, 3, 1, ws_o, ws_ml, counters, nullptr, 0, 0, nullptr,
                              stream);
 }

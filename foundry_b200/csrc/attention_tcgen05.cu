@@ -34,6 +34,12 @@
 // softmax (2,700 cycles a page whatever the softmax did; taking its loads, exps
 // and stores out changed nothing).
 //
+// Keys have D elements a head and values DV, each a multiple of 8 up to 128: a tile is one or
+// two 64-element blocks along its row, and TMA fills what lies beyond the row with zeros (a
+// query block's elements beyond D belong to the next head; they meet zeros of the keys). With
+// a window, position i sees j iff 0 <= i - j < window: the block walks the pages from the one
+// that holds its first query's first key on, and masks by row at both edges.
+//
 // Shared memory (96 KB at head size 128) and tensor memory (256 columns) are
 // sized so that two CTAs share an SM: the second CTA's warps fill the gaps that
 // a row's long dependent chain leaves on the schedulers and the tensor pipe.
@@ -62,6 +68,8 @@ struct FaParams {
   const int* kv_lens;
   const int* page_table;
   int max_pages, n_seqs, A, Kh;
+  int D, DV;   // elements of a key and of a value
+  int window;  // 0: every key up to the query's own position
   float scale_log2;
   // float32 per query head, or null: a sink's score. The softmax's sum has one more
   // term exp(sink_logits[head]) that has no key and no value: it starts the running
@@ -75,32 +83,34 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <int D>
+// KS, VS: 64-element (128-byte) blocks along a key row and a value row
+template <int KS, int VS>
 struct FaSmem {
-  static constexpr int Q_BYTES = BQ * D * 2;
-  static constexpr int PAGE_BYTES = FB_PAGE * D * 2;       // one K or V page of one head
-  static constexpr int USED = Q_BYTES + 2 * ST * PAGE_BYTES + 256;
+  static constexpr int Q_BYTES = BQ * KS * 128;
+  static constexpr int K_BYTES = FB_PAGE * KS * 128;       // one K page of one head
+  static constexpr int V_BYTES = FB_PAGE * VS * 128;       // one V page of one head
+  static constexpr int USED = Q_BYTES + ST * (K_BYTES + V_BYTES) + 256;
   // never three CTAs on an SM: they would need more tensor memory than it has
   static constexpr int BYTES = USED > 77 * 1024 ? USED : 77 * 1024;
   static_assert(BYTES <= (233472 - 2 * 1024) / 2, "two CTAs must fit an SM");
 };
 
-template <int D>
+template <int KS, int VS>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                        const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const FaParams p) {
-  constexpr int SUB = D / 64;                  // 64-element (128-byte) blocks along D
+  using Smem = FaSmem<KS, VS>;
   constexpr int Q_SUB = BQ * 128;              // bytes of one query sub-tile
   constexpr int KV_SUB = FB_PAGE * 128;        // bytes of one K or V sub-tile
-  constexpr int TMEM_COLS = 256;               // 2 x 64 score columns + D output columns
+  constexpr int TMEM_COLS = 256;               // 2 x 64 score columns + VS * 64 output columns
   constexpr uint32_t O_COL = 128;
   extern __shared__ __align__(1024) uint8_t smem_raw[];  // swizzled tiles start on 1,024 bytes
   uint8_t* base = smem_raw;
   uint8_t* sQ = base;
-  uint8_t* sK = sQ + FaSmem<D>::Q_BYTES;                 // [ST][SUB][64 keys][64]
-  uint8_t* sV = sK + ST * FaSmem<D>::PAGE_BYTES;         // [ST][SUB][64 keys][64]
-  uint64_t* bars = (uint64_t*)(sV + ST * FaSmem<D>::PAGE_BYTES);
+  uint8_t* sK = sQ + Smem::Q_BYTES;                      // [ST][KS][64 keys][64]
+  uint8_t* sV = sK + ST * Smem::K_BYTES;                 // [ST][VS][64 keys][64]
+  uint64_t* bars = (uint64_t*)(sV + ST * Smem::V_BYTES);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;         // [ST]
   uint64_t* v_full = k_full + ST;      // [ST]
@@ -168,32 +178,34 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
   const int kv_len = p.kv_lens[seq];
   const int pos0 = kv_len - q_len + row0;  // position of this block's first query
   const int rows_valid = min(BQ, q_len - row0);
-  const int n_pages = (pos0 + rows_valid - 1) / FB_PAGE + 1;
-  const int* pages = p.page_table + (size_t)seq * p.max_pages;
+  // the pages the block walks; j counts from the first of them
+  const int first_page = p.window > 0 ? max(0, pos0 - p.window + 1) / FB_PAGE : 0;
+  const int n_pages = (pos0 + rows_valid - 1) / FB_PAGE + 1 - first_page;
+  const int* pages = p.page_table + (size_t)seq * p.max_pages + first_page;
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA producer
     if (lane == 0) {
       fb_pdl_wait();  // the queries and this step's keys and values come from earlier kernels
-      mbar_expect_tx(q_full, FaSmem<D>::Q_BYTES);
+      mbar_expect_tx(q_full, Smem::Q_BYTES);
 #pragma unroll
-      for (int sb = 0; sb < SUB; ++sb)
-        tma_load_2d(sQ + sb * Q_SUB, &map_q, q_full, head * D + sb * 64, tok0 + row0);
+      for (int sb = 0; sb < KS; ++sb)
+        tma_load_2d(sQ + sb * Q_SUB, &map_q, q_full, head * p.D + sb * 64, tok0 + row0);
       for (int j = 0; j < n_pages; ++j) {
         const int s = j % ST;
         const uint32_t parity = (uint32_t)((j / ST) & 1) ^ 1u;
         const int page = pages[j];
         if (!mbar_wait(&k_empty[s], parity, abort_flag, 11, j)) break;
-        mbar_expect_tx(&k_full[s], FaSmem<D>::PAGE_BYTES);
+        mbar_expect_tx(&k_full[s], Smem::K_BYTES);
 #pragma unroll
-        for (int sb = 0; sb < SUB; ++sb)
-          tma_load_3d(sK + s * FaSmem<D>::PAGE_BYTES + sb * KV_SUB, &map_k, &k_full[s], sb * 64,
+        for (int sb = 0; sb < KS; ++sb)
+          tma_load_3d(sK + s * Smem::K_BYTES + sb * KV_SUB, &map_k, &k_full[s], sb * 64,
                       kvh * FB_PAGE, page);
         if (!mbar_wait(&v_empty[s], parity, abort_flag, 10, j)) break;
-        mbar_expect_tx(&v_full[s], FaSmem<D>::PAGE_BYTES);
+        mbar_expect_tx(&v_full[s], Smem::V_BYTES);
 #pragma unroll
-        for (int sb = 0; sb < SUB; ++sb)
-          tma_load_3d(sV + s * FaSmem<D>::PAGE_BYTES + sb * KV_SUB, &map_v, &v_full[s], sb * 64,
+        for (int sb = 0; sb < VS; ++sb)
+          tma_load_3d(sV + s * Smem::V_BYTES + sb * KV_SUB, &map_v, &v_full[s], sb * 64,
                       kvh * FB_PAGE, page);
       }
     }
@@ -201,7 +213,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     // -------------------------------------------------------------- MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_qk = make_idesc(BQ, FB_PAGE);
-      constexpr uint32_t idesc_pv = make_idesc_b_mn(BQ, D);
+      constexpr uint32_t idesc_pv = make_idesc_b_mn(BQ, VS * 64);
       bool ok = mbar_wait(q_full, 0, abort_flag, 12, 0);
       for (int j = 0; j <= n_pages && ok; ++j) {
         if (j < n_pages) {
@@ -212,9 +224,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
           if (!ok) break;
           tc_fence_after();
           const uint32_t q_addr = smem_u32(sQ);
-          const uint32_t k_addr = smem_u32(sK + s * FaSmem<D>::PAGE_BYTES);
+          const uint32_t k_addr = smem_u32(sK + s * Smem::K_BYTES);
 #pragma unroll
-          for (int sb = 0; sb < SUB; ++sb)
+          for (int sb = 0; sb < KS; ++sb)
 #pragma unroll
             for (int k = 0; k < 4; ++k)
               umma(tmem_base + (uint32_t)(b * FB_PAGE), make_desc(q_addr + sb * Q_SUB + k * 32),
@@ -229,7 +241,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                mbar_wait(&v_full[s], (uint32_t)((jj / ST) & 1), abort_flag, 9, jj);
           if (!ok) break;
           tc_fence_after();
-          const uint32_t v_addr = smem_u32(sV + s * FaSmem<D>::PAGE_BYTES);
+          const uint32_t v_addr = smem_u32(sV + s * Smem::V_BYTES);
 #pragma unroll
           for (int k = 0; k < 4; ++k)  // 16 keys per instruction: 8 columns of P, 16 rows of V
             umma_a_tmem(tmem_base + O_COL, tmem_base + (uint32_t)(b * FB_PAGE + k * 8),
@@ -269,12 +281,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         }
       }
 
-      const int key0 = j * FB_PAGE;
+      const int key0 = (first_page + j) * FB_PAGE;
       const bool diagonal = key0 + FB_PAGE - 1 > pos0 + quarter * 32;  // some key may be masked
       if (diagonal) {
 #pragma unroll
         for (int e = 0; e < FB_PAGE; ++e)
           if (key0 + e > qpos) sc[e] = -INFINITY;
+      }
+      // some key may lie behind some row's window (rows of the warp reach 31 further)
+      if (p.window > 0 && key0 <= pos0 + quarter * 32 + 31 - p.window) {
+        const int behind = qpos - p.window - key0;  // keys of the page up to this one are behind it
+#pragma unroll
+        for (int e = 0; e < FB_PAGE; ++e)
+          if (e <= behind) sc[e] = -INFINITY;
       }
       // the row maximum of the raw scores, by four independent chains; the scale is
       // positive, so it can be applied to the maximum afterwards
@@ -289,14 +308,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
       const bool grow = mx > m_ref + RESCALE_STEP;  // also the first page (m_ref = -inf)
       if (__any_sync(0xffffffffu, grow)) {
-        const float corr = grow ? exp2f(m_ref - mx) : 1.0f;  // 0 on the first page
+        const float corr = grow ? exp2f(m_ref - mx) : 1.0f;  // 0 on the row's first page
         if (j > 0) {
           // the accumulator must be at rest: wait for the product of page j - 1
           ok = mbar_wait(pv_done, (uint32_t)((j - 1) & 1), abort_flag, 18, j);
           if (!ok) break;
           tc_fence_after();
 #pragma unroll 1
-          for (int c = 0; c < D; c += 32) {
+          for (int c = 0; c < VS * 64; c += 32) {
             uint32_t r[32];
             tmem_ld32(tmem_base + lane_base + O_COL + (uint32_t)c, r);
             tmem_ld_wait();
@@ -312,7 +331,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       // probabilities against the reference maximum (at most 2^8), rounded to bfloat16
       // and packed two keys to a column: the A operand of the product, in the first 32
       // columns of this page's score buffer
-      const float neg_ref = -m_ref;
+      // (a row that has seen no key yet, all of its page being behind its window: scores of
+      // -inf against a reference of 0 give probabilities of 0)
+      const float neg_ref = m_ref == -INFINITY ? 0.f : -m_ref;
       float sum4[4] = {0.f, 0.f, 0.f, 0.f};
       uint32_t packed[32];
 #pragma unroll
@@ -337,17 +358,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     if (ok) ok = mbar_wait(o_final, 0, abort_flag, 19, n_pages);
     if (ok) {
       tc_fence_after();
-      const float inv = 1.0f / l;  // every valid row saw key 0
+      const float inv = 1.0f / l;  // every valid row saw its own key
       __nv_bfloat16* dst =
-          p.out + (long long)(tok0 + row0 + row) * p.out_stride + (long long)head * D;
+          p.out + (long long)(tok0 + row0 + row) * p.out_stride + (long long)head * p.DV;
 #pragma unroll 1
-      for (int c = 0; c < D; c += 32) {
+      for (int c = 0; c < VS * 64; c += 32) {
         uint32_t r[32];
         tmem_ld32(tmem_base + lane_base + O_COL + (uint32_t)c, r);
         tmem_ld_wait();
         if (row < rows_valid) {
 #pragma unroll
           for (int e = 0; e < 32; e += 8) {
+            if (c + e >= p.DV) break;  // (whole pieces: DV is a multiple of 8)
             uint4 pk;
             __nv_bfloat162 h0 = __floats2bfloat162_rn(__uint_as_float(r[e]) * inv, __uint_as_float(r[e + 1]) * inv);
             __nv_bfloat162 h1 = __floats2bfloat162_rn(__uint_as_float(r[e + 2]) * inv, __uint_as_float(r[e + 3]) * inv);
@@ -409,18 +431,18 @@ int make_map(CUtensorMap* map, const void* ptr, int rank, const long long* dims,
   return 0;
 }
 
-template <int D>
+template <int KS, int VS>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FaParams& p,
            int q_blocks, cudaStream_t stream) {
   static bool configured[64] = {};
   if (fb_first_use_on_device(configured)) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<D>,
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<KS, VS>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         FaSmem<D>::BYTES);
+                                         FaSmem<KS, VS>::BYTES);
     if (e != cudaSuccess) return fb_fail(2, "attention_tc: %s", cudaGetErrorString(e));
   }
-  fb_launch(attn_prefill_tc_kernel<D>, dim3(p.A, q_blocks), dim3(THREADS), FaSmem<D>::BYTES, stream,
-            mq, mk, mv, p);
+  fb_launch(attn_prefill_tc_kernel<KS, VS>, dim3(p.A, q_blocks), dim3(THREADS), FaSmem<KS, VS>::BYTES,
+            stream, mq, mk, mv, p);
   return fb_check_launch("attention_prefill_tc");
 }
 
@@ -428,21 +450,23 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 
 // Prompt attention on tcgen05. q: [T, A*D] bf16 rows with stride q_stride (all
 // heads of a token contiguous); k_cache / v_cache: one cache entry's views
-// [n_pages, Kh, 64, D] with strides (page_stride, 64*D, D, 1). `q_blocks` bounds
-// the number of 128-row query blocks: the sum over sequences of ceil(q_len / 128).
-// Head sizes 64 and 128.
+// [n_pages, Kh, 64, D] with strides (k_page, 64*D, D, 1), and with DV and v_page for the
+// values. `q_blocks` bounds the number of 128-row query blocks: the sum over sequences of
+// ceil(q_len / 128). D and DV: multiples of 8 up to 128. `window`: see the file's notes.
 FB_API int fb_attention_prefill_tc(const void* q, long long q_stride, int T, void* out,
                                    long long out_stride, const int* cu_tokens, const int* kv_lens,
                                    const int* page_table, int max_pages, const void* k_cache,
-                                   const void* v_cache, long long page_stride,
-                                   long long head_stride, int n_pages, int n_seqs, int q_blocks,
-                                   int A, int Kh, int D, float scale, const float* sink_logits,
-                                   cudaStream_t stream) {
-  FB_REQUIRE(D == 64 || D == 128, "attention_tc: head size %d is not built (64, 128)", D);
+                                   const void* v_cache, long long k_page, long long k_head,
+                                   long long v_page, long long v_head, int n_pages, int n_seqs,
+                                   int q_blocks, int A, int Kh, int D, int DV, int window,
+                                   float scale, const float* sink_logits, cudaStream_t stream) {
+  FB_REQUIRE(D > 0 && DV > 0 && D <= 128 && DV <= 128 && D % 8 == 0 && DV % 8 == 0 && window >= 0,
+             "attention_tc: head sizes %d and %d are not built (multiples of 8 up to 128)", D, DV);
   FB_REQUIRE(n_seqs > 0 && A > 0 && Kh > 0 && A % Kh == 0 && T > 0 && n_pages > 0,
              "attention_tc: bad sizes");
-  FB_REQUIRE(head_stride == (long long)FB_PAGE * D, "attention_tc: the heads of a page must be contiguous");
-  FB_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && page_stride % 8 == 0 &&
+  FB_REQUIRE(k_head == (long long)FB_PAGE * D && v_head == (long long)FB_PAGE * DV,
+             "attention_tc: the heads of a page must be contiguous");
+  FB_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && k_page % 8 == 0 && v_page % 8 == 0 &&
                  ((uintptr_t)q % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
                  ((uintptr_t)k_cache % 16) == 0 && ((uintptr_t)v_cache % 16) == 0,
              "attention_tc: pointers and strides must keep 16-byte alignment");
@@ -456,22 +480,25 @@ FB_API int fb_attention_prefill_tc(const void* q, long long q_stride, int T, voi
     if (rc) return rc;
   }
   {
-    const long long dims[3] = {D, (long long)Kh * FB_PAGE, n_pages};
-    const long long strides[2] = {D, page_stride};
     const int box[3] = {64, FB_PAGE, 1};
-    int rc = make_map(&mk, k_cache, 3, dims, strides, box);
+    const long long kdims[3] = {D, (long long)Kh * FB_PAGE, n_pages}, kstrides[2] = {D, k_page};
+    int rc = make_map(&mk, k_cache, 3, kdims, kstrides, box);
     if (rc) return rc;
-    rc = make_map(&mv, v_cache, 3, dims, strides, box);
+    const long long vdims[3] = {DV, (long long)Kh * FB_PAGE, n_pages}, vstrides[2] = {DV, v_page};
+    rc = make_map(&mv, v_cache, 3, vdims, vstrides, box);
     if (rc) return rc;
   }
   FaParams p;
   p.out = (__nv_bfloat16*)out; p.out_stride = out_stride;
   p.cu_tokens = cu_tokens; p.kv_lens = kv_lens; p.page_table = page_table;
   p.max_pages = max_pages; p.n_seqs = n_seqs; p.A = A; p.Kh = Kh;
+  p.D = D; p.DV = DV; p.window = window;
   p.scale_log2 = scale * LOG2E;
   p.sink_logits = sink_logits;
-  return D == 64 ? launch<64>(mq, mk, mv, p, q_blocks, stream)
-                 : launch<128>(mq, mk, mv, p, q_blocks, stream);
+  if (D <= 64) return DV <= 64 ? launch<1, 1>(mq, mk, mv, p, q_blocks, stream)
+                               : launch<1, 2>(mq, mk, mv, p, q_blocks, stream);
+  return DV <= 64 ? launch<2, 1>(mq, mk, mv, p, q_blocks, stream)
+                  : launch<2, 2>(mq, mk, mv, p, q_blocks, stream);
 }
 
 // As fb_gemm_tc_status, for the attention kernel of this file.

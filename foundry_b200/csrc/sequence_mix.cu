@@ -452,6 +452,266 @@ __global__ void __launch_bounds__(256) scan_kernel(ScanArgs a, int tc) {
   }
 }
 
+// ------------------------------------- chunks side by side, register tiles of the state
+// The chunked passes of the linear recurrence for sizes of whole 16-byte pieces. A thread
+// owns 8 key rows x 4 columns of a head's state, so that a token's k, g and q rows are read
+// from shared memory once per 4 columns (the scan above reads them once per column: its
+// threads hold a slice of one column, which suits single tokens and few chunks). Rows go in
+// pairs through the two-wide fma. Row groups lie over the warps' lanes and the warps; their
+// shares of a token's outputs meet by shuffles and, once per tile of tokens, in shared memory.
+// PASS 1: the chunk's contribution and the product of its decays; 2: its outputs. RG: row
+// groups (8 RG >= dim). GS: one decay a head.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float x, float y) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+  const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+}
+
+template <int RG>
+struct LcShape {
+  static constexpr int THREADS = RG <= 16 ? 128 : 256;
+  static constexpr int TOKENS = RG <= 16 ? 8 : 4;              // tokens staged at a time
+  static constexpr int CG = THREADS / RG, COLS = CG * 4;       // column groups, columns a block
+  static constexpr int RW = CG < 32 ? 32 / CG : 1;             // row groups within a warp
+  static constexpr int WG = RG / RW;                           // shares that meet in shared memory
+};
+
+template <int PASS, int RG, bool GS>
+__global__ void __launch_bounds__(LcShape<RG>::THREADS) linear_chunk_kernel(ScanArgs a) {
+  using Sh = LcShape<RG>;
+  constexpr int LC_TOKENS = Sh::TOKENS, DP = RG * 8, COLS = Sh::COLS, CG = Sh::CG, RW = Sh::RW, WG = Sh::WG;
+  // a token's record: k | g (or nothing) | q (pass 2) | v | step, decay of the head
+  constexpr int AT_G = DP, AT_Q = AT_G + (GS ? 0 : DP), AT_V = AT_Q + (PASS == 2 ? DP : 0),
+                AT_S = AT_V + COLS, REC = AT_S + 4;
+  static_assert(RW == 1 || RW == 2 || RW == 4, "row groups of a warp");
+  fb_pdl_wait();
+  __shared__ __align__(16) float buf[2][LC_TOKENS * REC];
+  __shared__ float part[PASS == 2 ? LC_TOKENS * WG * COLS : 1];
+  const int seq = blockIdx.x / a.n_chunks, h = blockIdx.y;
+  const int chunk = blockIdx.x - seq * a.n_chunks;
+  int start = a.cu_tokens[seq], n = a.cu_tokens[seq + 1] - start;
+  const bool last_chunk = (chunk + 1) * a.chunk >= n;
+  start += chunk * a.chunk;
+  n = min(n - chunk * a.chunk, a.chunk);
+  if (n <= 0 || (PASS == 1 && last_chunk)) return;
+  const int tid = threadIdx.x, cg = tid % CG, rg = tid / CG;
+  const int dim = a.dim, vdim = a.vdim, col0 = blockIdx.z * COLS, j = col0 + cg * 4, row0 = rg * 8;
+  const bool col = j < vdim;  // (whole pieces of four)
+
+  // what this thread copies of every token: up to two 16-byte pieces, and one of the scalars
+  constexpr int PIECES = AT_S / 4;
+  constexpr int MINE = (PIECES + Sh::THREADS - 1) / Sh::THREADS;
+  const float* src[MINE];
+  long long ld[MINE];
+#pragma unroll
+  for (int e = 0; e < MINE; ++e) {
+    const int at = (tid + e * Sh::THREADS) * 4;
+    src[e] = nullptr; ld[e] = 0;
+    if (at < AT_V) {
+      const int which = at / DP, row = at - which * DP;  // 0: k; then g unless GS; then q
+      if (row < dim) {
+        const bool is_q = which == (GS ? 1 : 2);
+        if (which == 0) { src[e] = a.k + (long long)(h / a.rep) * dim + row; ld[e] = a.k_ld; }
+        else if (is_q) { src[e] = a.q + (long long)(h / a.rep) * dim + row; ld[e] = a.q_ld; }
+        else { src[e] = a.g + (long long)h * dim + row; ld[e] = a.g_ld; }
+      }
+    } else if (at < AT_S && col0 + at - AT_V < vdim) {
+      src[e] = a.v + (long long)h * vdim + col0 + at - AT_V; ld[e] = a.v_ld;
+    }
+    if (src[e] != nullptr) {
+      src[e] += (long long)start * ld[e];
+    } else if (at < AT_S) {  // rows and columns beyond the head's: zeros, written once
+#pragma unroll
+      for (int b = 0; b < 2; ++b)
+        for (int t = 0; t < LC_TOKENS; ++t)
+          *reinterpret_cast<float4*>(&buf[b][t * REC + at]) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  }
+  auto stage = [&](int b, int t0, int nt) {
+    for (int t = 0; t < nt; ++t)
+#pragma unroll
+      for (int e = 0; e < MINE; ++e)
+        if (src[e] != nullptr) {
+          cp_async16(&buf[b][t * REC + (tid + e * Sh::THREADS) * 4], src[e]);
+          src[e] += ld[e];
+        }
+    if (tid < nt) {
+      const long long t = start + t0 + tid;
+      if (a.beta != nullptr) cp_async4(&buf[b][tid * REC + AT_S], a.beta + t * a.beta_ld + h);
+      if (GS) cp_async4(&buf[b][tid * REC + AT_S + 1], a.g + t * a.g_ld + h);
+    }
+  };
+
+  const long long unit = ((long long)blockIdx.x * a.H + h) * dim;  // this chunk's place in wg, ws
+  float* S_chunk = a.ws + unit * vdim;
+  const float skip = (PASS == 2 && a.bonus != nullptr) ? a.bonus[h] : 0.f;
+  f32x2 s[4][4], decayed[4];  // [row pair][column]
+#pragma unroll
+  for (int p = 0; p < 4; ++p) {
+    float4 r[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int row = row0 + 2 * p + i;
+      r[i] = (PASS == 2 && col && row < dim)
+          ? __ldcg(reinterpret_cast<const float4*>(S_chunk + (long long)row * vdim + j))
+          : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    s[p][0] = pack2(r[0].x, r[1].x); s[p][1] = pack2(r[0].y, r[1].y);
+    s[p][2] = pack2(r[0].z, r[1].z); s[p][3] = pack2(r[0].w, r[1].w);
+    decayed[p] = pack2(1.f, 1.f);
+  }
+  stage(0, 0, min(LC_TOKENS, n));
+  cp_async_commit();
+  for (int c0 = 0; c0 < n; c0 += LC_TOKENS) {
+    const int b = (c0 / LC_TOKENS) & 1, nt = min(LC_TOKENS, n - c0);
+    if (c0 + LC_TOKENS < n) stage(b ^ 1, c0 + LC_TOKENS, min(LC_TOKENS, n - c0 - LC_TOKENS));
+    cp_async_commit();
+    cp_async_wait_but_one();
+    __syncthreads();
+    for (int t = 0; t < nt; ++t) {
+      const float* tok = &buf[b][t * REC];
+      float4 v = *reinterpret_cast<const float4*>(tok + AT_V + cg * 4);
+      if (a.beta != nullptr) {
+        const float u = tok[AT_S];
+        v.x *= u; v.y *= u; v.z *= u; v.w *= u;
+      }
+      const f32x2 v2[4] = {pack2(v.x, v.x), pack2(v.y, v.y), pack2(v.z, v.z), pack2(v.w, v.w)};
+      f32x2 o[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) o[c] = pack2(0.f, 0.f);
+      const f32x2 gs = GS ? pack2(tok[AT_S + 1], tok[AT_S + 1]) : pack2(0.f, 0.f);
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(tok + row0 + half * 4);
+        ulonglong2 g4, q4;
+        if (GS) g4 = make_ulonglong2(gs, gs);
+        else g4 = *reinterpret_cast<const ulonglong2*>(tok + AT_G + row0 + half * 4);
+        if (PASS == 2) q4 = *reinterpret_cast<const ulonglong2*>(tok + AT_Q + row0 + half * 4);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int p = half * 2 + i;
+          const f32x2 k = i ? k4.y : k4.x, g = i ? g4.y : g4.x;
+#pragma unroll
+          for (int c = 0; c < 4; ++c) s[p][c] = fma2(g, s[p][c], mul2(k, v2[c]));
+          if (PASS == 2) {
+            const f32x2 q = i ? q4.y : q4.x;
+#pragma unroll
+            for (int c = 0; c < 4; ++c) o[c] = fma2(q, s[p][c], o[c]);
+          } else {
+            decayed[p] = mul2(decayed[p], g);
+          }
+        }
+      }
+      if (PASS == 2) {
+        float w[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float2 f = unpack2(o[c]);
+          w[c] = f.x + f.y;
+        }
+        float* dst = part + ((t * WG + rg / RW) * COLS) + cg * 4;
+        if constexpr (RW == 4) {  // a lane ends up with one column of the warp's four row groups
+          const bool up = (rg & 2) != 0, odd = (rg & 1) != 0;
+          const float s0 = __shfl_xor_sync(0xffffffffu, up ? w[0] : w[2], 2 * CG);
+          const float s1 = __shfl_xor_sync(0xffffffffu, up ? w[1] : w[3], 2 * CG);
+          const float x0 = (up ? w[2] : w[0]) + s0, x1 = (up ? w[3] : w[1]) + s1;
+          const float s2 = __shfl_xor_sync(0xffffffffu, odd ? x0 : x1, CG);
+          dst[(up ? 2 : 0) + (odd ? 1 : 0)] = (odd ? x1 : x0) + s2;
+        } else if constexpr (RW == 2) {
+          const bool odd = (rg & 1) != 0;
+          const float s0 = __shfl_xor_sync(0xffffffffu, odd ? w[0] : w[2], CG);
+          const float s1 = __shfl_xor_sync(0xffffffffu, odd ? w[1] : w[3], CG);
+          *reinterpret_cast<float2*>(dst + (odd ? 2 : 0)) =
+              make_float2((odd ? w[2] : w[0]) + s0, (odd ? w[3] : w[1]) + s1);
+        } else {
+          *reinterpret_cast<float4*>(dst) = make_float4(w[0], w[1], w[2], w[3]);
+        }
+      }
+    }
+    __syncthreads();
+    if (PASS == 2) {
+      for (int i = tid; i < nt * COLS; i += Sh::THREADS) {
+        const int t = i / COLS, c = i - t * COLS;
+        float x = 0.f;
+#pragma unroll
+        for (int g = 0; g < WG; ++g) x += part[(t * WG + g) * COLS + c];
+        // the skip: the token's own value straight to its output
+        x = fmaf(skip, buf[b][t * REC + AT_V + c], a.out_scale * x);
+        if (col0 + c < vdim)
+          a.out[(long long)(start + c0 + t) * a.H * vdim + (long long)h * vdim + col0 + c] = x;
+      }
+      __syncthreads();  // the buffers are refilled by the next iteration
+    }
+  }
+  if (PASS == 2 && !last_chunk) return;  // the next chunk's starting state is known already
+  float* S = PASS == 1 ? S_chunk
+                       : a.state + (long long)a.slots[seq] * a.state_stride + a.s_offset +
+                             (long long)h * dim * vdim;
+#pragma unroll
+  for (int p = 0; p < 4; ++p) {
+    const float2 x = unpack2(s[p][0]), y = unpack2(s[p][1]), z = unpack2(s[p][2]), w = unpack2(s[p][3]);
+    const float2 d = unpack2(decayed[p]);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int row = row0 + 2 * p + i;
+      if (row >= dim) continue;
+      if (col)
+        *reinterpret_cast<float4*>(S + (long long)row * vdim + j) =
+            i ? make_float4(x.y, y.y, z.y, w.y) : make_float4(x.x, y.x, z.x, w.x);
+      if (PASS == 1 && j == 0) a.wg[unit + row] = i ? d.y : d.x;
+    }
+  }
+}
+
+// Whether a scan's rows and states are whole 16-byte pieces.
+bool linear_chunks_fit(const ScanArgs& a) {
+  auto whole = [](const float* p, long long stride) { return ((uintptr_t)p % 16) == 0 && stride % 4 == 0; };
+  return a.dim % 4 == 0 && a.dim <= 256 && a.vdim % 4 == 0 && whole(a.q, a.q_ld) &&
+         whole(a.k, a.k_ld) && whole(a.v, a.v_ld) && (a.g_scalar || whole(a.g, a.g_ld)) &&
+         whole(a.state + a.s_offset, a.state_stride) && whole(a.ws, 4);
+}
+
+template <int PASS, int RG>
+void launch_linear_chunks(const ScanArgs& a, int n_seqs, cudaStream_t stream) {
+  const dim3 grid(n_seqs * a.n_chunks, a.H, (a.vdim + LcShape<RG>::COLS - 1) / LcShape<RG>::COLS);
+  const dim3 block(LcShape<RG>::THREADS);
+  // (pass 1 as a launch without the dependent mark, like any long scan: see launch_scan)
+  if (PASS == 1) {
+    if (a.g_scalar) fb_launch_serial(linear_chunk_kernel<1, RG, true>, grid, block, 0, stream, a);
+    else fb_launch_serial(linear_chunk_kernel<1, RG, false>, grid, block, 0, stream, a);
+  } else {
+    if (a.g_scalar) fb_launch(linear_chunk_kernel<2, RG, true>, grid, block, 0, stream, a);
+    else fb_launch(linear_chunk_kernel<2, RG, false>, grid, block, 0, stream, a);
+  }
+}
+template <int PASS>
+void launch_linear_pass(const ScanArgs& a, int n_seqs, cudaStream_t stream) {
+  if (a.dim <= 32) launch_linear_chunks<PASS, 4>(a, n_seqs, stream);
+  else if (a.dim <= 64) launch_linear_chunks<PASS, 8>(a, n_seqs, stream);
+  else if (a.dim <= 128) launch_linear_chunks<PASS, 16>(a, n_seqs, stream);
+  else launch_linear_chunks<PASS, 32>(a, n_seqs, stream);
+}
+
 // From the chunks' contributions to their starting states, in place: one thread an element
 // of a head's state, walking the sequence's chunks; a few chunks' loads are in flight at once.
 __global__ void scan_chunk_starts_kernel(ScanArgs a) {
@@ -560,14 +820,14 @@ __global__ void head_norm_gate_kernel(const float* o, const float* __restrict__ 
 // as exp(-softplus(-z) / tau). A block takes `tokens` token rows, a thread a channel: its
 // weight row is read once for all of them. low: float32 rows of stride ld, staged in
 // shared memory; w in the stored type; bias float32.
-constexpr int LR_TOKENS = 8;
+constexpr int LR_TOKENS = 16, LR_RANK = 8;  // tokens a block; weights a thread holds at a time
 template <typename T>
 __global__ void low_rank_decay_kernel(const float* low, long long ld, const T* __restrict__ w,
                                       const float* __restrict__ bias, float inv_tau,
                                       float* __restrict__ out, int T_, int rank, int n) {
   fb_pdl_launch();
   fb_pdl_wait();
-  extern __shared__ float rows[];  // [rank][LR_TOKENS]
+  extern __shared__ __align__(16) float rows[];  // [rank][LR_TOKENS]
   const int t0 = blockIdx.x * LR_TOKENS;
   for (int i = threadIdx.x; i < rank * LR_TOKENS; i += blockDim.x) {
     const int t = i / rank, r = i - t * rank;
@@ -580,14 +840,31 @@ __global__ void low_rank_decay_kernel(const float* low, long long ld, const T* _
 #pragma unroll
   for (int t = 0; t < LR_TOKENS; ++t) z[t] = bias[c];
   const T* wr = w + (size_t)c * rank;
-  for (int r = 0; r < rank; ++r) {
-    const float v = fb_to_float<T>(wr[r]);
-    const float4* x = reinterpret_cast<const float4*>(rows + r * LR_TOKENS);
-    const float4 lo = x[0], hi = x[1];
-    z[0] = fmaf(lo.x, v, z[0]); z[1] = fmaf(lo.y, v, z[1]);
-    z[2] = fmaf(lo.z, v, z[2]); z[3] = fmaf(lo.w, v, z[3]);
-    z[4] = fmaf(hi.x, v, z[4]); z[5] = fmaf(hi.y, v, z[5]);
-    z[6] = fmaf(hi.z, v, z[6]); z[7] = fmaf(hi.w, v, z[7]);
+  const bool whole = rank % LR_RANK == 0 && ((uintptr_t)w % 16) == 0;  // rows of 16-byte pieces
+  for (int r0 = 0; r0 < rank; r0 += LR_RANK) {
+    float v[LR_RANK];
+    if (whole) {
+      __align__(16) T raw[LR_RANK];
+#pragma unroll
+      for (int i = 0; i < (int)(LR_RANK * sizeof(T) / 16); ++i)
+        reinterpret_cast<uint4*>(raw)[i] = reinterpret_cast<const uint4*>(wr + r0)[i];
+#pragma unroll
+      for (int i = 0; i < LR_RANK; ++i) v[i] = fb_to_float<T>(raw[i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < LR_RANK; ++i) v[i] = r0 + i < rank ? fb_to_float<T>(wr[r0 + i]) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < LR_RANK; ++i) {
+      if (r0 + i >= rank) break;
+      const float4* x = reinterpret_cast<const float4*>(rows + (r0 + i) * LR_TOKENS);
+#pragma unroll
+      for (int t = 0; t < LR_TOKENS; t += 4) {
+        const float4 f = x[t / 4];
+        z[t] = fmaf(f.x, v[i], z[t]); z[t + 1] = fmaf(f.y, v[i], z[t + 1]);
+        z[t + 2] = fmaf(f.z, v[i], z[t + 2]); z[t + 3] = fmaf(f.w, v[i], z[t + 3]);
+      }
+    }
   }
 #pragma unroll
   for (int t = 0; t < LR_TOKENS; ++t)
@@ -748,6 +1025,13 @@ FB_API int fb_state_scan(int mode, const float* q, long long q_ld, const float* 
   ScanArgs a{q, q_ld, k, k_ld, v, v_ld, g, g_ld, beta, beta_ld, bonus, state, state_stride,
              s_offset, out, cu_tokens, slots, H, rep, dim, vdim, g_scalar ? 1 : 0, out_scale,
              n_chunks, chunk, ws, wg};
+  if (mode == 2 && n_chunks > 1 && linear_chunks_fit(a)) {
+    launch_linear_pass<1>(a, n_seqs, stream);
+    fb_launch(scan_chunk_starts_kernel, dim3(n_seqs, H, (dim * vdim + 255) / 256), dim3(256), 0,
+              stream, a);
+    launch_linear_pass<2>(a, n_seqs, stream);
+    return fb_check_launch("state_scan");
+  }
   // a column is shared by kp lanes: eight key rows a lane where the head allows it
   // (a token's step is a chain of dependent instructions; fewer rows a lane shorten it)
   int kp = 1;

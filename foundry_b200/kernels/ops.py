@@ -77,12 +77,13 @@ _SIGNATURES = {
                              c_void_p, c_void_p, c_ll, c_ll, c_int, c_int, c_int, c_int, c_int,
                              c_float, c_void_p],
     "fb_attention_prefill_tc": [c_void_p, c_ll, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
-                                c_int, c_void_p, c_void_p, c_ll, c_ll, c_int, c_int, c_int, c_int,
-                                c_int, c_int, c_float, c_void_p, c_void_p],
+                                c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll, c_int, c_int,
+                                c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
+                                c_void_p],
     "fb_attention_tc_status": [c_void_p],
     "fb_attention_decode": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int,
                             c_void_p, c_void_p, c_ll, c_ll, c_int, c_int, c_int, c_int, c_float,
-                            c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_ll, c_int, c_void_p, c_void_p],
     "fb_gemm_rows": [c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_void_p, c_ll, c_int,
                      c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_ll, c_void_p,
@@ -1538,16 +1539,20 @@ def _tc_attention_ok(q: torch.Tensor, out: torch.Tensor) -> bool:
 
 def attention_prefill_tc(q, out, cu_tokens, kv_lens, page_table, k_cache, v_cache, num_heads,
                          num_kv_heads, head_dim, scale, q_blocks,
-                         sink_logits: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         sink_logits: Optional[torch.Tensor] = None, v_dim: Optional[int] = None,
+                         window: int = 0) -> torch.Tensor:
     """Prompt attention on tcgen05 (csrc/attention_tcgen05.cu); `q_blocks` is the
-    sum over sequences of ceil(tokens / 128)."""
-    _check_cache_views(k_cache, v_cache, num_kv_heads, head_dim, torch.bfloat16)
+    sum over sequences of ceil(tokens / 128); `v_dim`: the values' size where it is not the
+    keys'; `window`: a token sees the last `window` positions, its own included (0: all)."""
+    v_dim = head_dim if v_dim is None else v_dim
+    _check_kv_pair(k_cache, v_cache, num_kv_heads, head_dim, v_dim, torch.bfloat16)
     _call("fb_attention_prefill_tc", _dev(q, "q", torch.bfloat16, contiguous=False), _rows(q, "q"),
           q.shape[0], _dev(out, "out", torch.bfloat16, contiguous=False), _rows(out, "out"),
           _dev(cu_tokens, "cu_tokens", torch.int32), _dev(kv_lens, "kv_lens", torch.int32),
           _dev(page_table, "page_table", torch.int32), page_table.shape[1], k_cache.data_ptr(),
-          v_cache.data_ptr(), k_cache.stride(0), k_cache.stride(1), k_cache.shape[0],
-          kv_lens.numel(), q_blocks, num_heads, num_kv_heads, head_dim, float(scale),
+          v_cache.data_ptr(), k_cache.stride(0), k_cache.stride(1), v_cache.stride(0),
+          v_cache.stride(1), k_cache.shape[0], kv_lens.numel(), q_blocks, num_heads, num_kv_heads,
+          head_dim, v_dim, int(window), float(scale),
           0 if sink_logits is None else _dev(sink_logits, "sink_logits", torch.float32), _stream())
     return out
 
@@ -1576,7 +1581,7 @@ def attention_decode(q, out, cu_tokens, kv_lens, page_table, k_cache, v_cache, n
                      num_kv_heads, head_dim, scale, splits, stages: int = 3,
                      then_reads: Optional[torch.Tensor] = None,
                      cluster: Optional[int] = None,
-                     sink_logits: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sink_logits: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
     """Tensor-core attention for one token per sequence, the cache range split
     over `splits` CTAs per (sequence, kv head). `cluster` of them (by default as
     many as divide `splits`, up to 8) form a thread-block cluster and merge their
@@ -1602,7 +1607,7 @@ def attention_decode(q, out, cu_tokens, kv_lens, page_table, k_cache, v_cache, n
           _dev(cu_tokens, "cu_tokens", torch.int32), _dev(kv_lens, "kv_lens", torch.int32),
           _dev(page_table, "page_table", torch.int32), page_table.shape[1], k_cache.data_ptr(),
           v_cache.data_ptr(), k_cache.stride(0), k_cache.stride(1), n, num_heads, num_kv_heads,
-          head_dim, float(scale), splits, stages, cluster,
+          head_dim, float(scale), int(window), splits, stages, cluster,
           0 if ws_o is None else ws_o.data_ptr(), 0 if ws_ml is None else ws_ml.data_ptr(),
           0 if counters is None else counters.data_ptr(), *_prefetch_range(then_reads),
           1 if n > SKINNY_ROWS else 0,  # what follows is a tcgen05 product, not the streaming one
@@ -2005,6 +2010,41 @@ def attention_sink(ctx, q: torch.Tensor, out: torch.Tensor, page_table, k_cache,
     return out
 
 
+WINDOW_ATTENTION_TC = _os.environ.get("FOUNDRY_B200_WINDOW_ATTENTION_TC", "1") != "0"
+
+
+def attention_window(ctx, q: torch.Tensor, out: torch.Tensor, page_table, k_cache, v_cache, H: int,
+                     G: int, dim: int, vdim: int, scale: float, window: int = 0,
+                     then_reads: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Softmax attention of a step's tokens over the last `window` positions of their
+    sequences, each token's own included (0: all of them). bfloat16: prompts whose key and
+    value sizes are multiples of 8 up to 128 run on tcgen05, single tokens with one size
+    that the split-range kernel has run there; everything else on the CUDA cores."""
+    if WINDOW_ATTENTION_TC and q.dtype == torch.bfloat16 and scale > 0.0 and q.shape[0] > 0:
+        if not ctx.is_decode and dim % 8 == 0 and vdim % 8 == 0 and max(dim, vdim) <= 128 \
+                and _tc_attention_ok(q, out):
+            if ctx.cu_tokens_host is None:  # a replayed step: the bucket's bound
+                blocks = (ctx.query_blocks_bound + 1) // 2 + ctx.n_seqs
+            else:
+                cu = ctx.cu_tokens_host
+                blocks = sum((cu[i + 1] - cu[i] + 127) // 128 for i in range(ctx.n_seqs))
+            return attention_prefill_tc(q, out, ctx.cu_tokens, ctx.kv_lens, page_table, k_cache,
+                                        v_cache, H, G, dim, scale, blocks, v_dim=vdim, window=window)
+        if ctx.is_decode and dim == vdim and dim in FAST_HEAD_DIMS and H // G <= 16 \
+                and k_cache.stride() == v_cache.stride() and out.stride(0) % 2 == 0 \
+                and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0:
+            pages = (ctx.max_kv_len + PAGE - 1) // PAGE
+            if window:
+                pages = min(pages, (window + PAGE - 2) // PAGE + 1)
+            splits, stages = decode_plan(ctx.n_seqs * G, pages, dim,
+                                         getattr(ctx, "unequal_lengths", False) and not window)
+            return attention_decode(q, out, ctx.cu_tokens, ctx.kv_lens, page_table, k_cache, v_cache,
+                                    H, G, dim, scale, splits, stages, then_reads=then_reads,
+                                    window=window)
+    return attention_sink(ctx, q, out, page_table, k_cache, v_cache, H, G, dim, vdim, scale,
+                          window=window)
+
+
 def q_temp_cache_write(qkv: torch.Tensor, q_out: torch.Tensor, coef: float, every: int, positions,
                        seq_of_token, page_table, k_cache, v_cache, G: int, k_row: int, vdim: int,
                        write_cache: bool = True) -> torch.Tensor:
@@ -2387,19 +2427,22 @@ def decay_gate(x: torch.Tensor, per_head: int, bias: torch.Tensor, A: Optional[t
 SCAN_DELTA, SCAN_WKV, SCAN_LINEAR = 0, 1, 2
 SCAN_SSD = SCAN_LINEAR  # with one decay a head, a step size and a skip
 # Chunks of a prompt that a scan works side by side (not the delta rule, whose update reads
-# the state): at least this many tokens a chunk, and about this many warps in all.
+# the state): at least this many tokens a chunk (twice that in long prompts), and a bound on
+# the chunks' states, in units of 256 floats.
 SCAN_CHUNK_TOKENS = int(_os.environ.get("FOUNDRY_B200_SCAN_CHUNK_TOKENS", "64"))  # 0: one by one
-SCAN_CHUNK_WARPS = 148 * 64
+SCAN_CHUNK_UNITS = 148 * 512
 
 
 def scan_chunks(ctx, mode: int, H: int, dim: int, vdim: int):
     """(chunks a sequence, tokens a chunk) of a step's scan. A chunked scan walks every token
-    twice, so it takes at least four chunks, and enough idle warps, to be worth it."""
+    twice, so it takes at least four chunks, and room for their states, to be worth it."""
     longest, least = ctx.max_q_len, SCAN_CHUNK_TOKENS
     if mode == SCAN_DELTA or ctx.is_decode or least <= 0 or longest < 4 * least:
         return 1, 0
-    warps = max(1, ctx.n_seqs * H * ((vdim * ((dim + 7) // 8) + 31) // 32))
-    count = min((longest + least - 1) // least, SCAN_CHUNK_WARPS // warps)
+    if longest >= 16 * least:
+        least *= 2
+    units = max(1, ctx.n_seqs * H * ((vdim * dim + 255) // 256))
+    count = min((longest + least - 1) // least, SCAN_CHUNK_UNITS // units)
     if count < 4:
         return 1, 0
     chunk = ((longest + count - 1) // count + 15) // 16 * 16

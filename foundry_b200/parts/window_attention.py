@@ -112,8 +112,9 @@ class WindowAttention(Part):
                                        self.heads, self.kv_heads, self.dim, self.vdim,
                                        write_cache=cache.writes, bias=self.bias,
                                        rot_factor=self.rot_factor)
-        ops.attention_sink(ctx, q, out, table, cache.k, cache.v, self.heads, self.kv_heads, self.dim,
-                           self.vdim, self.scale, window=self.window)
+        ops.attention_window(ctx, q, out, table, cache.k, cache.v, self.heads, self.kv_heads,
+                             self.dim, self.vdim, self.scale, self.window,
+                             then_reads=self.o.weight)
         return out
 
     def forward(self, ctx, x, cache: KVView):

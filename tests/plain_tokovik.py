@@ -162,3 +162,10 @@ def forward(cfg, weights, tokens, streams=None):
             streams.append(x)
     x = rms_around_zero(x, w["final.norm"], cfg["norm"]["eps"])
     return (x @ w["head"].T) * cfg["logit_scale"]
+
+
+def greedy_generate(cfg, weights, prompt, count):
+    tokens = list(prompt)
+    for _ in range(count):
+        tokens.append(int(torch.argmax(forward(cfg, weights, tokens)[-1])))
+    return tokens[len(prompt):]
