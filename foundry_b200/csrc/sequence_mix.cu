@@ -817,7 +817,8 @@ __global__ void head_norm_gate_kernel(const float* o, const float* __restrict__ 
 
 // ------------------------------------- decays from a low-rank projection, per key channel
 // out[t, c] = sigmoid(z)^(1 / tau),  z = sum_r low[t, r] w[c, r] + bias[c]
-// as exp(-softplus(-z) / tau). A block takes `tokens` token rows, a thread a channel: its
+// as exp((min(z, 0) - log(1 + exp(-|z|))) / tau): where the sum rounds, the decay, being
+// next to one, rounds as much. A block takes `tokens` token rows, a thread a channel: its
 // weight row is read once for all of them. low: float32 rows of stride ld, staged in
 // shared memory; w in the stored type; bias float32.
 constexpr int LR_TOKENS = 16, LR_RANK = 8;  // tokens a block; weights a thread holds at a time
@@ -869,7 +870,7 @@ __global__ void low_rank_decay_kernel(const float* low, long long ld, const T* _
 #pragma unroll
   for (int t = 0; t < LR_TOKENS; ++t)
     if (t0 + t < T_)
-      out[(size_t)(t0 + t) * n + c] = expf((fminf(z[t], 0.f) - log1pf(expf(-fabsf(z[t])))) * inv_tau);
+      out[(size_t)(t0 + t) * n + c] = expf((fminf(z[t], 0.f) - logf(1.0f + expf(-fabsf(z[t])))) * inv_tau);
 }
 
 // out = act(in) rounded to the activation type; act: 0 identity, 1 tanh, 2 the square of relu

@@ -1,12 +1,7 @@
 // Grouped-query attention whose weights are sigmoids, not a softmax, over the
-// keys of the query's own chunk of the sequence; and the kernel in front of it.
+// keys of the query's own chunk of the sequence (the norms, the rotation and the
+// cache write in front of it: head_rows.cu).
 //
-//   (q | k | v rows first plus a bias vector, where given)
-//   q, k: per head  x / sqrt(mean(x^2) + eps) * w   (w [dim], the same for every head;
-//         absent: no weight), then rotated on the first `rot` elements of a head:
-//         (x_i, x_{i + rot/2}) at position p turn by the angle p * f_i, cosine and sine
-//         times `rot_factor`
-//   v:    per head  x / sqrt(mean(x^2) + eps)  where `value_norm`; cached so
 //   s_ij = (q_i . k_j) * scale + bias[head]
 //   j visible to i  iff  j <= i and floor(i / chunk) == floor(j / chunk)   (chunk 0: j <= i)
 //   o_i = out_scale * gate_i[head] * sum_j sigmoid(s_ij) v_j ,  gate = sigmoid(raw gate)  (absent: 1)
@@ -14,8 +9,7 @@
 // The weights are not normalised over the keys, so there is no running maximum
 // and no sum to divide by: a key's share does not depend on the other keys.
 // Every constant is a parameter. Positions are the tokens' own, and a chunk's
-// borders are multiples of `chunk` in them, whatever the step brings. Angles are
-// the double-precision product of the position and a double-precision frequency.
+// borders are multiples of `chunk` in them, whatever the step brings.
 //
 // This file holds the CUDA-core forms (32-bit arithmetic, any sizes): a block
 // per (token, query head) whose warps take the visible keys 32 at a time, a
@@ -44,94 +38,6 @@ __device__ __forceinline__ void sg_load8<__nv_bfloat16>(const __nv_bfloat16* p, 
     const float2 f = __bfloat1622float2(h[i]);
     v[2 * i] = f.x;
     v[2 * i + 1] = f.y;
-  }
-}
-
-// One block a token. Rows of `qkv` are [q: H x dim | k: G x dim | v: G x vdim] in
-// float32. Queries go to `q_out` in the activation type, keys and values into the
-// token's cache row. `qk_norm` 0 leaves queries and keys as they are; `interleaved`
-// 1 turns elements (2i, 2i + 1) instead of (i, i + rot / 2); G may be 0 (a mixer that
-// reads another's keys and values has queries only).
-template <typename T>
-__global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld,
-                                            const float* __restrict__ bias, T* __restrict__ q_out,
-                                            const float* __restrict__ wq,
-                                            const float* __restrict__ wk, float eps,
-                                            int qk_norm, int value_norm,
-                                            const double* __restrict__ freq, int rot,
-                                            int interleaved, float rot_factor,
-                                            const int* __restrict__ positions,
-                                            const int* __restrict__ seq_of_token,
-                                            const int* __restrict__ page_table, int max_pages,
-                                            T* __restrict__ k_cache, T* __restrict__ v_cache,
-                                            long long k_page, long long k_head, long long v_page,
-                                            long long v_head, int H, int G, int dim, int vdim,
-                                            int write_cache, int head_floats) {
-  fb_pdl_launch();
-  fb_pdl_wait();
-  extern __shared__ float sg_smem[];  // cos [rot/2] | sin [rot/2] | a head's elements per warp
-  const int t = blockIdx.x;
-  const int seq = seq_of_token[t];
-  const int pos = seq >= 0 ? positions[t] : 0;
-  const int half = rot / 2;
-  float* cs = sg_smem;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const double angle = (double)pos * freq[i];
-    cs[i] = (float)cos(angle) * rot_factor;
-    cs[half + i] = (float)sin(angle) * rot_factor;
-  }
-  __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
-  float* buf = sg_smem + rot + (size_t)warp * head_floats;
-  const float* row = qkv + (size_t)t * ld;
-  long long page = 0;
-  int r_in_page = 0;
-  const bool cached = write_cache && seq >= 0;
-  if (cached) {
-    page = page_table[(size_t)seq * max_pages + pos / FB_PAGE];
-    r_in_page = pos % FB_PAGE;
-  }
-  // a warp a head; a token's heads (queries, keys, values) are spread over blockIdx.y
-  for (int u = blockIdx.y * nwarps + warp; u < H + 2 * G; u += gridDim.y * nwarps) {
-    const bool is_q = u < H, is_k = !is_q && u < H + G;
-    const int g = is_q ? u : (is_k ? u - H : u - H - G);
-    const int n = (is_q || is_k) ? dim : vdim;
-    const float* src = is_q ? row + (size_t)g * dim
-                            : is_k ? row + (size_t)H * dim + (size_t)g * dim
-                                   : row + (size_t)(H + G) * dim + (size_t)g * vdim;
-    const float* badd = bias != nullptr ? bias + (src - row) : nullptr;
-    float ss = 0.f;
-    for (int d = lane; d < n; d += 32) {
-      const float x = __ldcg(src + d) + (badd != nullptr ? badd[d] : 0.f);
-      buf[d] = x;
-      ss = fmaf(x, x, ss);
-    }
-    ss = fb_warp_sum(ss);
-    const bool normed = (is_q || is_k) ? qk_norm != 0 : value_norm != 0;
-    const float r = normed ? 1.0f / sqrtf(ss / (float)n + eps) : 1.0f;
-    const float* w = is_q ? wq : is_k ? wk : nullptr;
-    __syncwarp();
-    for (int d = lane; d < n; d += 32) buf[d] = buf[d] * r * (w != nullptr ? w[d] : 1.0f);
-    __syncwarp();
-    if (is_q || is_k) {
-      for (int i = lane; i < half; i += 32) {
-        const int ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + half;
-        const float a = buf[ia], b = buf[ib];
-        const float c = cs[i], s = cs[half + i];
-        buf[ia] = a * c - b * s;
-        buf[ib] = b * c + a * s;
-      }
-      __syncwarp();
-    }
-    if (is_q) {
-      T* dst = q_out + ((size_t)t * H + g) * dim;
-      for (int d = lane; d < n; d += 32) dst[d] = fb_from_float<T>(buf[d]);
-    } else if (cached) {
-      T* dst = is_k ? k_cache + page * k_page + (long long)g * k_head + (long long)r_in_page * dim
-                    : v_cache + page * v_page + (long long)g * v_head + (long long)r_in_page * vdim;
-      for (int d = lane; d < n; d += 32) dst[d] = fb_from_float<T>(buf[d]);
-    }
-    __syncwarp();
   }
 }
 
@@ -436,37 +342,6 @@ __global__ void attention_sigmoid_runs_kernel(const float* partial, int runs, T*
   }
 }
 }  // namespace
-
-FB_API int fb_head_norm_rope_cache_write(const float* qkv, long long ld, const float* bias,
-                                         void* q_out, int dtype,
-                                         const float* wq, const float* wk, float eps,
-                                         int qk_norm, int value_norm, const double* freq,
-                                         int rot, int interleaved, float rot_factor,
-                                         const int* positions,
-                                         const int* seq_of_token,
-                                         const int* page_table, int max_pages, void* k_cache,
-                                         void* v_cache, long long k_page, long long k_head,
-                                         long long v_page, long long v_head, int T, int H, int G,
-                                         int dim, int vdim, int write_cache, cudaStream_t stream) {
-  FB_REQUIRE(T >= 0 && H > 0 && G >= 0 && dim > 0 && vdim > 0, "head_norm_rope_cache_write: bad sizes");
-  FB_REQUIRE(G > 0 || !write_cache, "head_norm_rope_cache_write: no keys to write");
-  FB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dim && (rot == 0 || freq != nullptr),
-             "head_norm_rope_cache_write: %d rotated elements of %d", rot, dim);
-  FB_REQUIRE(ld >= (long long)(H + G) * dim + (long long)G * vdim,
-             "head_norm_rope_cache_write: rows of %lld are too short", ld);
-  if (T == 0) return 0;
-  const int heads = H + 2 * G;
-  const int warps = heads < 8 ? heads : 8;
-  const int head_floats = dim > vdim ? dim : vdim;
-  const size_t smem = (size_t)(rot + warps * head_floats) * 4;
-  FB_REQUIRE(smem <= 48 * 1024, "head_norm_rope_cache_write: heads of %d do not fit", head_floats);
-  const int parts = T <= 256 ? (heads + warps - 1) / warps : 1;  // few tokens: more blocks
-  FB_DISPATCH_DTYPE(dtype, E, (fb_launch(head_norm_rope_cache_kernel<E>, dim3(T, parts), dim3(warps * 32),
-      smem, stream, qkv, ld, bias, (E*)q_out, wq, wk, eps, qk_norm, value_norm, freq, rot, interleaved,
-      rot_factor, positions, seq_of_token, page_table, max_pages, (E*)k_cache, (E*)v_cache, k_page, k_head, v_page,
-      v_head, H, G, dim, vdim, write_cache, head_floats)));
-  return fb_check_launch("head_norm_rope_cache_write");
-}
 
 FB_API int fb_attention_sigmoid(const void* q, long long q_stride, void* out, long long out_stride,
                                 int dtype, const int* positions, const int* seq_of_token,

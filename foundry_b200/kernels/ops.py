@@ -13,6 +13,7 @@ from typing import Optional
 
 import os as _os
 
+import numpy as np
 import torch
 
 from . import library
@@ -99,10 +100,11 @@ _SIGNATURES = {
                      c_void_p],
     "fb_softcap": [c_void_p, c_ll, c_float, c_void_p],
     "fb_head_norm_rope_cache_write": [c_void_p, c_ll, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                                      c_float, c_int, c_int, c_void_p, c_int, c_int, c_float,
+                                      c_float, c_int, c_int, c_void_p, c_int, c_int,
                                       c_void_p, c_void_p,
                                       c_void_p, c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll,
                                       c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "fb_step_angles": [c_void_p, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p],
     "fb_attention_sigmoid": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p,
                              c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll, c_void_p, c_void_p,
                              c_ll, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -163,6 +165,11 @@ _SIGNATURES = {
                       c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_ll, c_void_p, c_void_p, c_void_p,
                       c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
                       c_void_p, c_int, c_void_p],
+    "fb_linear_step_fits": [c_int, c_int, c_int],
+    "fb_linear_step": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
+                       c_void_p, c_int, c_void_p, c_ll, c_ll, c_void_p, c_ll, c_int, c_void_p,
+                       c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float,
+                       c_void_p],
     "fb_low_rank_decay": [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int,
                           c_int, c_int, c_void_p],
     "fb_head_norm_gate": [c_void_p, c_void_p, c_int, c_void_p, c_ll, c_int, c_float, c_void_p,
@@ -2223,22 +2230,45 @@ def attention_maps_rows(ctx, q: torch.Tensor, out: torch.Tensor, k: torch.Tensor
     return out
 
 
-# ------------------------------------------ attention with sigmoid weights in chunks
+# --------------------------------------- from projections to queries, keys and values
+class Rotation:
+    """A rotation's frequencies (float64), the constant on its cosines and sines and which
+    elements it pairs ("half": i with i + len(freq); "interleaved": 2i with 2i + 1).
+    `of(ctx)` is the step's table of angles, made by the first layer that asks and shared
+    with every other layer that has the same frequencies and constant."""
+
+    def __init__(self, freq, device, factor: float = 1.0, pairing: str = "half"):
+        host = np.asarray(() if freq is None else freq, dtype=np.float64)
+        _pairing_code(pairing)
+        self.factor, self.pairing, self.dims = float(factor), pairing, 2 * int(host.size)
+        self.freq = torch.from_numpy(host.copy()).to(device)
+        self.key = ("step angles", host.tobytes(), self.factor)
+
+    def of(self, ctx) -> Optional[torch.Tensor]:
+        if not self.dims:
+            return None
+        table = ctx.shared.get(self.key)
+        if table is None:
+            T = ctx.positions.numel()
+            table = torch.empty((T, self.dims), dtype=torch.float32, device=ctx.positions.device)
+            _call("fb_step_angles", _dev(ctx.positions, "positions", torch.int32),
+                  _dev(self.freq, "freq", torch.float64), self.factor, T, self.dims // 2,
+                  table.data_ptr(), _stream())
+            ctx.shared[self.key] = table
+        return table
+
+
 def head_norm_rope_cache_write(qkv: torch.Tensor, q_out: torch.Tensor,
                                wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float,
-                               value_norm: bool, freq: Optional[torch.Tensor], positions,
-                               seq_of_token, page_table, k_cache, v_cache, H: int, G: int,
-                               dim: int, vdim: int, write_cache: bool = True,
-                               qk_norm: bool = True, pairing: str = "half",
-                               bias: Optional[torch.Tensor] = None,
-                               rot_factor: float = 1.0) -> torch.Tensor:
+                               value_norm: bool, ctx, rotation: Rotation, page_table, k_cache,
+                               v_cache, H: int, G: int, dim: int, vdim: int,
+                               write_cache: bool = True, qk_norm: bool = True,
+                               bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Per-head RMS norms of queries and keys (weights [dim] shared by the heads, or
-    none; `qk_norm` False: queries and keys stay as they are), the rotation of their first
-    2 * len(freq) elements (`pairing` "half": element i with element i + len(freq);
-    "interleaved": 2i with 2i + 1; `freq` float64), the values' RMS norm without weight
+    none; `qk_norm` False: queries and keys stay as they are), the `rotation` of their first
+    elements by the angles of the tokens' positions, the values' RMS norm without weight
     where `value_norm`; queries to `q_out`, keys and values into the token's cache row.
-    `bias` (float32 [H * dim + G * (dim + vdim)]) is added to the rows first; `rot_factor`
-    multiplies the rotation's cosines and sines.
+    `bias` (float32 [H * dim + G * (dim + vdim)]) is added to the rows first.
     `qkv`: float32 rows [q | k | v]; with G = 0 rows of queries only (nothing is cached)."""
     T = qkv.shape[0]
     kp = vp = 0
@@ -2247,7 +2277,7 @@ def head_norm_rope_cache_write(qkv: torch.Tensor, q_out: torch.Tensor,
         _check_kv_pair(k_cache, v_cache, G, dim, vdim, q_out.dtype)
         kp, vp = k_cache.data_ptr(), v_cache.data_ptr()
         ks, vs = (k_cache.stride(0), k_cache.stride(1)), (v_cache.stride(0), v_cache.stride(1))
-    rot = 0 if freq is None else 2 * freq.numel()
+    angles = rotation.of(ctx)
     for name, w in (("wq", wq), ("wk", wk)):
         if w is not None and tuple(w.shape) != (dim,):
             raise KernelError(f"head_norm_rope_cache_write: {name} {tuple(w.shape)} for heads of {dim}")
@@ -2257,14 +2287,16 @@ def head_norm_rope_cache_write(qkv: torch.Tensor, q_out: torch.Tensor,
           _rows(qkv, "qkv"), 0 if bias is None else _dev(bias, "bias", torch.float32),
           _dev(q_out, "q_out"), code_of(q_out.dtype), 0 if wq is None else _dev(wq, "wq", torch.float32),
           0 if wk is None else _dev(wk, "wk", torch.float32), float(eps), 1 if qk_norm else 0,
-          1 if value_norm else 0, 0 if freq is None else _dev(freq, "freq", torch.float64), rot,
-          _pairing_code(pairing), float(rot_factor), _dev(positions, "positions", torch.int32),
-          _dev(seq_of_token, "seq_of_token", torch.int32),
+          1 if value_norm else 0, 0 if angles is None else _dev(angles, "angles", torch.float32),
+          rotation.dims, _pairing_code(rotation.pairing),
+          _dev(ctx.positions, "positions", torch.int32),
+          _dev(ctx.seq_of_token, "seq_of_token", torch.int32),
           _dev(page_table, "page_table", torch.int32), page_table.shape[1], kp, vp, *ks, *vs,
           T, H, G, dim, vdim, 1 if write_cache else 0, _stream())
     return q_out
 
 
+# ------------------------------------------ attention with sigmoid weights in chunks
 # (key, value) sizes of the tensor-core prompt kernel; a prompt step in bfloat16 of such
 # sizes takes it, every other step the CUDA-core kernel
 SIGMOID_TC_SIZES = {(32, 32), (64, 64), (128, 128), (64, 128), (128, 64), (96, 64), (32, 64),
@@ -2494,6 +2526,36 @@ def state_scan(ctx, mode: int, q, k, v, g, state: StateRows, field: str, out: to
           1 if decay_per_head else 0, float(out_scale), n_chunks, chunk,
           0 if starts is None else starts.data_ptr(), 0 if decays is None else decays.data_ptr(),
           0 if ctx.is_decode else 1, _stream())
+    return out
+
+
+LINEAR_STEP = _os.environ.get("FOUNDRY_B200_LINEAR_STEP", "1") != "0"
+
+
+def linear_step_fits(ctx, state: StateRows, field: str, dim: int, vdim: int, rank: int) -> bool:
+    """Whether `linear_step` takes this step (single tokens, sizes of whole 16-byte pieces)."""
+    return (LINEAR_STEP and ctx.is_decode and state.stride % 4 == 0
+            and (state.rows.data_ptr() + 4 * state.offset[field]) % 16 == 0
+            and bool(_fn("fb_linear_step_fits")(dim, vdim, rank)))
+
+
+def linear_step(ctx, p: torch.Tensor, at, a2: torch.Tensor, a2_bias: torch.Tensor, tau: float,
+                norm: torch.Tensor, act: str, state: StateRows, field: str, out: torch.Tensor, H: int,
+                dim: int, vdim: int, q_scale: float, eps: float, out_scale: float = 1.0) -> torch.Tensor:
+    """One token a sequence of gated linear attention between its products
+    (csrc/linear_step.cu): `low_rank_decay`, `state_scan` and `head_norm_gate` in one launch.
+    `at`: where q, k, v, gate and the decays' low-rank rows begin in a row of `p` (float32)."""
+    rank = a2.shape[1]
+    if tuple(a2.shape) != (H * dim, rank) or a2_bias.numel() != H * dim or norm.numel() != vdim \
+            or a2.dtype != out.dtype or out.shape[0] != p.shape[0] or at[4] + rank > p.shape[1]:
+        raise KernelError(f"linear_step: {tuple(a2.shape)} decays for {H} heads of {dim} x {vdim}")
+    _call("fb_linear_step", _dev(p, "p", torch.float32, contiguous=False), _rows(p, "p"), *at,
+          _dev(a2, "a2"), _dev(a2_bias, "a2_bias", torch.float32), float(tau),
+          _dev(norm, "norm", torch.float32), {"sigmoid": 0, "silu": 1}[act], state.rows.data_ptr(),
+          state.stride, state.offset[field], _dev(out, "out", contiguous=False), _rows(out, "out"),
+          code_of(out.dtype), _dev(ctx.cu_tokens, "cu_tokens", torch.int32),
+          _dev(ctx.slots, "slots", torch.int32), ctx.n_seqs, H, dim, vdim, rank, float(q_scale),
+          float(eps), float(out_scale), _stream())
     return out
 
 

@@ -261,6 +261,10 @@ class GatedLinearAttention(Part):
         n, m = H * d, H * v
         f32 = dict(dtype=torch.float32, device=p.device)
         state = ops.StateRows(cache.rows, self.fields)
+        if ops.linear_step_fits(ctx, state, "S", d, v, self.decay_rank):
+            return ops.linear_step(ctx, p, (0, n, 2 * n, 2 * n + m, 2 * n + 2 * m), self.a2,
+                                   self.decay_bias, self.tau, self.norm, self.gate, state, "S", out,
+                                   H, d, v, d ** -0.5, self.eps, out_scale)
         decay = ops.low_rank_decay(p[:, 2 * n + 2 * m:2 * n + 2 * m + self.decay_rank], self.a2,
                                    self.decay_bias, self.tau, torch.empty((T, n), **f32))
         o = torch.empty((T, m), **f32)

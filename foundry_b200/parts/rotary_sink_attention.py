@@ -60,7 +60,7 @@ class RotarySinkAttention(Part):
         self.scale, self.sink, self.own_kv, self.pairing = float(scale), bool(sink), bool(own_kv), pairing
         self.dtype, self.device = dtype, device
         self.nq, self.nk, self.nv = heads * dim, kv_heads * dim, kv_heads * vdim
-        self.freq = torch.from_numpy(freq.copy()).to(device) if freq.size else None
+        self.rotation = ops.Rotation(freq, device, pairing=pairing)
         # for the projections that rotate in their epilogue (bfloat16 steps)
         self.inv_freq = torch.from_numpy(freq.astype(np.float32)).to(device)
         self.angles_key = ("rotary angles", freq.astype(np.float32).tobytes())
@@ -114,10 +114,9 @@ class RotarySinkAttention(Part):
             return product_to_residual(ctx, attn, self.w_o)
         rows = product_f32(x, self.w_in)  # [T, q | k | v] or [T, q]
         q = torch.empty((T, self.nq), dtype=x.dtype, device=x.device)
-        ops.head_norm_rope_cache_write(rows, q, None, None, 1.0, False, self.freq, ctx.positions,
-                                       ctx.seq_of_token, table, cache.k, cache.v, H,
-                                       G if self.own_kv else 0, d, e, write_cache=writes,
-                                       qk_norm=False, pairing=self.pairing)
+        ops.head_norm_rope_cache_write(rows, q, None, None, 1.0, False, ctx, self.rotation, table,
+                                       cache.k, cache.v, H, G if self.own_kv else 0, d, e,
+                                       write_cache=writes, qk_norm=False)
         attn = torch.empty((T, H * e), dtype=x.dtype, device=x.device)
         if self._as_plain_heads(x, cache):  # a reader of another run's keys and values
             ops.attention(ctx, q, attn, table, cache.k, cache.v, H, G, d, self.scale,

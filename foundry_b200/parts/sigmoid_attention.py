@@ -22,7 +22,6 @@ from __future__ import annotations
 
 from typing import Dict, Optional
 
-import numpy as np
 import torch
 
 from ..cache.store import KVRequest, KVView
@@ -31,6 +30,7 @@ from ..weights.loader import ExpectedTensor
 from .base import Fetch, Part, register_mixer
 from .linear import Linear
 from .products import product_f32
+from .rope import banded_frequencies
 
 
 @register_mixer("chunked_sigmoid_attention")
@@ -60,7 +60,8 @@ class ChunkedSigmoidAttention(Part):
             outs.append(("g", heads))
         self.qkvg = Linear(width, outs, dtype=dtype, device=device, suffix="")
         self.o = Linear(heads * vdim, [("o", width)], dtype=dtype, device=device, suffix="")
-        self.q_norm = self.k_norm = self.bias = self.freq = None
+        self.rotation = ops.Rotation(banded_frequencies(self.rotary, self.rotary_base), device)
+        self.q_norm = self.k_norm = self.bias = None
 
     def expected_tensors(self, prefix: str) -> Dict[str, ExpectedTensor]:
         out = {**self.qkvg.expected_tensors(prefix), **self.o.expected_tensors(prefix),
@@ -77,10 +78,6 @@ class ChunkedSigmoidAttention(Part):
         self.k_norm = fetch(f"{prefix}.k.norm").to(torch.float32).contiguous()
         if self.head_bias:
             self.bias = fetch(f"{prefix}.pb").to(torch.float32).contiguous()
-        if self.rotary:
-            f = np.power(np.float64(self.rotary_base),
-                         -2.0 * np.arange(self.rotary // 2, dtype=np.float64) / self.rotary)
-            self.freq = torch.from_numpy(f).to(self.q_norm.device)
 
     def cache_request(self) -> KVRequest:
         return KVRequest(self.kv_heads, self.dim, None, self.vdim)
@@ -117,8 +114,8 @@ class ChunkedSigmoidAttention(Part):
         table = ctx.page_table(cache.group)
         q = torch.empty((T, self.nq), dtype=out.dtype, device=p.device)
         ops.head_norm_rope_cache_write(p, q, self.q_norm, self.k_norm, self.eps, self.value_norm,
-                                       self.freq, ctx.positions, ctx.seq_of_token, table, cache.k,
-                                       cache.v, self.heads, self.kv_heads, self.dim, self.vdim,
+                                       ctx, self.rotation, table, cache.k, cache.v, self.heads,
+                                       self.kv_heads, self.dim, self.vdim,
                                        write_cache=cache.writes)
         at = self.nq + self.nk + self.nv
         gate = p[:, at:at + self.heads] if self.output_gate else None

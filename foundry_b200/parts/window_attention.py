@@ -48,10 +48,10 @@ class WindowAttention(Part):
             raise ValueError(f"{2 * freq.size} rotated elements of heads of {dim}")
         self.width, self.heads, self.kv_heads, self.dim, self.vdim = width, heads, kv_heads, dim, vdim
         self.scale, self.eps, self.window = float(scale), float(eps), int(window) if window else 0
-        self.rot_factor, self.biased = float(rot_factor), bool(bias)
+        self.biased = bool(bias)
         self.dtype, self.device = dtype, device
         self.nq, self.nk, self.nv = heads * dim, kv_heads * dim, kv_heads * vdim
-        self.freq = torch.from_numpy(freq.copy()).to(device) if freq.size else None
+        self.rotation = ops.Rotation(freq, device, rot_factor)
         self.qkv = Linear(width, [("q", self.nq), ("k", self.nk), ("v", self.nv)], dtype=dtype,
                           device=device, suffix="")
         self.o = Linear(heads * vdim, [("o", width)], dtype=dtype, device=device, suffix="")
@@ -107,11 +107,10 @@ class WindowAttention(Part):
             raise ValueError("window_attention: softmax outputs take no constant")
         table = ctx.page_table(cache.group)
         q = torch.empty((p.shape[0], self.nq), dtype=out.dtype, device=p.device)
-        ops.head_norm_rope_cache_write(p, q, self.q_norm, self.k_norm, self.eps, False, self.freq,
-                                       ctx.positions, ctx.seq_of_token, table, cache.k, cache.v,
-                                       self.heads, self.kv_heads, self.dim, self.vdim,
-                                       write_cache=cache.writes, bias=self.bias,
-                                       rot_factor=self.rot_factor)
+        ops.head_norm_rope_cache_write(p, q, self.q_norm, self.k_norm, self.eps, False, ctx,
+                                       self.rotation, table, cache.k, cache.v, self.heads,
+                                       self.kv_heads, self.dim, self.vdim,
+                                       write_cache=cache.writes, bias=self.bias)
         ops.attention_window(ctx, q, out, table, cache.k, cache.v, self.heads, self.kv_heads,
                              self.dim, self.vdim, self.scale, self.window,
                              then_reads=self.o.weight)

@@ -316,6 +316,32 @@ def test_chunks_side_by_side_equal_the_scan_in_order(dims, chunk_tokens, monkeyp
         assert torch.equal(results[1][1][others], start[others])  # nobody else's state is touched
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(4, 16, 24, 5), (2, 64, 64, 16), (3, 128, 128, 33), (1, 256, 256, 64),
+                                   (2, 40, 20, 1), (5, 100, 80, 9)])
+def test_single_tokens_in_one_kernel_equal_the_three(sizes, dtype, monkeypatch):
+    """The fused single-token kernel against decays, scan and gated norm one by one, on the
+    same states (each slot's moved on by the same tokens), and counted."""
+    from foundry_b200.kernels import ops
+    H, d, e, rank = sizes
+    m = {"left": {"heads": 1, "kv_heads": 1, "dim": 8, "vdim": 8, "scale": 0.3},
+         "right": {"heads": H, "dim": d, "vdim": e, "tau": 3.0}}
+    weights = tiny.random_tensors(tiny.mixer_shapes("a", m, 64, rank), seed=rank)
+    part = mixer_part(m, 64, 1e-5, weights, dtype, rank, side="right")
+    torch.manual_seed(rank)
+    xs = [torch.randn(9, 64).to(dtype).float() for _ in range(3)]
+    results = []
+    for fused in (True, False):
+        monkeypatch.setattr(ops, "LINEAR_STEP", fused)
+        cache = new_cache(part, 256, 4, dtype)
+        got, counts = counted(lambda: run_mixer(part, cache, xs, [[4] + [1] * 5] * 3, dtype))
+        assert counts.get("linear_step", 0) == (5 if fused else 0)
+        results.append((got, cache.view(0, True).rows.cpu()))
+    for g, w in zip(*(r[0] for r in results)):
+        assert rel_error(g, w) < (1e-5 if dtype == torch.float32 else 1e-2)
+    assert rel_error(results[0][1][:3], results[1][1][:3]) < 1e-5
+
+
 # --------------------------------------------- one key that stands out, anywhere
 def crafted_attention(W, d, e, window, heads=1, kv_heads=1):
     """A window attention made so that a query that carries input 1 matches only a key that
