@@ -33,6 +33,10 @@
 // scale, so scaling after the sum over K is the same normalisation, with the one
 // rounding to bfloat16 made before the scale instead of after it.
 //
+// Two products of the same tokens with inputs and weights of their own (the output
+// projections of two mixers side by side) may share a launch: the grid's first CTAs
+// work the first, the others the second, and together they fill the SMs better.
+//
 // Larger token counts run on the tcgen05 kernel (gemm_tcgen05.cu).
 #include "common.cuh"
 
@@ -112,12 +116,26 @@ struct ResidualSink {
 template <bool ROPE> struct RopeArg { using type = NoRope; };
 template <> struct RopeArg<true> { using type = RopeWrite; };
 struct NoSink {};
+// The second product of a pair: CTAs from `first` on work it (float32 out, plain epilogue).
+struct SecondProduct {
+  const __nv_bfloat16* x;
+  long long ldx;
+  const __nv_bfloat16* w;
+  long long ldw;
+  float* out;
+  long long ldo;
+  int N, K, first;
+};
+struct NoSecond {};
+template <bool PAIR> struct PairArg { using type = NoSecond; };
+template <> struct PairArg<true> { using type = SecondProduct; };
 template <bool SINK> struct SinkArg { using type = NoSink; };
 template <> struct SinkArg<true> { using type = ResidualSink; };
 // what a kernel instance ends with
 constexpr int MODE_PLAIN = 0;  // store, or SiLU(gate) * up
 constexpr int MODE_ROPE = 1;   // rotate and write queries, keys, values
 constexpr int MODE_SINK = 2;   // add into the residual rows in front of a norm
+constexpr int MODE_PAIR = 3;   // store; the grid holds two products
 
 // NT: token tiles of 8 (1 or 2). WARPS: warps per CTA, each with a K range.
 // UNROLL: chunks whose loads are in flight together.
@@ -137,14 +155,25 @@ gemm_skinny_kernel(const __nv_bfloat16* x, long long ldx,
                    int late_trigger, int early_from,
                    const typename RopeArg<MODE == MODE_ROPE>::type rw,
                    const RowScale scale,
-                   const typename SinkArg<MODE == MODE_SINK>::type sink) {
+                   const typename SinkArg<MODE == MODE_SINK>::type sink,
+                   const typename PairArg<MODE == MODE_PAIR>::type second) {
   constexpr bool ROPE = MODE == MODE_ROPE, SINK = MODE == MODE_SINK;
   __shared__ float red[WARPS][16][8 * NT + 1];
   __shared__ float scale_part[4][16];
   extern __shared__ __align__(16) float shares[];  // [scale.count][16] when there is a row scale
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
-  const int n0 = blockIdx.x * 16;
+  int group = blockIdx.x;
+  if constexpr (MODE == MODE_PAIR) {
+    if (group >= second.first) {
+      group -= second.first;
+      x = second.x; ldx = second.ldx;
+      w = second.w; ldw = second.ldw;
+      out = second.out; ldo = second.ldo;
+      N = second.N; K = second.K;
+    }
+  }
+  const int n0 = group * 16;
   // The CTAs that are placed last let the next kernel's blocks be placed as they
   // start: no CTA of this kernel waits for room any more, and what room there is
   // (a thin last round, SMs with one CTA of two) goes to blocks that ask for their
@@ -481,7 +510,8 @@ int launch_skinny(const void* x, long long ldx, const void* w, long long ldw, vo
                   long long ldo, int out_f32, int T, int N, int K, int epilogue, const void* next,
                   long long next_bytes, int ksplit, long long plane_stride, int warps,
                   int late_trigger, const RopeWrite& rw, const RowScale& scale,
-                  const ResidualSink& sink, cudaStream_t stream) {
+                  const ResidualSink& sink, cudaStream_t stream,
+                  SecondProduct second = SecondProduct{}) {
   FB_REQUIRE(next_bytes >= 0 && next_bytes % 16 == 0 && ((uintptr_t)next % 16) == 0,
              "gemm_skinny: the prefetch range must be 16-byte aligned and a multiple of 16 bytes");
   FB_REQUIRE(T > 0 && T <= 16 && N > 0 && K > 0, "gemm_skinny: bad sizes T=%d N=%d K=%d", T, N, K);
@@ -505,12 +535,14 @@ int launch_skinny(const void* x, long long ldx, const void* w, long long ldw, vo
                                sink.ldr >= N && sink.ldxg >= N && sink.ss_stride >= T),
              "gemm_skinny: the residual sink needs its four arrays, rows of %d and shares of %d",
              N, T);
-  const int blocks = (N + 15) / 16;
+  second.first = (N + 15) / 16;
+  const int blocks = second.first + (second.w != nullptr ? (second.N + 15) / 16 : 0);
   // Warps per CTA: as many as still let every CTA of the grid be resident at
   // once (one CTA of 16 warps, two of 8 or five of 4 fit an SM). A second, thin
   // round of CTAs costs a whole round's latency: measured on the 3B decode step,
   // 192 CTAs of 16 warps (148 + 44) were 4 us a call slower than 192 of 8.
-  const int chunks = ((K + CHUNK - 1) / CHUNK + ksplit - 1) / ksplit;
+  const int longest = second.w != nullptr && second.K > K ? second.K : K;
+  const int chunks = ((longest + CHUNK - 1) / CHUNK + ksplit - 1) / ksplit;
   if (warps == 0) {
     const long long ctas = (long long)blocks * ksplit;
     warps = ctas <= 148 ? 16 : ctas <= 296 ? 8 : 4;
@@ -520,17 +552,18 @@ int launch_skinny(const void* x, long long ldx, const void* w, long long ldw, vo
   const int unroll = per >= 4 ? 4 : per >= 3 ? 3 : 2;
   // CTAs from this one on are the last half round of the grid (16 / warps CTAs fit an SM)
   const int early_from = blocks * ksplit - (16 / warps) * (sm_count() / 2);
-#define FB_SKINNY_R(NT, W, U, MODE, ROPE_ARG, SINK_ARG)                                        \
+#define FB_SKINNY_R(NT, W, U, MODE, ROPE_ARG, SINK_ARG, PAIR_ARG)                                       \
   do {                                                                                         \
   fb_launch(gemm_skinny_kernel<NT, W, U, MODE>, dim3(blocks, ksplit), dim3(W * 32),            \
             shares_bytes, stream, (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, ldw,   \
             out, ldo, out_f32, T, N, K, epilogue, next, next_bytes, plane_stride,               \
-            late_trigger, early_from, ROPE_ARG, scale, SINK_ARG); } while (0)
+            late_trigger, early_from, ROPE_ARG, scale, SINK_ARG, PAIR_ARG); } while (0)
 #define FB_SKINNY(NT, W, U)                                                      \
   do {                                                                           \
-    if (epilogue == 2) FB_SKINNY_R(NT, W, U, MODE_ROPE, rw, NoSink{});            \
-    else if (epilogue == 3) FB_SKINNY_R(NT, W, U, MODE_SINK, NoRope{}, sink);     \
-    else FB_SKINNY_R(NT, W, U, MODE_PLAIN, NoRope{}, NoSink{});                   \
+    if (epilogue == 2) FB_SKINNY_R(NT, W, U, MODE_ROPE, rw, NoSink{}, NoSecond{});            \
+    else if (epilogue == 3) FB_SKINNY_R(NT, W, U, MODE_SINK, NoRope{}, sink, NoSecond{});     \
+    else if (second.w != nullptr) FB_SKINNY_R(NT, W, U, MODE_PAIR, NoRope{}, NoSink{}, second); \
+    else FB_SKINNY_R(NT, W, U, MODE_PLAIN, NoRope{}, NoSink{}, NoSecond{});                   \
   } while (0)
 #define FB_SKINNY_U(NT, W)                                    \
   do {                                                        \
@@ -579,6 +612,22 @@ FB_API int fb_gemm_skinny(const void* x, long long ldx, const void* w, long long
                        scale_dim > 0 ? 1.0f / (float)scale_dim : 0.f, scale_eps};
   return launch_skinny(x, ldx, w, ldw, out, ldo, out_f32, T, N, K, epilogue, next, next_bytes,
                        ksplit, plane_stride, warps, 1, RopeWrite{}, scale, ResidualSink{}, stream);
+}
+
+// Two products of the same T tokens in one launch, float32 out: out1 = x1 w1^T ([T, N1]) and
+// out2 = x2 w2^T ([T, N2]).
+FB_API int fb_gemm_skinny_pair(const void* x1, long long ldx1, const void* w1, long long ldw1,
+                               float* out1, long long ldo1, int N1, int K1, const void* x2,
+                               long long ldx2, const void* w2, long long ldw2, float* out2,
+                               long long ldo2, int N2, int K2, int T, const void* next,
+                               long long next_bytes, cudaStream_t stream) {
+  FB_REQUIRE(N2 > 0 && K2 > 0 && K2 % 8 == 0 && ldx2 % 8 == 0 && ldw2 % 8 == 0 && w2 != nullptr &&
+                 ((uintptr_t)x2 % 16) == 0 && ((uintptr_t)w2 % 16) == 0,
+             "gemm_skinny_pair: the second product's sizes must keep 16-byte alignment");
+  const SecondProduct second{(const __nv_bfloat16*)x2, ldx2, (const __nv_bfloat16*)w2, ldw2, out2,
+                             ldo2, N2, K2, 0};
+  return launch_skinny(x1, ldx1, w1, ldw1, out1, ldo1, 1, T, N1, K1, 0, next, next_bytes, 1, 0, 0, 1,
+                       RopeWrite{}, RowScale{}, ResidualSink{}, stream, second);
 }
 
 // The projection in front of a norm (see the top of the file): resid [T, N]

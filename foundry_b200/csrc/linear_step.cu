@@ -87,6 +87,7 @@ __global__ void __launch_bounds__(THREADS) linear_step_kernel(const StepArgs a) 
     float z = 0.f;
     if (i < dim) {
       const TO* w = (const TO*)a.a2 + ((long long)h * dim + i) * a.rank;
+#pragma unroll 8
       for (int r = tid & 1; r < a.rank; r += 2) z = fmaf(low[r], fb_to_float<TO>(w[r]), z);
     }
     z += __shfl_xor_sync(0xffffffffu, z, 1);

@@ -62,6 +62,9 @@ _SIGNATURES = {
     "fb_rope_table": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "fb_gemm_tc_status": [c_void_p],
     "fb_gemm_tc_pair_status": [c_void_p],
+    "fb_gemm_skinny_pair": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_void_p,
+                            c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_ll,
+                            c_void_p],
     "fb_gemm_skinny": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int,
                        c_int, c_void_p, c_ll, c_int, c_ll, c_int, c_void_p, c_int, c_int, c_int,
                        c_float, c_void_p],
@@ -823,6 +826,33 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: i
           *_prefetch_range(then_reads), ksplit, M * N if ksplit > 1 else 0, warps, *scale,
           _stream(), tag=("m{} k{} n{}", M, K, N))
     return out
+
+
+def skinny_pair_fits(x1: torch.Tensor, w1: torch.Tensor, x2: torch.Tensor, w2: torch.Tensor) -> bool:
+    """Whether `gemm_skinny_pair` takes these two products."""
+    same = all(t.dtype == torch.bfloat16 for t in (x1, w1, x2, w2))
+    return (same and 0 < x1.shape[0] <= SKINNY_ROWS and x1.shape[0] == x2.shape[0]
+            and _tc_usable(x1, w1, x1) and _tc_usable(x2, w2, x2))
+
+
+def gemm_skinny_pair(x1: torch.Tensor, w1: torch.Tensor, x2: torch.Tensor, w2: torch.Tensor,
+                     then_reads: Optional[torch.Tensor] = None):
+    """(x1 w1^T, x2 w2^T) in float32 for up to 16 token rows, one launch of the
+    weight-streaming kernel for both products."""
+    M = x1.shape[0]
+    outs = []
+    for x, w in ((x1, w1), (x2, w2)):
+        if x.shape != (M, w.shape[1]):
+            raise KernelError(f"gemm_skinny_pair: x {tuple(x.shape)}, w {tuple(w.shape)}")
+        outs.append(torch.empty((M, w.shape[0]), dtype=torch.float32, device=x.device))
+    args = []
+    for x, w, out in ((x1, w1, outs[0]), (x2, w2, outs[1])):
+        args += [_dev(x, "x", torch.bfloat16, contiguous=False), _rows(x, "x"),
+                 _dev(w, "w", torch.bfloat16, contiguous=False), _rows(w, "w"), out.data_ptr(),
+                 w.shape[0], w.shape[0], w.shape[1]]
+    _call("fb_gemm_skinny_pair", *args, M, *_prefetch_range(then_reads), _stream(),
+          tag=("m{} k{}+{} n{}+{}", M, w1.shape[1], w2.shape[1], w1.shape[0], w2.shape[0]))
+    return tuple(outs)
 
 
 def gemm_skinny_residual(x: torch.Tensor, w: torch.Tensor, sink: ResidualSink,

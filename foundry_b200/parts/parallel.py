@@ -18,7 +18,7 @@ the model width before the two are added:
 
 (weights `<prefix>.<side name>.out`). The output projections are then two
 products, and the pair leaves as an `ops.NormedPair`, which the norm behind the
-mixer joins in its own pass.
+mixer joins in its own pass (a handful of tokens: both products in one launch).
 
 A side is any mixer that offers `input_weight()`, `output_weight()`,
 `inner_size` and `between(ctx, projections, cache_view, out, out_scale)`. The
@@ -37,7 +37,7 @@ from ..config.spec import PartSpec
 from ..kernels import ops
 from ..weights.loader import ExpectedTensor
 from .base import MIXERS, Fetch, Part, register_mixer
-from .products import product_f32, product_planes
+from .products import product_f32, product_pair
 
 
 @register_mixer("parallel")
@@ -121,16 +121,14 @@ class ParallelMixer(Part):
         return product_f32(both, self.w_out)
 
     def _normed_pair(self, ctx, p, inner, cache, dtype):
-        at, results = 0, []
-        then = [self.sides[1].output_weight(), getattr(ctx, "reads_after_part", None)]
-        mixed = []
+        at, mixed = 0, []
         for side, rows, n, scale in zip(self.sides, self.rows, inner, self.scales):
             out = torch.empty((p.shape[0], n), dtype=dtype, device=p.device)
             side.between(ctx, p[:, at:at + rows], self._view_for(side, cache), out, scale)
             mixed.append(out)
             at += rows
-        for side, rows, after in zip(self.sides, mixed, then):
-            results.append(product_planes(rows, side.output_weight(), then_reads=after))
+        left, right = product_pair(mixed[0], self.sides[0].output_weight(), mixed[1],
+                                   self.sides[1].output_weight(),
+                                   then_reads=getattr(ctx, "reads_after_part", None))
         eps, scale = self.out_norm
-        return ops.NormedPair(results[0], self.out_weights[0], results[1], self.out_weights[1],
-                              eps, scale)
+        return ops.NormedPair(left, self.out_weights[0], right, self.out_weights[1], eps, scale)

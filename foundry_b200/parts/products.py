@@ -31,6 +31,15 @@ def product_planes(x: torch.Tensor, w: torch.Tensor, then_reads=None):
     return matmul_nt(x, w, out_dtype=torch.float32, allow_planes=True, then_reads=then_reads)
 
 
+def product_pair(x1: torch.Tensor, w1: torch.Tensor, x2: torch.Tensor, w2: torch.Tensor,
+                 then_reads=None):
+    """(x1 w1^T, x2 w2^T), each as `product_planes` gives it; a handful of tokens takes one
+    launch for both."""
+    if min(x1.shape[1], x2.shape[1]) >= SMALL_K and ops.skinny_pair_fits(x1, w1, x2, w2):
+        return ops.gemm_skinny_pair(x1, w1, x2, w2, then_reads)
+    return product_planes(x1, w1, then_reads=w2), product_planes(x2, w2, then_reads=then_reads)
+
+
 def product_to_residual(ctx, x: torch.Tensor, w: torch.Tensor):
     """A part's last product, whose result joins the residual: float32 as
     `product_f32` gives it, or, where the block offers the next norm's sink

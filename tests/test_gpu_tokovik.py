@@ -252,6 +252,20 @@ def test_norms_behind_parts(width, planes):
             assert rel_error(picked.cpu(), want[[3, 0]]) < 2e-6
 
 
+@pytest.mark.parametrize("sizes", [(64, 256, 128, 128), (2048, 512, 512, 1024), (96, 40, 328, 24), (520, 100, 64, 7)])
+def test_two_products_of_a_handful_of_tokens_in_one_launch(sizes):
+    from foundry_b200.parts.products import product_pair
+    k1, n1, k2, n2 = sizes
+    gen = torch.Generator().manual_seed(k1)
+    draw = lambda *s: torch.randn(s, generator=gen).to(torch.bfloat16)
+    for T in (1, 3, 8, 11, 16, 40):
+        x1, w1, x2, w2 = draw(T, k1), draw(n1, k1), draw(T, k2), draw(n2, k2)
+        got, counts = counted(lambda: product_pair(*(t.to(DEV) for t in (x1, w1, x2, w2))))
+        assert counts.get("gemm_skinny_pair", 0) == (1 if T <= 16 else 0)
+        for g, x, w in zip(got, (x1, x2), (w1, w2)):
+            assert rel_error(joined(g).cpu(), x.double() @ w.double().T) < 1e-5
+
+
 @pytest.mark.parametrize("rank, channels, tau", [(1, 5, 1.0), (16, 200, 16.0), (40, 300, 3.0), (27, 64, 0.5)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_decays_from_a_low_rank_projection(rank, channels, tau, dtype):
