@@ -712,36 +712,54 @@ void launch_linear_pass(const ScanArgs& a, int n_seqs, cudaStream_t stream) {
   else launch_linear_chunks<PASS, 32>(a, n_seqs, stream);
 }
 
-// From the chunks' contributions to their starting states, in place: one thread an element
-// of a head's state, walking the sequence's chunks; a few chunks' loads are in flight at once.
-__global__ void scan_chunk_starts_kernel(ScanArgs a) {
+// From the chunks' contributions to their starting states, in place: one thread V neighbouring
+// columns of a row of a head's state, walking the sequence's chunks; several chunks' loads are
+// in flight at once.
+template <int V>
+__global__ void __launch_bounds__(128) scan_chunk_starts_kernel(ScanArgs a) {
   fb_pdl_wait();
   const int seq = blockIdx.x, h = blockIdx.y;
   const int n = a.cu_tokens[seq + 1] - a.cu_tokens[seq];
   const int elements = a.dim * a.vdim;
-  const int i = blockIdx.z * blockDim.x + threadIdx.x;
+  const int i = (blockIdx.z * blockDim.x + threadIdx.x) * V;
   if (n <= 0 || i >= elements) return;
   const int chunks = (n + a.chunk - 1) / a.chunk;
-  float s = __ldcg(a.state + (long long)a.slots[seq] * a.state_stride + a.s_offset +
-                   (long long)h * elements + i);
+  auto load = [](const float* p, float (&v)[V]) {
+    if constexpr (V == 4) {
+      const float4 f = __ldcg(reinterpret_cast<const float4*>(p));
+      v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    } else {
+      v[0] = __ldcg(p);
+    }
+  };
+  float s[V];
+  load(a.state + (long long)a.slots[seq] * a.state_stride + a.s_offset + (long long)h * elements + i, s);
   const long long first = ((long long)seq * a.n_chunks * a.H + h) * a.dim;
   const long long step = (long long)a.H * a.dim;
   float* ws = a.ws + first * a.vdim + i;
   const float* wg = a.wg + first + i / a.vdim;
   constexpr int AHEAD = 8;
   for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-    float d[AHEAD], g[AHEAD];
+    float d[AHEAD][V], g[AHEAD];
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u) {
-      const bool there = c0 + u + 1 < chunks;  // (the last chunk has no contribution)
-      d[u] = there ? __ldcg(ws + (c0 + u) * step * a.vdim) : 0.f;
-      g[u] = there ? __ldcg(wg + (c0 + u) * step) : 0.f;
+      if (c0 + u + 1 < chunks) {  // (the last chunk has no contribution)
+        load(ws + (c0 + u) * step * a.vdim, d[u]);
+        g[u] = __ldcg(wg + (c0 + u) * step);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) d[u][e] = 0.f;
+        g[u] = 0.f;
+      }
     }
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u) {
       if (c0 + u >= chunks) break;
-      ws[(c0 + u) * step * a.vdim] = s;
-      s = fmaf(g[u], s, d[u]);
+      float* at = ws + (c0 + u) * step * a.vdim;
+      if constexpr (V == 4) *reinterpret_cast<float4*>(at) = make_float4(s[0], s[1], s[2], s[3]);
+      else *at = s[0];
+#pragma unroll
+      for (int e = 0; e < V; ++e) s[e] = fmaf(g[u], s[e], d[u][e]);
     }
   }
 }
@@ -1028,7 +1046,7 @@ FB_API int fb_state_scan(int mode, const float* q, long long q_ld, const float* 
              n_chunks, chunk, ws, wg};
   if (mode == 2 && n_chunks > 1 && linear_chunks_fit(a)) {
     launch_linear_pass<1>(a, n_seqs, stream);
-    fb_launch(scan_chunk_starts_kernel, dim3(n_seqs, H, (dim * vdim + 255) / 256), dim3(256), 0,
+    fb_launch(scan_chunk_starts_kernel<4>, dim3(n_seqs, H, (dim * vdim / 4 + 127) / 128), dim3(128), 0,
               stream, a);
     launch_linear_pass<2>(a, n_seqs, stream);
     return fb_check_launch("state_scan");
@@ -1095,7 +1113,7 @@ FB_API int fb_state_scan(int mode, const float* q, long long q_ld, const float* 
       }
     }
     if (as_mode == mode) break;
-    fb_launch(scan_chunk_starts_kernel, dim3(n_seqs, H, (dim * vdim + 255) / 256), dim3(256), 0,
+    fb_launch(scan_chunk_starts_kernel<1>, dim3(n_seqs, H, (dim * vdim + 127) / 128), dim3(128), 0,
               stream, a);
   }
 #undef FB_SCAN
