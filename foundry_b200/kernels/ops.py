@@ -2489,8 +2489,8 @@ def decay_gate(x: torch.Tensor, per_head: int, bias: torch.Tensor, A: Optional[t
 SCAN_DELTA, SCAN_WKV, SCAN_LINEAR = 0, 1, 2
 SCAN_SSD = SCAN_LINEAR  # with one decay a head, a step size and a skip
 # Chunks of a prompt that a scan works side by side (not the delta rule, whose update reads
-# the state): at least this many tokens a chunk (twice that in long prompts), and a bound on
-# the chunks' states, in units of 256 floats.
+# the state): at least this many tokens a chunk, and a bound on the chunks' states, in units
+# of 256 floats.
 SCAN_CHUNK_TOKENS = int(_os.environ.get("FOUNDRY_B200_SCAN_CHUNK_TOKENS", "64"))  # 0: one by one
 SCAN_CHUNK_UNITS = 148 * 512
 
@@ -2501,8 +2501,6 @@ def scan_chunks(ctx, mode: int, H: int, dim: int, vdim: int):
     longest, least = ctx.max_q_len, SCAN_CHUNK_TOKENS
     if mode == SCAN_DELTA or ctx.is_decode or least <= 0 or longest < 4 * least:
         return 1, 0
-    if longest >= 16 * least:
-        least *= 2
     units = max(1, ctx.n_seqs * H * ((vdim * dim + 255) // 256))
     count = min((longest + least - 1) // least, SCAN_CHUNK_UNITS // units)
     if count < 4:

@@ -413,7 +413,7 @@ def places(window):
     front of it, the first token of the sequence, the query itself and its neighbour,
     for queries at the first tokens, on both sides of page borders and far out."""
     out = []
-    for q in (5, 63, 64, 128, 129, 200, 700):
+    for q in (5, 63, 64, 129, 200, 700):
         lo = max(0, q - window + 1) if window else 0
         seen = {lo, q, max(lo, q - 1), min(q, lo + 1)}
         hidden = {lo - 1, 0, lo - 64} if lo > 0 else set()
@@ -423,7 +423,7 @@ def places(window):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("window", [1, 2, 64, 65, 100, 640, None])
+@pytest.mark.parametrize("window", [1, 64, 65, 640, None])
 @pytest.mark.parametrize("sizes", [(8, 8, 1, 1), (64, 64, 2, 1), (32, 128, 2, 2), (128, 128, 4, 1),
                                    (80, 56, 20, 1)])
 def test_one_key_that_stands_out_on_both_sides_of_every_edge(sizes, window, dtype):
