@@ -7,6 +7,7 @@ and a recurrence side by side), or nothing. Cache entries with the same key-valu
 and policy form a group with storage and a page pool of its own:
 
     storage[entry, page, 0 = keys / 1 = values, kv head, row in page, head_dim]
+    storage[entry, page, kv head, rows of a page | a float32 a row]    (`row_scales`)
 
 so one (page, head) block of `PAGE x head_dim` elements is contiguous. The
 reference holds `[batch, kv heads, max_cache_len, head_dim]` per layer, all
@@ -34,6 +35,9 @@ class KVRequest:
     # None: values have the keys' size; 0: no value rows are stored (a mixer whose
     # values are a part of its key rows; both views of the entry are the key rows)
     v_head_dim: Optional[int] = None
+    # with v_head_dim 0: one float32 a row, behind the rows of a (page, head) block (the
+    # factor of a row's scores, for rows that are read as keys and as values)
+    row_scales: bool = False
 
 
 @dataclass(frozen=True)
@@ -61,7 +65,14 @@ class KVGroup:
         self.pages = GroupPages(page_count, request.window)
         self.v_storage = None
         self.keys_only = request.v_head_dim == 0
-        if self.keys_only:
+        if request.row_scales:
+            if not self.keys_only:
+                raise ValueError("row scales belong to rows that are keys and values at once")
+            tail = 4 // torch.empty((), dtype=dtype).element_size()  # elements a float32 takes
+            self.storage = torch.zeros(
+                (len(entries), page_count, request.kv_heads, PAGE * (request.head_dim + tail)),
+                dtype=dtype, device=device)
+        elif self.keys_only:
             self.storage = torch.zeros(
                 (len(entries), page_count, request.kv_heads, PAGE, request.head_dim),
                 dtype=dtype, device=device)
@@ -77,6 +88,7 @@ class KVGroup:
                 (len(entries), page_count, request.kv_heads, PAGE, request.v_head_dim),
                 dtype=dtype, device=device)
         self._views: Dict[int, Tuple[torch.Tensor, torch.Tensor]] = {}
+        self._scales: Dict[int, torch.Tensor] = {}
 
     @property
     def ring_pages(self) -> int:
@@ -90,7 +102,10 @@ class KVGroup:
         views = self._views.get(entry)
         if views is None:  # the views never change: made once per entry
             block = self.storage[self.index_of[entry]]
-            if self.keys_only:
+            if self.request.row_scales:
+                rows = block[..., :PAGE * self.request.head_dim].unflatten(-1, (PAGE, -1))
+                views = self._views[entry] = (rows, rows)
+            elif self.keys_only:
                 views = self._views[entry] = (block, block)
             elif self.v_storage is None:
                 views = self._views[entry] = (block[:, 0], block[:, 1])
@@ -98,10 +113,19 @@ class KVGroup:
                 views = self._views[entry] = (block, self.v_storage[self.index_of[entry]])
         return views
 
+    def row_scales(self, entry: int) -> torch.Tensor:
+        """float32 [pages, kv heads, PAGE]: the numbers beside an entry's rows."""
+        view = self._scales.get(entry)
+        if view is None:
+            view = self._scales[entry] = self.storage[self.index_of[entry]].view(
+                torch.float32)[..., -PAGE:]
+        return view
+
     def bytes_per_token(self) -> int:
         r = self.request
         v = r.head_dim if r.v_head_dim is None else r.v_head_dim
-        return len(self.entries) * r.kv_heads * (r.head_dim + v) * self.storage.element_size()
+        row = (r.head_dim + v) * self.storage.element_size() + (4 if r.row_scales else 0)
+        return len(self.entries) * r.kv_heads * row
 
 
 @dataclass
@@ -118,6 +142,10 @@ class KVView:
     @property
     def v(self) -> torch.Tensor:
         return self.group.kv(self.entry)[1]
+
+    @property
+    def row_scales(self) -> torch.Tensor:
+        return self.group.row_scales(self.entry)
 
 
 @dataclass

@@ -84,6 +84,9 @@ class ModelSpec:
     junctions: Tuple[PartSpec, ...] = ()
     junction_prefixes: Tuple[str, ...] = ()  # tensor-name prefix of each junction
     logit_softcap: Optional[float] = None  # c: logits <- c * tanh(logits / c)
+    # copies of the stream that the layers' block keeps and mixes; 0: one plain residual.
+    # The final norm reads their sum.
+    streams: int = 0
 
     def cache_entry_count(self) -> int:
         return 1 + max((e.cache for e in self.schedule), default=-1)

@@ -372,6 +372,41 @@ FB_API int fb_silu_mul(const void* gate_up, int in_dtype, void* out, int out_dty
   return fb_check_launch("silu_mul");
 }
 
+// ------------------------------------------------- clamped gated activation
+// Rows of 2I products, column 2i gate i and column 2i+1 up i; `bias` (float32 [2I], the same
+// order) or null joins them first:
+//   out = min(g, limit) * sigmoid(alpha min(g, limit)) * (clamp(u, -limit, limit) + shift)
+template <typename TI, typename TO>
+__global__ void glu_clamped_kernel(const TI* gate_up, const float* __restrict__ bias,
+                                   TO* __restrict__ out, int I, size_t total, float limit,
+                                   float alpha, float shift) {
+  fb_pdl_wait();
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
+       idx += (size_t)gridDim.x * blockDim.x) {
+    const int i = (int)(idx % I);
+    float g = fb_load_coherent<TI>(gate_up + 2 * idx), u = fb_load_coherent<TI>(gate_up + 2 * idx + 1);
+    if (bias != nullptr) { g += bias[2 * i]; u += bias[2 * i + 1]; }
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    out[idx] = fb_from_float<TO>(g * (1.0f / (1.0f + expf(-alpha * g))) * (u + shift));
+  }
+}
+
+FB_API int fb_glu_clamped(const void* gate_up, int in_dtype, const float* bias, void* out,
+                          int out_dtype, int T, int I, float limit, float alpha, float shift,
+                          cudaStream_t stream) {
+  FB_REQUIRE(T >= 0 && I > 0 && limit > 0.f, "glu_clamped: bad sizes T=%d I=%d limit=%f", T, I,
+             (double)limit);
+  const size_t total = (size_t)T * I;
+  if (total == 0) return 0;
+  const size_t want = (total + 255) / 256;
+  const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+  FB_DISPATCH_DTYPE(in_dtype, TI, FB_DISPATCH_DTYPE(out_dtype, TO, (
+      fb_launch(glu_clamped_kernel<TI, TO>, dim3(blocks), dim3(256), 0, stream,
+                (const TI*)gate_up, bias, (TO*)out, I, total, limit, alpha, shift))));
+  return fb_check_launch("glu_clamped");
+}
+
 // ---------------------------------------------------------------- row gather
 // dst[r,:] = src[rows[r],:]; a negative row index gives a zero row.
 template <typename T>

@@ -8,6 +8,10 @@
 //         cosine and sine times a constant
 //   v:    per head  x / sqrt(mean(x^2) + eps)  where `value_norm`; cached so
 //
+// With `key_scales` keys and values are one row: x is cached as it is and 1 / sqrt(mean(x^2) +
+// eps) beside it, as the factor of that row's scores (the key norm's weight then belongs to
+// the queries' weight); such keys are not rotated, and rows are [q | k | anything].
+//
 // The angles of a step are the same for all of its layers that share the frequencies, so
 // they come from a table that one small kernel makes per step: the angle is the
 // double-precision product of the position and a double-precision frequency, its cosine
@@ -51,7 +55,8 @@ __global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld,
                                             T* __restrict__ k_cache, T* __restrict__ v_cache,
                                             long long k_page, long long k_head, long long v_page,
                                             long long v_head, int H, int G, int dim, int vdim,
-                                            int write_cache, int head_floats) {
+                                            int write_cache, int head_floats, float* key_scales,
+                                            long long s_page, long long s_head) {
   fb_pdl_launch();
   fb_pdl_wait();
   extern __shared__ float sg_smem[];  // cos [rot/2] | sin [rot/2] | a head's elements per warp
@@ -73,7 +78,8 @@ __global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld,
     r_in_page = pos % FB_PAGE;
   }
   // a warp a head; a token's heads (queries, keys, values) are spread over blockIdx.y
-  for (int u = blockIdx.y * nwarps + warp; u < H + 2 * G; u += gridDim.y * nwarps) {
+  const int units = H + (key_scales != nullptr ? G : 2 * G);
+  for (int u = blockIdx.y * nwarps + warp; u < units; u += gridDim.y * nwarps) {
     const bool is_q = u < H, is_k = !is_q && u < H + G;
     const int g = is_q ? u : (is_k ? u - H : u - H - G);
     const int n = (is_q || is_k) ? dim : vdim;
@@ -89,8 +95,12 @@ __global__ void head_norm_rope_cache_kernel(const float* qkv, long long ld,
     }
     ss = fb_warp_sum(ss);
     const bool normed = (is_q || is_k) ? qk_norm != 0 : value_norm != 0;
-    const float r = normed ? 1.0f / sqrtf(ss / (float)n + eps) : 1.0f;
+    float r = normed ? 1.0f / sqrtf(ss / (float)n + eps) : 1.0f;
     const float* w = is_q ? wq : is_k ? wk : nullptr;
+    if (is_k && key_scales != nullptr) {  // the row as it is, its factor beside it
+      if (cached && lane == 0) key_scales[page * s_page + (long long)g * s_head + r_in_page] = r;
+      r = 1.0f;
+    }
     __syncwarp();
     for (int d = lane; d < n; d += 32) buf[d] = buf[d] * r * (w != nullptr ? w[d] : 1.0f);
     __syncwarp();
@@ -146,10 +156,12 @@ head_rows_vec_kernel(const float* qkv, long long ld, const float* __restrict__ b
                      const int* __restrict__ page_table, int max_pages, T* __restrict__ k_cache,
                      T* __restrict__ v_cache, long long k_page, long long k_head,
                      long long v_page, long long v_head, int H, int G, int dim, int vdim,
-                     int write_cache, int n_tokens) {
+                     int write_cache, int n_tokens, float* key_scales, long long s_page,
+                     long long s_head) {
   fb_pdl_launch();
   fb_pdl_wait();
-  const int units = H + 2 * G;  // heads of a token: queries, keys, values
+  // heads of a token: queries, keys, values
+  const int units = H + (key_scales != nullptr ? G : 2 * G);
   const long long at = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / LPH;
   const int lane = threadIdx.x % LPH;
   if (at - (threadIdx.x % 32) / LPH >= (long long)n_tokens * units) return;  // (a whole warp)
@@ -177,8 +189,9 @@ head_rows_vec_kernel(const float* qkv, long long ld, const float* __restrict__ b
   float ss = x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3];
 #pragma unroll
   for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if (normed) {
-    const float r = 1.0f / sqrtf(ss / (float)n + eps);
+  const bool as_is = key_scales != nullptr && !is_q;
+  const float r = 1.0f / sqrtf(ss / (float)n + eps);
+  if (normed && !as_is) {
     const float* w = is_q ? wq : is_v ? nullptr : wk;
     float wv[4] = {1.f, 1.f, 1.f, 1.f};
     if (w != nullptr && in) load4(w + d, wv);
@@ -222,9 +235,10 @@ head_rows_vec_kernel(const float* qkv, long long ld, const float* __restrict__ b
   if (!write_cache || seq < 0) return;
   const int pos = positions[t];
   const long long page = page_table[(size_t)seq * max_pages + pos / FB_PAGE];
-  const int r = pos % FB_PAGE;
-  store4<T>(is_v ? v_cache + page * v_page + (long long)g * v_head + (long long)r * vdim + d
-                 : k_cache + page * k_page + (long long)g * k_head + (long long)r * dim + d, x);
+  const int r_in_page = pos % FB_PAGE;
+  if (as_is && lane == 0) key_scales[page * s_page + (long long)g * s_head + r_in_page] = r;
+  store4<T>(is_v ? v_cache + page * v_page + (long long)g * v_head + (long long)r_in_page * vdim + d
+                 : k_cache + page * k_page + (long long)g * k_head + (long long)r_in_page * dim + d, x);
 }
 }  // namespace
 
@@ -248,15 +262,18 @@ FB_API int fb_head_norm_rope_cache_write(const float* qkv, long long ld, const f
                                          const int* page_table, int max_pages, void* k_cache,
                                          void* v_cache, long long k_page, long long k_head,
                                          long long v_page, long long v_head, int T, int H, int G,
-                                         int dim, int vdim, int write_cache, cudaStream_t stream) {
+                                         int dim, int vdim, int write_cache, float* key_scales,
+                                         long long s_page, long long s_head, cudaStream_t stream) {
   FB_REQUIRE(T >= 0 && H > 0 && G >= 0 && dim > 0 && vdim > 0, "head_norm_rope_cache_write: bad sizes");
   FB_REQUIRE(G > 0 || !write_cache, "head_norm_rope_cache_write: no keys to write");
   FB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dim && (rot == 0 || angles != nullptr),
              "head_norm_rope_cache_write: %d rotated elements of %d", rot, dim);
-  FB_REQUIRE(ld >= (long long)(H + G) * dim + (long long)G * vdim,
+  FB_REQUIRE(key_scales == nullptr || (G > 0 && qk_norm && rot == 0),
+             "head_norm_rope_cache_write: keys with a factor beside them are not rotated");
+  FB_REQUIRE(ld >= (long long)(H + G) * dim + (key_scales != nullptr ? 0 : (long long)G * vdim),
              "head_norm_rope_cache_write: rows of %lld are too short", ld);
   if (T == 0) return 0;
-  const int heads = H + 2 * G;
+  const int heads = H + (key_scales != nullptr ? G : 2 * G);
   auto whole = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
   const int longest = G > 0 && vdim > dim ? vdim : dim;
   if (dim % 4 == 0 && vdim % 4 == 0 && longest <= 128 && rot % (interleaved ? 4 : 8) == 0 &&
@@ -267,7 +284,8 @@ FB_API int fb_head_norm_rope_cache_write(const float* qkv, long long ld, const f
   fb_launch(head_rows_vec_kernel<E, LPH>, dim3((unsigned)(((long long)T * heads * LPH + 127) / 128)), \
             dim3(128), 0, stream, qkv, ld, bias, (E*)q_out, wq, wk, eps, qk_norm, value_norm, angles, \
             rot, interleaved, positions, seq_of_token, page_table, max_pages, (E*)k_cache,            \
-            (E*)v_cache, k_page, k_head, v_page, v_head, H, G, dim, vdim, write_cache, T)
+            (E*)v_cache, k_page, k_head, v_page, v_head, H, G, dim, vdim, write_cache, T, key_scales,    \
+            s_page, s_head)
     FB_DISPATCH_DTYPE(dtype, E, {
       if (longest <= 16) FB_HEAD_ROWS(E, 4);
       else if (longest <= 32) FB_HEAD_ROWS(E, 8);
@@ -285,6 +303,6 @@ FB_API int fb_head_norm_rope_cache_write(const float* qkv, long long ld, const f
   FB_DISPATCH_DTYPE(dtype, E, (fb_launch(head_norm_rope_cache_kernel<E>, dim3(T, parts), dim3(warps * 32),
       smem, stream, qkv, ld, bias, (E*)q_out, wq, wk, eps, qk_norm, value_norm, angles, rot, interleaved,
       positions, seq_of_token, page_table, max_pages, (E*)k_cache, (E*)v_cache, k_page, k_head, v_page,
-      v_head, H, G, dim, vdim, write_cache, head_floats)));
+      v_head, H, G, dim, vdim, write_cache, head_floats, key_scales, s_page, s_head)));
   return fb_check_launch("head_norm_rope_cache_write");
 }

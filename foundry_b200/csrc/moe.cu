@@ -1,12 +1,16 @@
 // A feed-forward of routed experts.
 //
-//   z = W_router h (+ b) (32-bit). Two scoring rules (`score`):
+//   z = W_router h (+ b) (32-bit). Three scoring rules (`score`):
 //   0: the `top` experts of largest z are chosen (the lower index among equals);
 //      their weights are the softmax over the chosen z only
 //   1: s = sigmoid(z); the experts form `groups` equal groups of neighbours, a group's
 //      score is the sum of its two largest s, only experts of the `keep` best groups can
 //      be chosen (groups 1: all); the `top` largest s are chosen and weighted by s itself
+//   2: as 1 with s = softmax(z) over all of the router's outputs
+//   (`group_best` 1: a group's score is its largest s alone)
 //   y = sum_c weight_c * expert_c(h)
+//   The router may have more outputs than there are experts with matrices: the last ones
+//   are identity experts, whose output is h itself.
 //   expert:  g = min(W_gate h, limit),  u = clamp(W_up h, -limit, limit)
 //            a = g * sigmoid(alpha g) * (u + shift);  out = W_down a
 //   (limit = infinity, alpha = 1, shift = 0: silu(g) * u)
@@ -28,8 +32,8 @@ __device__ __forceinline__ void route_token(const float* z, long long ld,
                                             int* __restrict__ chosen, float* __restrict__ weights,
                                             int score, int groups, int keep,
                                             const float* __restrict__ correction, int normalise,
-                                            float sum_floor, float weight_scale, int t, int lane,
-                                            float* s_all, float* s_group, float* s_plain) {
+                                            float sum_floor, float weight_scale, int group_best,
+                                            int t, int lane, float* s_all, float* s_group, float* s_plain) {
   // each lane keeps the experts lane, lane + 32, ... (up to 8 of them).
   // v[] is what the choice goes by (the score, plus `correction` where given); the
   // weights come from the scores themselves (s_plain).
@@ -37,18 +41,37 @@ __device__ __forceinline__ void route_token(const float* z, long long ld,
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
     const int e = lane + 32 * i;
-    v[i] = -INFINITY;
+    v[i] = e < E ? __ldcg(z + (size_t)t * ld + e) + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
+  }
+  if (score == 2) {  // softmax over all outputs
+    float top_z = v[0], total = 0.f;
+#pragma unroll
+    for (int i = 1; i < 8; ++i) top_z = fmaxf(top_z, v[i]);
+    top_z = fb_warp_max(top_z);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      v[i] = expf(v[i] - top_z);  // (0 beyond the last output)
+      total += v[i];
+    }
+    total = fb_warp_sum(total);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = v[i] / total;
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int e = lane + 32 * i;
     if (e < E) {
-      const float x = __ldcg(z + (size_t)t * ld + e) + (bias != nullptr ? bias[e] : 0.f);
-      const float sc = score == 1 ? 1.0f / (1.0f + expf(-x)) : x;
+      const float sc = score == 1 ? 1.0f / (1.0f + expf(-v[i])) : v[i];
       s_plain[e] = sc;
       v[i] = correction != nullptr ? sc + correction[e] : sc;
+    } else {
+      v[i] = -INFINITY;
     }
   }
   __syncwarp();
-  if (score == 1 && groups > 1) {
-    // a group's score: the sum of its two largest (a group of one: that one); the `keep`
-    // best groups stay, the lower index among equals
+  if (score != 0 && groups > 1) {
+    // a group's score: the sum of its two largest (a group of one: that one), or with
+    // `group_best` 1 its largest; the `keep` best groups stay, the lower index among equals
     const int per = E / groups;
 #pragma unroll
     for (int i = 0; i < 8; ++i)
@@ -60,7 +83,7 @@ __device__ __forceinline__ void route_token(const float* z, long long ld,
         const float x = s_all[g * per + k];
         if (x > a) { b = a; a = x; } else if (x > b) { b = x; }
       }
-      s_group[g] = per > 1 ? a + b : a;
+      s_group[g] = per > 1 && group_best == 2 ? a + b : a;
     }
     __syncwarp();
     for (int c = 0; c < keep; ++c) {
@@ -100,7 +123,7 @@ __device__ __forceinline__ void route_token(const float* z, long long ld,
     }
     if (c == 0) first = best;  // values are chosen in falling order: the first is the largest
     if (at >= E) at = 0;  // only when every value left is NaN: any expert, never a wild index
-    const float e = score == 1 ? s_plain[at] : expf(best - first);
+    const float e = score != 0 ? s_plain[at] : expf(best - first);
     sum += e;
     if (lane == c) mine = e;
     if (lane == 0) chosen[(size_t)t * top + c] = at;
@@ -108,11 +131,11 @@ __device__ __forceinline__ void route_token(const float* z, long long ld,
     for (int i = 0; i < 8; ++i)
       if (at == lane + 32 * i) v[i] = -INFINITY;
   }
-  // sigmoid scores: the chosen scores themselves, or (normalise) their shares of their sum
+  // scores of their own: the chosen scores themselves, or (normalise) their shares of their sum
   // plus `sum_floor`; both times `weight_scale`. Softmax over the chosen: mine / sum.
   if (lane < top)
     weights[(size_t)t * top + lane] =
-        score == 1 ? (normalise ? mine / (sum + sum_floor) * weight_scale : mine * weight_scale)
+        score != 0 ? (normalise ? mine / (sum + sum_floor) * weight_scale : mine * weight_scale)
                    : mine / sum;
   __syncwarp();  // a warp that goes on to another token writes the shared tables again
 }
@@ -121,7 +144,7 @@ __global__ void moe_route_kernel(const float* z, long long ld, const float* __re
                                  int E, int top, int* __restrict__ chosen,
                                  float* __restrict__ weights, int score, int groups, int keep,
                                  const float* __restrict__ correction, int normalise,
-                                 float sum_floor, float weight_scale) {
+                                 float sum_floor, float weight_scale, int group_best) {
   fb_pdl_launch();
   fb_pdl_wait();
   // one warp per token
@@ -129,7 +152,8 @@ __global__ void moe_route_kernel(const float* z, long long ld, const float* __re
   __shared__ float s_group[256];
   __shared__ float s_plain[256];
   route_token(z, ld, bias, E, top, chosen, weights, score, groups, keep, correction, normalise,
-              sum_floor, weight_scale, blockIdx.x, threadIdx.x & 31, s_all, s_group, s_plain);
+              sum_floor, weight_scale, group_best, blockIdx.x, threadIdx.x & 31, s_all, s_group,
+              s_plain);
 }
 
 template <typename T>
@@ -182,8 +206,12 @@ moe_experts_rows_kernel(const T* h, const T* __restrict__ gate_up, const T* __re
   __syncthreads();
   for (int c = 0; c < top; ++c) {
     const int e = __ldcg(chosen + (size_t)t * top + c);
-    if (e < 0 || e >= E) continue;  // uniform over the block
     const float wt = __ldcg(weights + (size_t)t * top + c);
+    if (e < 0 || e >= E) {  // an identity expert (uniform over the block)
+      for (int i = threadIdx.x; i < W; i += blockDim.x) acc[i] = fmaf(wt, x[i], acc[i]);
+      __syncthreads();
+      continue;
+    }
     const T* gu = gate_up + (size_t)e * 2 * ff * W;
     for (int f = warp; f < ff; f += nwarps) {
       float g = dot_row<T>(gu + (size_t)f * W, x, W, lane);
@@ -209,21 +237,22 @@ moe_experts_rows_kernel(const T* h, const T* __restrict__ gate_up, const T* __re
 FB_API int fb_moe_route(const float* z, long long ld, const float* bias, int E, int top,
                         int* chosen, float* weights, int T, int score, int groups, int keep,
                         const float* correction, int normalise, float sum_floor,
-                        float weight_scale, cudaStream_t stream) {
+                        float weight_scale, int group_best, cudaStream_t stream) {
   FB_REQUIRE(T >= 0 && E > 0 && E <= 256 && top > 0 && top <= E && top <= 32 && ld >= E,
              "moe_route: %d experts (at most 256), %d chosen (at most 32)", E, top);
-  FB_REQUIRE(score == 0 || score == 1, "moe_route: unknown scoring rule %d", score);
+  FB_REQUIRE(score >= 0 && score <= 2 && (group_best == 1 || group_best == 2),
+             "moe_route: unknown scoring rule %d (groups by their best %d)", score, group_best);
   FB_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups &&
              (long long)keep * (E / groups) >= top,
              "moe_route: %d groups of %d experts, %d kept, %d chosen", groups, E, keep, top);
-  FB_REQUIRE(score == 1 || groups == 1, "moe_route: groups need the sigmoid scores");
-  FB_REQUIRE(score == 1 || (correction == nullptr && !normalise && weight_scale == 1.0f),
+  FB_REQUIRE(score != 0 || groups == 1, "moe_route: groups need scores of their own");
+  FB_REQUIRE(score != 0 || (correction == nullptr && !normalise && weight_scale == 1.0f),
              "moe_route: a correction of the choice, shares of the sum and a constant on the "
-             "weights need the sigmoid scores");
+             "weights need scores of their own");
   if (T == 0) return 0;
   // a warp per token
   fb_launch(moe_route_kernel, dim3(T), dim3(32), 0, stream, z, ld, bias, E, top, chosen, weights,
-            score, groups, keep, correction, normalise, sum_floor, weight_scale);
+            score, groups, keep, correction, normalise, sum_floor, weight_scale, group_best);
   return fb_check_launch("moe_route");
 }
 
@@ -307,7 +336,7 @@ __device__ __forceinline__ void sort_pairs(const int* chosen, int n_pairs, int E
     if (lane == 0) { counts[e] = cnt[e]; starts[e] = start[e]; }
   }
   if (threadIdx.x == 0) starts[E] = start[E];
-  // pairs without a valid expert (never for finite logits) are put nowhere
+  // pairs without an expert among the first E (identity experts) are put nowhere
   for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
     const int e = chosen[i];
     if (e < 0 || e >= E) place[i] = -1;
@@ -328,7 +357,8 @@ __global__ void __launch_bounds__(ROUTE_SORT_WARPS * 32)
 moe_route_sort_kernel(const float* z, long long ld, const float* __restrict__ bias, int E, int top,
                       int* chosen, float* __restrict__ weights, int score, int groups, int keep,
                       const float* __restrict__ correction, int normalise, float sum_floor,
-                      float weight_scale, int T, int* __restrict__ counts,
+                      float weight_scale, int group_best, int experts, int T,
+                      int* __restrict__ counts,
                       int* __restrict__ starts, int* __restrict__ place,
                       int* __restrict__ pair_at) {
   fb_pdl_launch();
@@ -339,9 +369,10 @@ moe_route_sort_kernel(const float* z, long long ld, const float* __restrict__ bi
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int t = warp; t < T; t += ROUTE_SORT_WARPS)
     route_token(z, ld, bias, E, top, chosen, weights, score, groups, keep, correction, normalise,
-                sum_floor, weight_scale, t, lane, s_all[warp], s_group[warp], s_plain[warp]);
+                sum_floor, weight_scale, group_best, t, lane, s_all[warp], s_group[warp],
+                s_plain[warp]);
   __syncthreads();  // the block's own writes of `chosen` are visible to all its threads
-  sort_pairs(chosen, T * top, E, counts, starts, place, pair_at);
+  sort_pairs(chosen, T * top, experts, counts, starts, place, pair_at);
 }
 
 template <typename T>
@@ -596,17 +627,21 @@ moe_grouped_mma_kernel(const __nv_bfloat16* x, long long ldx, const __nv_bfloat1
 }
 
 // out[t] = sum_c weights[t, c] * y[place[t, c]] (+ addend[t], what every token gets
-// beside its experts: a shared expert's rows)
+// beside its experts: a shared expert's rows). A choice without a place is an identity
+// expert where `h` is given: weights[t, c] * h[t].
+template <typename T>
 __global__ void moe_combine_kernel(const float* y, const int* place, const float* weights, int top,
-                                   float* __restrict__ out, int W, const float* addend) {
+                                   float* __restrict__ out, int W, const float* addend, const T* h) {
   fb_pdl_launch();
   fb_pdl_wait();
   const size_t t = blockIdx.x;
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < W; i += gridDim.y * blockDim.x) {
     float acc = 0.f;
+    const float own = h != nullptr ? fb_load_coherent<T>(h + t * W + i) : 0.f;
     for (int c = 0; c < top; ++c) {
       const int at = place[t * top + c];
-      if (at >= 0) acc = fmaf(weights[t * top + c], __ldcg(y + (size_t)at * W + i), acc);
+      if (at < 0) acc = fmaf(weights[t * top + c], own, acc);
+      else acc = fmaf(weights[t * top + c], __ldcg(y + (size_t)at * W + i), acc);
     }
     if (addend != nullptr) acc += __ldcg(addend + t * W + i);
     out[t * W + i] = acc;
@@ -623,24 +658,27 @@ FB_API int fb_moe_sort(const int* chosen, int n_pairs, int E, int* counts, int* 
 }
 
 // fb_moe_route and fb_moe_sort as one launch of one block (for up to a few dozen tokens).
+// `experts`: how many of the E outputs have matrices; pairs of the others are sorted nowhere.
 FB_API int fb_moe_route_sort(const float* z, long long ld, const float* bias, int E, int top,
                              int* chosen, float* weights, int T, int score, int groups, int keep,
                              const float* correction, int normalise, float sum_floor,
-                             float weight_scale, int* counts, int* starts, int* place,
-                             int* pair_at, cudaStream_t stream) {
+                             float weight_scale, int group_best, int experts, int* counts,
+                             int* starts, int* place, int* pair_at, cudaStream_t stream) {
   FB_REQUIRE(T >= 0 && E > 0 && E <= 256 && top > 0 && top <= E && top <= 32 && ld >= E,
              "moe_route_sort: %d experts (at most 256), %d chosen (at most 32)", E, top);
-  FB_REQUIRE(score == 0 || score == 1, "moe_route_sort: unknown scoring rule %d", score);
+  FB_REQUIRE(score >= 0 && score <= 2 && (group_best == 1 || group_best == 2),
+             "moe_route_sort: unknown scoring rule %d (groups by their best %d)", score, group_best);
   FB_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups &&
              (long long)keep * (E / groups) >= top,
              "moe_route_sort: %d groups of %d experts, %d kept, %d chosen", groups, E, keep, top);
-  FB_REQUIRE(score == 1 || (groups == 1 && correction == nullptr && !normalise &&
+  FB_REQUIRE(score != 0 || (groups == 1 && correction == nullptr && !normalise &&
                             weight_scale == 1.0f),
              "moe_route_sort: groups, a correction, shares of the sum and a constant on the "
-             "weights need the sigmoid scores");
+             "weights need scores of their own");
+  FB_REQUIRE(experts > 0 && experts <= E, "moe_route_sort: %d experts of %d outputs", experts, E);
   fb_launch(moe_route_sort_kernel, dim3(1), dim3(ROUTE_SORT_WARPS * 32), 0, stream, z, ld, bias, E,
             top, chosen, weights, score, groups, keep, correction, normalise, sum_floor,
-            weight_scale, T, counts, starts, place, pair_at);
+            weight_scale, group_best, experts, T, counts, starts, place, pair_at);
   return fb_check_launch("moe_route_sort");
 }
 
@@ -740,12 +778,13 @@ FB_API int fb_moe_grouped_mma(int gated, const void* x, long long ldx, const voi
 }
 
 FB_API int fb_moe_combine(const float* y, const int* place, const float* weights, int top,
-                          float* out, int T, int W, const float* addend, cudaStream_t stream) {
+                          float* out, int T, int W, const float* addend, const void* h,
+                          int h_dtype, cudaStream_t stream) {
   FB_REQUIRE(T >= 0 && W > 0 && top > 0, "moe_combine: bad sizes");
   if (T == 0) return 0;
   const int want = (W + 255) / 256;  // few tokens: a row's columns go to several blocks
   const int parts = T <= 256 ? (want < 32 ? want : 32) : 1;
-  fb_launch(moe_combine_kernel, dim3(T, parts), dim3(256), 0, stream, y, place, weights, top, out, W,
-            addend);
+  FB_DISPATCH_DTYPE(h_dtype, E, (fb_launch(moe_combine_kernel<E>, dim3(T, parts), dim3(256), 0,
+      stream, y, place, weights, top, out, W, addend, (const E*)h)));
   return fb_check_launch("moe_combine");
 }

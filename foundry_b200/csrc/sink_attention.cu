@@ -119,10 +119,37 @@ struct ScoreRule {
   const float* sink_logit;
   float scale, steep, softcap;
   float lambda, post_eps, post_scale;
+  // A learnt bias by distance, float32 [H, dist_last + 1], or null: a score gains
+  // dist_bias[head][min(i - j, dist_last)] behind the constant and the cap.
+  const float* dist_bias;
+  int dist_last;
+  // A number a key row that its scores are multiplied by (the reciprocal root mean square of
+  // a row that is cached as it was projected), or null: [pages][G][FB_PAGE] with these strides.
+  const float* key_scale;
+  long long ks_page, ks_head;
+  // float32 rows [T, H * VD], or null: the output is multiplied by sigmoid(gate) at the end.
+  const float* gate;
+  long long gate_stride;
 };
 
 __device__ __forceinline__ float capped(float s, float cap) {
   return cap > 0.f ? cap * tanhf(s / cap) : s;
+}
+
+__device__ __forceinline__ float key_factor(const ScoreRule& rule, int g, long long page, int r) {
+  return rule.key_scale == nullptr
+             ? rule.scale
+             : rule.scale * __ldcg(rule.key_scale + page * rule.ks_page + g * rule.ks_head + r);
+}
+__device__ __forceinline__ float distance_bias(const ScoreRule& rule, int head, int away) {
+  return rule.dist_bias == nullptr
+             ? 0.f
+             : rule.dist_bias[(size_t)head * (rule.dist_last + 1) + min(away, rule.dist_last)];
+}
+__device__ __forceinline__ float gate_factor(const ScoreRule& rule, size_t t, size_t column) {
+  return rule.gate == nullptr
+             ? 1.0f
+             : 1.0f / (1.0f + expf(-__ldcg(rule.gate + t * rule.gate_stride + column)));
 }
 
 // Value rows lie `v_row` elements apart and key rows `k_row` (so values may be a
@@ -200,6 +227,8 @@ attention_sink_kernel(const T* q, long long q_stride, T* __restrict__ out, long 
         const int r = j % FB_PAGE;
         v_off = page * v_page + (long long)r * v_row;
         const T* krow = kbase + page * k_page + (long long)r * k_row;
+        const float factor = key_factor(rule, g, page, r);
+        const float by_distance = distance_bias(rule, a, pos - j) - slope * (float)(pos - j);
 #pragma unroll
         for (int mm = 0; mm < MAPS; ++mm) {
           const float* qm = qs + mm * D;
@@ -220,7 +249,7 @@ attention_sink_kernel(const T* q, long long q_stride, T* __restrict__ out, long 
           } else {
             for (int d = 0; d < D; ++d) dot = fmaf(qm[d], fb_load_coherent<T>(km + d), dot);
           }
-          s[mm] = capped(dot * rule.scale, rule.softcap) - slope * (float)(pos - j);
+          s[mm] = capped(dot * factor, rule.softcap) + by_distance;
         }
       }
       float p[MAPS];
@@ -324,7 +353,8 @@ attention_sink_kernel(const T* q, long long q_stride, T* __restrict__ out, long 
 #pragma unroll
     for (int i = 0; i < NACC; ++i) {
       const int d = place(i);
-      if (writer && d < VD) o[d] = fb_from_float<T>(acc[0][i] * inv_l);
+      if (writer && d < VD)
+        o[d] = fb_from_float<T>(acc[0][i] * inv_l * gate_factor(rule, t, (size_t)a * VD + d));
     }
     return;
   }
@@ -340,7 +370,8 @@ attention_sink_kernel(const T* q, long long q_stride, T* __restrict__ out, long 
 #pragma unroll
   for (int i = 0; i < NACC; ++i) {
     const int d = place(i);
-    if (writer && d < VD) o[d] = fb_from_float<T>(acc[0][i] * r);
+    if (writer && d < VD)
+      o[d] = fb_from_float<T>(acc[0][i] * r * gate_factor(rule, t, (size_t)a * VD + d));
   }
 }
 
@@ -469,6 +500,11 @@ attention_sink_staged_kernel(const T* q, long long q_stride, T* __restrict__ out
       if (!active) continue;
       const int j = j0 + lane;
       float s[MAPS], p[MAPS];
+      float factor = 0.f, by_distance = 0.f;
+      if (lane < n) {
+        factor = key_factor(rule, g, pages[j / FB_PAGE], j % FB_PAGE);
+        by_distance = distance_bias(rule, a, pos - j) - slope * (float)(pos - j);
+      }
 #pragma unroll
       for (int mm = 0; mm < MAPS; ++mm) {
         s[mm] = -INFINITY;
@@ -490,7 +526,7 @@ attention_sink_staged_kernel(const T* q, long long q_stride, T* __restrict__ out
 #pragma unroll
               for (int e = 0; e < 8; ++e) d1 = fmaf(qb[e], kb[e], d1);
           }
-          s[mm] = capped((d0 + d1) * rule.scale, rule.softcap) - slope * (float)(pos - j);
+          s[mm] = capped((d0 + d1) * factor, rule.softcap) + by_distance;
         }
         const float m_new = fmaxf(m[mm], fb_warp_max(s[mm]));
         const float corr = expf(m[mm] - m_new);
@@ -548,7 +584,8 @@ attention_sink_staged_kernel(const T* q, long long q_stride, T* __restrict__ out
 #pragma unroll
     for (int i = 0; i < NACC; ++i) {
       const int d = place(i);
-      if (writer && d < VD) o[d] = fb_from_float<T>(acc[0][i] * inv_l);
+      if (writer && d < VD)
+        o[d] = fb_from_float<T>(acc[0][i] * inv_l * gate_factor(rule, t, (size_t)a * VD + d));
     }
     return;
   }
@@ -564,7 +601,8 @@ attention_sink_staged_kernel(const T* q, long long q_stride, T* __restrict__ out
 #pragma unroll
   for (int i = 0; i < NACC; ++i) {
     const int d = place(i);
-    if (writer && d < VD) o[d] = fb_from_float<T>(acc[0][i] * r);
+    if (writer && d < VD)
+      o[d] = fb_from_float<T>(acc[0][i] * r * gate_factor(rule, t, (size_t)a * VD + d));
   }
 }
 
@@ -638,7 +676,7 @@ __global__ void attention_sink_merge_kernel(const float* partial, T* __restrict_
 #pragma unroll
   for (int i = 0; i < NACC; ++i) {
     const int d = lane + 32 * i;
-    if (d < VD) o[d] = fb_from_float<T>(acc[0][i] * r);
+    if (d < VD) o[d] = fb_from_float<T>(acc[0][i] * r * gate_factor(rule, t, (size_t)a * VD + d));
   }
 }
 
@@ -873,9 +911,15 @@ FB_API int fb_attention_sink(const void* q, long long q_stride, void* out, long 
                              long long v_page, long long v_head, int k_row, int v_row, int window,
                              int keep_first, int sink, const float* sink_logit, float scale,
                              float steep, float softcap, int maps, float lambda, float post_eps,
-                             float post_scale, int T, int H, int G, int D, int VD, int splits,
-                             float* partial, cudaStream_t stream) {
+                             float post_scale, const float* dist_bias, int dist_last,
+                             const float* key_scale, long long ks_page, long long ks_head,
+                             const float* gate, long long gate_stride, int T, int H, int G, int D,
+                             int VD, int splits, float* partial, cudaStream_t stream) {
   FB_REQUIRE(T >= 0 && H > 0 && G > 0 && D > 0 && VD > 0, "attention_sink: bad sizes");
+  FB_REQUIRE(dist_bias == nullptr || dist_last >= 0, "attention_sink: a bias table ending at %d",
+             dist_last);
+  FB_REQUIRE(gate == nullptr || gate_stride >= (long long)H * VD,
+             "attention_sink: gate rows of %lld", gate_stride);
   FB_REQUIRE(H % G == 0, "attention_sink: %d query heads are not a multiple of %d key-value heads",
              H, G);
   FB_REQUIRE(maps == 1 || maps == 2, "attention_sink: %d maps a head (1 or 2)", maps);
@@ -892,7 +936,7 @@ FB_API int fb_attention_sink(const void* q, long long q_stride, void* out, long 
              "attention_sink: %d runs need a workspace", splits);
   if (T == 0) return 0;
   ScoreRule rule{window, keep_first, sink, sink_logit, scale, steep, softcap, lambda, post_eps,
-                 post_scale};
+                 post_scale, dist_bias, dist_last, key_scale, ks_page, ks_head, gate, gate_stride};
   dim3 grid(T, (H + WARPS - 1) / WARPS, splits);
   const bool vec = VD % 8 == 0 && v_row % 8 == 0 && v_page % 8 == 0 && v_head % 8 == 0 &&
                    ((uintptr_t)v_cache % 32) == 0;
@@ -960,7 +1004,8 @@ FB_API int fb_attention_sink_merge(const float* partial, void* out, long long ou
   FB_REQUIRE(T >= 0 && H > 0 && VD > 0 && VD <= 768 && splits >= 1 && splits <= 64 && partial != nullptr,
              "attention_sink_merge: bad sizes");
   if (T == 0) return 0;
-  ScoreRule rule{0, 0, sink_logit != nullptr ? 2 : 0, sink_logit, 1.f, 0.f, 0.f, 0.f, 0.f, 1.f};
+  ScoreRule rule{0, 0, sink_logit != nullptr ? 2 : 0, sink_logit, 1.f, 0.f, 0.f, 0.f, 0.f, 1.f,
+                 nullptr, 0, nullptr, 0, 0, nullptr, 0};
   if (VD > 256) {
     FB_DISPATCH_DTYPE(dtype, E, (fb_launch(attention_sink_merge_kernel<E, 1, 24>,
         dim3(T, (H + WARPS - 1) / WARPS), dim3(WARPS * 32), 0, stream, partial, (E*)out, out_stride,

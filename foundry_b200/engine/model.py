@@ -163,6 +163,8 @@ class Model:
             self.embedder.forward(ctx, self.embedding, resid, x0)
         if keeps:
             ctx.shared[EMBEDDING_OUTPUT] = x0
+        if spec.streams:  # copies of the stream, equal until the first part's result joins them
+            resid = ops.Streams(spec.streams, first=resid)
         delta = None
         for i, entry in enumerate(spec.schedule):
             block = self.blocks[entry.layer]
@@ -183,6 +185,11 @@ class Model:
         logits = torch.empty((n, spec.vocab_size), dtype=torch.float32, device=self.device)
         if n == 0:
             return logits
+        if spec.streams:
+            normed = self.final_norm.add_norm(
+                resid.take(ctx.want_rows, n).read(None),
+                None if delta is None else delta.take(ctx.want_rows, n))
+            return self._logits(normed, logits)
         if isinstance(delta, ops.DepthMix):  # the last stream is a sum over the kept ones
             delta = delta.settle(resid)
         rows = torch.empty((n, spec.hidden_size), dtype=torch.float32, device=self.device)
@@ -202,7 +209,10 @@ class Model:
             ops.gather_rows(delta, ctx.want_rows, rows_delta)
             if scale is not None:
                 rows_delta = ops.ScaledDelta(rows_delta, scale)
-        normed = self.final_norm.add_norm(rows, rows_delta)
+        return self._logits(self.final_norm.add_norm(rows, rows_delta), logits)
+
+    def _logits(self, normed, logits: torch.Tensor) -> torch.Tensor:
+        spec = self.spec
         matmul_nt(normed, self.output_head, logits)
         if spec.logit_softcap is not None:  # logits <- cap * tanh(logits / cap)
             ops.softcap(logits, spec.logit_softcap)

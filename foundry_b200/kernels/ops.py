@@ -35,6 +35,11 @@ _SIGNATURES = {
     "fb_add_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_ll, c_void_p, c_float, c_void_p, c_int,
                        c_int, c_int, c_float, c_void_p],
     "fb_silu_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "fb_glu_clamped": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float,
+                       c_float, c_void_p],
+    "fb_stream_mix_norm": [c_void_p, c_ll, c_ll, c_void_p, c_int, c_int, c_ll, c_void_p, c_void_p,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                           c_int, c_float, c_void_p],
     "fb_gather_rows": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "fb_cast": [c_void_p, c_int, c_void_p, c_int, c_ll, c_void_p],
     "fb_rope_kv_write": [c_void_p, c_int, c_ll, c_int, c_ll, c_void_p, c_int, c_ll, c_void_p,
@@ -106,7 +111,8 @@ _SIGNATURES = {
                                       c_float, c_int, c_int, c_void_p, c_int, c_int,
                                       c_void_p, c_void_p,
                                       c_void_p, c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll,
-                                      c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                                      c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll,
+                                      c_ll, c_void_p],
     "fb_step_angles": [c_void_p, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p],
     "fb_attention_sigmoid": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p,
                              c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll, c_void_p, c_void_p,
@@ -132,8 +138,8 @@ _SIGNATURES = {
     "fb_attention_sink": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p,
                           c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll, c_int, c_int, c_int,
                           c_int, c_int, c_void_p, c_float, c_float, c_float, c_int, c_float,
-                          c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                          c_void_p],
+                          c_float, c_float, c_void_p, c_int, c_void_p, c_ll, c_ll, c_void_p, c_ll,
+                          c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "fb_q_temp_cache_write": [c_void_p, c_ll, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p,
                               c_void_p, c_int, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll, c_int,
                               c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -181,10 +187,10 @@ _SIGNATURES = {
     "fb_add_into": [c_void_p, c_void_p, c_ll, c_void_p],
     "fb_sigmoid_gate": [c_void_p, c_int, c_ll, c_void_p, c_ll, c_int, c_int, c_void_p],
     "fb_moe_route_sort": [c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
-                          c_int, c_int, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p,
-                          c_void_p, c_void_p, c_void_p],
+                          c_int, c_int, c_void_p, c_int, c_float, c_float, c_int, c_int, c_void_p,
+                          c_void_p, c_void_p, c_void_p, c_void_p],
     "fb_moe_route": [c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                     c_int, c_void_p, c_int, c_float, c_float, c_void_p],
+                     c_int, c_void_p, c_int, c_float, c_float, c_int, c_void_p],
     "fb_moe_experts_rows": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p,
                             c_void_p],
@@ -199,7 +205,7 @@ _SIGNATURES = {
     "fb_moe_grouped_mma": [c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_int,
                            c_int, c_float, c_float, c_float, c_void_p, c_int, c_void_p],
     "fb_moe_combine": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
-                       c_void_p],
+                       c_void_p, c_int, c_void_p],
 }
 
 _FUNCS = {}
@@ -530,6 +536,20 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False
     _call("fb_silu_mul", _dev(gate_up, "gate_up"), code_of(gate_up.dtype), _dev(out, "out"),
           code_of(out.dtype), T, two_i // 2, 1 if interleaved else 0, GLU_ACTIVATIONS[act],
           _stream())
+    return out
+
+
+def glu_clamped(gate_up: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
+                limit: float, alpha: float, shift: float) -> torch.Tensor:
+    """out[t,i] = min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, +-limit) + shift) with
+    g, u = columns 2i, 2i + 1 of `gate_up` plus `bias` (float32 [2I], the same order)."""
+    T, two_i = gate_up.shape
+    if two_i % 2 or tuple(out.shape) != (T, two_i // 2) or (bias is not None
+                                                            and bias.numel() != two_i):
+        raise KernelError(f"glu_clamped: gate_up {tuple(gate_up.shape)} / out {tuple(out.shape)}")
+    _call("fb_glu_clamped", _dev(gate_up, "gate_up"), code_of(gate_up.dtype),
+          0 if bias is None else _dev(bias, "bias", torch.float32), _dev(out, "out"),
+          code_of(out.dtype), T, two_i // 2, float(limit), float(alpha), float(shift), _stream())
     return out
 
 
@@ -1823,6 +1843,99 @@ def post_norm_add(resid: torch.Tensor, pending: Optional[PostNormed], weight: Op
     return out
 
 
+class Streams:
+    """A residual of several streams: float32 `values` [T, S, W], or, before the first part
+    has written them, one row a token (`first` [T, W]) that all streams are equal to."""
+
+    def __init__(self, count: int, first: Optional[torch.Tensor] = None,
+                 values: Optional[torch.Tensor] = None):
+        self.count, self.first, self.values = int(count), first, values
+
+    @property
+    def shape(self):
+        """[T, W]: of what a part reads."""
+        if self.values is None:
+            return tuple(self.first.shape)
+        return (self.values.shape[0], self.values.shape[2])
+
+    @property
+    def device(self):
+        return (self.first if self.values is None else self.values).device
+
+    def read(self, weights: Optional[torch.Tensor]) -> "StreamRead":
+        return StreamRead(self, weights)
+
+    def take(self, rows: torch.Tensor, n: int) -> "Streams":
+        """The same for `n` rows of the step only."""
+        if self.values is None:
+            return Streams(self.count, first=_taken(self.first, rows, n))
+        T, S, W = self.values.shape
+        return Streams(S, values=_taken(self.values.view(T, S * W), rows, n).view(n, S, W))
+
+
+class StreamRead:
+    """What a norm in front of a part normalises: the sum of `streams` with `weights`
+    (float32 [S]; None: the plain sum, the model's end, where nothing is kept)."""
+
+    def __init__(self, streams: Streams, weights: Optional[torch.Tensor]):
+        self.streams, self.weights = streams, weights
+
+    @property
+    def shape(self):
+        return self.streams.shape
+
+    @property
+    def device(self):
+        return self.streams.device
+
+
+class StreamDelta:
+    """A part's output on its way into the streams: z_t = sum_s mix[s, t] x_s + share[t] *
+    (values + bias). Rows (float32 or bfloat16) or float32 split-K `Planes`."""
+
+    def __init__(self, values, mix: torch.Tensor, share: torch.Tensor,
+                 bias: Optional[torch.Tensor] = None):
+        self.values, self.mix, self.share, self.bias = values, mix, share, bias
+
+    def take(self, rows: torch.Tensor, n: int) -> "StreamDelta":
+        return StreamDelta(_taken(self.values, rows, n), self.mix, self.share, self.bias)
+
+
+def stream_mix_norm(read: StreamRead, delta: Optional[StreamDelta], weight: torch.Tensor,
+                    eps: float, out: torch.Tensor) -> torch.Tensor:
+    """The pending output goes into the streams (written in place, or made from the one row
+    they were), out = rms_norm(their weighted sum): one pass over every token's row
+    (csrc/stream_mix.cu)."""
+    st = read.streams
+    T, W = st.shape
+    S = st.count
+    if tuple(out.shape) != (T, W) or tuple(weight.shape) != (W,):
+        raise KernelError(f"stream_mix_norm: out {tuple(out.shape)}, weight {tuple(weight.shape)} "
+                          f"for rows {(T, W)}")
+    x, strides = (st.first, (W, 0)) if st.values is None else (st.values, (S * W, W))
+    y, planes, plane_stride, bias, z = None, 1, 0, None, None
+    if delta is not None:
+        y, bias = delta.values, delta.bias
+        if isinstance(y, Planes):
+            y, planes, plane_stride = y.tensor, y.count, T * W
+        if tuple(y.shape[-2:]) != (T, W) or tuple(delta.mix.shape) != (S, S) \
+                or tuple(delta.share.shape) != (S,):
+            raise KernelError(f"stream_mix_norm: a result of {tuple(y.shape)} for {S} streams of "
+                              f"{(T, W)}")
+        if read.weights is not None:  # (at the model's end nothing reads the streams again)
+            if st.values is None:
+                st.values = torch.empty((T, S, W), dtype=torch.float32, device=x.device)
+            z = st.values
+    f32 = lambda t, n: 0 if t is None else _dev(t, n, torch.float32)
+    _call("fb_stream_mix_norm", _dev(x, "streams", torch.float32), *strides,
+          0 if y is None else _dev(y, "values"), F32 if y is None else code_of(y.dtype), planes,
+          plane_stride, f32(bias, "bias"), f32(None if delta is None else delta.mix, "mix"),
+          f32(None if delta is None else delta.share, "share"), f32(read.weights, "in"),
+          f32(z, "streams"), _dev(weight, "weight", torch.float32), _dev(out, "out"),
+          code_of(out.dtype), T, S, W, float(eps), _stream())
+    return out
+
+
 class DepthMix:
     """A stream that is still to be replaced by a weighted sum over the streams
     the layers so far have left: with X_0 = `first`, X_1 .. X_(n-1) the first rows
@@ -1968,14 +2081,20 @@ def attention_sink(ctx, q: torch.Tensor, out: torch.Tensor, page_table, k_cache,
                    G: int, dim: int, vdim: int, scale: float, window: int = 0, keep_first: int = 0,
                    sink: bool = False, steep: float = 0.0, softcap: float = 0.0,
                    sink_logits: Optional[torch.Tensor] = None, maps: int = 1,
-                   combine: Optional[tuple] = None, values_in_keys: bool = False) -> torch.Tensor:
+                   combine: Optional[tuple] = None, values_in_keys: bool = False,
+                   dist_bias: Optional[torch.Tensor] = None,
+                   key_scales: Optional[torch.Tensor] = None,
+                   gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of every token of the step over its sequence's cache,
     with the mask, bias, score cap, sink and maps of csrc/sink_attention.cu.
     `sink_logits` (float32 [H]): the sink's score per head instead of 0. `maps` 2: a
     query head has two query vectors and a key row two key vectors of `dim` side by
     side, and `combine` = (lambda, eps, scale) joins the two maps' outputs as
     (a1 - lambda a2) / rms * scale. `values_in_keys`: the value of a token is the first
-    `vdim` elements of its key row (`v_cache` is not looked at).
+    `vdim` elements of its key row (`v_cache` is not looked at). `dist_bias` (float32
+    [H, n]): a score of distance m gains dist_bias[head, min(m, n - 1)]. `key_scales`
+    (float32 [pages, G, PAGE], contiguous rows): a factor of each key row's scores. `gate`
+    (float32 rows [T, H * vdim]): the outputs are multiplied by its sigmoid.
     Prompts in bfloat16 with none of these, whose keys and values have one
     tensor-core head size, run the masked form of the tensor-core prompt kernel;
     everything else the CUDA-core kernel, whose single-token steps cut every
@@ -1993,7 +2112,15 @@ def attention_sink(ctx, q: torch.Tensor, out: torch.Tensor, page_table, k_cache,
         _check_kv_pair(k_cache, v_cache, G, k_row, vdim, q.dtype)
     if maps not in (1, 2) or (maps == 2) != (combine is not None):
         raise KernelError("attention_sink: two maps a head need `combine`, one map takes none")
-    plain_rule = softcap == 0.0 and maps == 1 and not values_in_keys
+    plain_rule = (softcap == 0.0 and maps == 1 and not values_in_keys and dist_bias is None
+                  and key_scales is None and gate is None)
+    if dist_bias is not None and (dist_bias.dim() != 2 or dist_bias.shape[0] != H):
+        raise KernelError(f"attention_sink: a bias table of {tuple(dist_bias.shape)} for {H} heads")
+    if key_scales is not None and (tuple(key_scales.shape) != (k_cache.shape[0], G, PAGE)
+                                   or key_scales.stride(2) != 1):
+        raise KernelError(f"attention_sink: key scales of {tuple(key_scales.shape)}")
+    if gate is not None and tuple(gate.shape) != (T, H * vdim):
+        raise KernelError(f"attention_sink: a gate of {tuple(gate.shape)}")
     if sink_logits is not None and tuple(sink_logits.shape) != (H,):
         raise KernelError(f"attention_sink: {tuple(sink_logits.shape)} sink scores for {H} heads")
     if (SINK_ATTENTION_TC and plain_rule and not ctx.is_decode and q.dtype == torch.bfloat16
@@ -2043,8 +2170,31 @@ def attention_sink(ctx, q: torch.Tensor, out: torch.Tensor, page_table, k_cache,
           v_cache.stride(0), v_cache.stride(1), k_row, v_row, window, keep_first, sink_mode,
           0 if sink_logits is None else _dev(sink_logits, "sink_logits", torch.float32),
           float(scale), float(steep), float(softcap), maps, float(lam), float(post_eps),
-          float(post_scale), T, H, G, dim, vdim, splits, partial, _stream())
+          float(post_scale),
+          0 if dist_bias is None else _dev(dist_bias, "dist_bias", torch.float32),
+          0 if dist_bias is None else dist_bias.shape[1] - 1,
+          0 if key_scales is None else _dev(key_scales, "key_scales", torch.float32,
+                                            contiguous=False),
+          *((0, 0) if key_scales is None else key_scales.stride()[:2]),
+          0 if gate is None else _dev(gate, "gate", torch.float32, contiguous=False),
+          0 if gate is None else _rows(gate, "gate"), T, H, G, dim, vdim, splits, partial,
+          _stream())
     return out
+
+
+def attention_shared_rows(ctx, q: torch.Tensor, out: torch.Tensor, page_table, rows, scales, H: int,
+                          G: int, dim: int, scale: float, window: int = 0, keep_first: int = 0,
+                          dist_bias: Optional[torch.Tensor] = None,
+                          gate: Optional[torch.Tensor] = None,
+                          then_reads: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Softmax attention whose values are its keys before their norm: a token has ONE cached
+    row a head (`rows` [pages, G, PAGE, dim]), read as the value and, times its factor
+    (`scales` [pages, G, PAGE], the reciprocal root mean square), as the key. Position i sees
+    j <= i where i - j < window or j < keep_first (window 0: all); `dist_bias` and `gate` as
+    in `attention_sink`."""
+    return attention_sink(ctx, q, out, page_table, rows, rows, H, G, dim, dim, scale, window=window,
+                          keep_first=keep_first, values_in_keys=True, dist_bias=dist_bias,
+                          key_scales=scales, gate=gate)
 
 
 WINDOW_ATTENTION_TC = _os.environ.get("FOUNDRY_B200_WINDOW_ATTENTION_TC", "1") != "0"
@@ -2293,16 +2443,23 @@ def head_norm_rope_cache_write(qkv: torch.Tensor, q_out: torch.Tensor,
                                value_norm: bool, ctx, rotation: Rotation, page_table, k_cache,
                                v_cache, H: int, G: int, dim: int, vdim: int,
                                write_cache: bool = True, qk_norm: bool = True,
-                               bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                               bias: Optional[torch.Tensor] = None,
+                               key_scales: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Per-head RMS norms of queries and keys (weights [dim] shared by the heads, or
     none; `qk_norm` False: queries and keys stay as they are), the `rotation` of their first
     elements by the angles of the tokens' positions, the values' RMS norm without weight
     where `value_norm`; queries to `q_out`, keys and values into the token's cache row.
     `bias` (float32 [H * dim + G * (dim + vdim)]) is added to the rows first.
-    `qkv`: float32 rows [q | k | v]; with G = 0 rows of queries only (nothing is cached)."""
+    `qkv`: float32 rows [q | k | v]; with G = 0 rows of queries only (nothing is cached).
+    `key_scales` (float32 [pages, G, PAGE]): keys and values are one row, cached as it was
+    projected with its reciprocal root mean square there; `qkv` is [q | k | anything] and
+    `wq` carries the keys' weight, too."""
     T = qkv.shape[0]
     kp = vp = 0
     ks = vs = (0, 0)
+    if key_scales is not None and (tuple(key_scales.shape) != (k_cache.shape[0], G, PAGE)
+                                   or key_scales.stride(2) != 1):
+        raise KernelError(f"head_norm_rope_cache_write: key scales of {tuple(key_scales.shape)}")
     if write_cache:
         _check_kv_pair(k_cache, v_cache, G, dim, vdim, q_out.dtype)
         kp, vp = k_cache.data_ptr(), v_cache.data_ptr()
@@ -2322,7 +2479,9 @@ def head_norm_rope_cache_write(qkv: torch.Tensor, q_out: torch.Tensor,
           _dev(ctx.positions, "positions", torch.int32),
           _dev(ctx.seq_of_token, "seq_of_token", torch.int32),
           _dev(page_table, "page_table", torch.int32), page_table.shape[1], kp, vp, *ks, *vs,
-          T, H, G, dim, vdim, 1 if write_cache else 0, _stream())
+          T, H, G, dim, vdim, 1 if write_cache else 0,
+          0 if key_scales is None else _dev(key_scales, "key_scales", torch.float32, contiguous=False),
+          *((0, 0) if key_scales is None else key_scales.stride()[:2]), _stream())
     return q_out
 
 
@@ -2623,21 +2782,23 @@ def unary_cast(x: torch.Tensor, out: torch.Tensor, act: str = "identity") -> tor
 
 
 # ------------------------------------------------------------------ routed experts
-MOE_SCORES = {"softmax_chosen": 0, "sigmoid": 1}
+MOE_SCORES = {"softmax_chosen": 0, "sigmoid": 1, "softmax": 2}
 
 
 def moe_route(z: torch.Tensor, bias: Optional[torch.Tensor], top: int, chosen: torch.Tensor,
               weights: torch.Tensor, score: str = "softmax_chosen", groups: int = 1,
               keep: int = 1, correction: Optional[torch.Tensor] = None,
               normalise: bool = False, sum_floor: float = 0.0,
-              weight_scale: float = 1.0) -> None:
+              weight_scale: float = 1.0, group_best: int = 2) -> None:
     """The `top` experts of every token and their weights from the router's float32
     rows `z` (+ `bias`). "softmax_chosen": the largest z, weighted by the softmax over
     the chosen ones. "sigmoid": scores s = sigmoid(z); the choice goes by s (+ `correction`,
     float32 [E], which never enters a weight); of `groups` equal groups of neighbouring
     experts only the `keep` with the largest sum of their two best choice values can be
     chosen (the others count as minus infinity); the weights are the chosen s themselves or,
-    with `normalise`, s / (their sum + `sum_floor`), times `weight_scale`."""
+    with `normalise`, s / (their sum + `sum_floor`), times `weight_scale`. "softmax": the
+    same with s = softmax(z) over all outputs. `group_best` 1: a group's score is its largest
+    choice value alone."""
     T, E = z.shape
     if correction is not None and tuple(correction.shape) != (E,):
         raise KernelError(f"moe_route: a correction of {tuple(correction.shape)} for {E} experts")
@@ -2646,7 +2807,7 @@ def moe_route(z: torch.Tensor, bias: Optional[torch.Tensor], top: int, chosen: t
           _dev(chosen, "chosen", torch.int32), _dev(weights, "weights", torch.float32), T,
           MOE_SCORES[score], int(groups), int(keep),
           0 if correction is None else _dev(correction, "correction", torch.float32),
-          1 if normalise else 0, float(sum_floor), float(weight_scale), _stream())
+          1 if normalise else 0, float(sum_floor), float(weight_scale), int(group_best), _stream())
 
 
 def moe_experts_rows(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor,
@@ -2694,23 +2855,28 @@ def moe_route_sorted(z: torch.Tensor, bias: Optional[torch.Tensor], top: int, ch
                      weights: torch.Tensor, score: str = "softmax_chosen", groups: int = 1,
                      keep: int = 1, correction: Optional[torch.Tensor] = None,
                      normalise: bool = False, sum_floor: float = 0.0,
-                     weight_scale: float = 1.0) -> ExpertOrder:
+                     weight_scale: float = 1.0, group_best: int = 2,
+                     experts: Optional[int] = None) -> ExpertOrder:
     """`moe_route` and the sort of the chosen pairs by expert: for up to
-    `MOE_ROUTE_SORT_ROWS` tokens one launch of one block, else the two kernels."""
+    `MOE_ROUTE_SORT_ROWS` tokens one launch of one block, else the two kernels. `experts`:
+    how many of the router's outputs have matrices (all by default); a pair of one of the
+    others has no place in the order."""
     T, E = z.shape
+    experts = E if experts is None else experts
     if not 0 < T <= MOE_ROUTE_SORT_ROWS:
         moe_route(z, bias, top, chosen, weights, score, groups, keep, correction, normalise,
-                  sum_floor, weight_scale)
-        return ExpertOrder(chosen, E)
+                  sum_floor, weight_scale, group_best)
+        return ExpertOrder(chosen, experts)
     if correction is not None and tuple(correction.shape) != (E,):
         raise KernelError(f"moe_route: a correction of {tuple(correction.shape)} for {E} experts")
-    order = ExpertOrder(chosen, E, sort=False)
+    order = ExpertOrder(chosen, experts, sort=False)
     _call("fb_moe_route_sort", _dev(z, "z", torch.float32, contiguous=False), _rows(z, "z"),
           0 if bias is None else _dev(bias, "bias", torch.float32), E, top,
           _dev(chosen, "chosen", torch.int32), _dev(weights, "weights", torch.float32), T,
           MOE_SCORES[score], int(groups), int(keep),
           0 if correction is None else _dev(correction, "correction", torch.float32),
-          1 if normalise else 0, float(sum_floor), float(weight_scale), order.counts.data_ptr(),
+          1 if normalise else 0, float(sum_floor), float(weight_scale), int(group_best), experts,
+          order.counts.data_ptr(),
           order.starts.data_ptr(), order.place.data_ptr(), order.pair_at.data_ptr(), _stream())
     return order
 
@@ -2838,10 +3004,15 @@ def moe_grouped_mma(x: torch.Tensor, w: torch.Tensor, order: ExpertOrder, gated:
 
 
 def moe_combine(y: torch.Tensor, order: ExpertOrder, weights: torch.Tensor,
-                out: torch.Tensor, addend: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[t] = the weighted sum of token t's experts' rows of `y` (+ addend[t])."""
+                out: torch.Tensor, addend: Optional[torch.Tensor] = None,
+                identity: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t] = the weighted sum of token t's experts' rows of `y` (+ addend[t]); a choice
+    without a place in the order counts the token's row of `identity` (the part's input)."""
+    if identity is not None and tuple(identity.shape) != (order.T, out.shape[1]):
+        raise KernelError(f"moe_combine: identity rows {tuple(identity.shape)}")
     _call("fb_moe_combine", _dev(y, "y", torch.float32), order.place.data_ptr(),
           _dev(weights, "weights", torch.float32), order.top, _dev(out, "out", torch.float32),
           order.T, out.shape[1], 0 if addend is None else _dev(addend, "addend", torch.float32),
-          _stream())
+          0 if identity is None else _dev(identity, "identity"),
+          F32 if identity is None else code_of(identity.dtype), _stream())
     return out

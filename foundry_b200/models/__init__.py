@@ -1,2 +1,2 @@
 """Built-in architectures; importing this package registers them."""
-from . import kutepel, llama, rupotar, tokovik, vikarax, vonulorn  # noqa: F401
+from . import kutepel, llama, nemasun, rupotar, tokovik, vikarax, vonulorn  # noqa: F401

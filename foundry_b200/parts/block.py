@@ -440,6 +440,97 @@ class ParallelResidualBlock(Part):
         return ops.ScaledDelta(both, self.residual_scale)
 
 
+@register_block("stream_mix_residual")
+class StreamMixBlock(Part):
+    """Several residual streams x_1 .. x_S in place of one. For the mixer and then the
+    feed-forward (where the layer has one), each with three tensors of its own:
+
+        u = sum_s in[s] x_s;  y = part(norm(u));  x_t <- sum_s mix[s, t] x_s + out[t] * y
+
+    all streams at once from the old ones. A part's output leaves as an `ops.StreamDelta`,
+    and the norm that runs next mixes the streams, adds the shares, reads its own weighted
+    sum and normalises it in one pass over the row. A feed-forward that says `defers_bias`
+    leaves the bias on its output to that pass, too."""
+    replay_safe = True
+
+    def __init__(self, layer: LayerSpec, streams: int, mixer_name: str = "hc1",
+                 feed_forward_name: str = "hc2", *, dtype: torch.dtype, device: torch.device):
+        ctx = dict(dtype=dtype, device=device)
+        if streams < 1:
+            raise ValueError(f"{streams} streams")
+        self.streams = int(streams)
+        self.prefix = layer.prefix
+        self.names = dict(layer.names)
+        self.mixer = MIXERS.build(layer.mixer, **ctx)
+        self.mixer_norm = NORMS.build(layer.mixer_norm, **ctx)
+        self.weights = {mixer_name: None}
+        self.mixer_name, self.feed_forward_name = mixer_name, feed_forward_name
+        self.feed_forward = self.feed_forward_norm = None
+        if layer.feed_forward is not None:
+            if layer.feed_forward_norm is None:
+                raise ValueError("stream_mix_residual: a feed-forward needs its norm")
+            self.feed_forward = FEED_FORWARDS.build(layer.feed_forward, **ctx)
+            self.feed_forward_norm = NORMS.build(layer.feed_forward_norm, **ctx)
+            self.weights[feed_forward_name] = None
+
+    def _named(self):
+        p, n = self.prefix, self.names
+        named = [(self.mixer_norm, f"{p}.{n['mixer_norm']}"), (self.mixer, f"{p}.{n['mixer']}")]
+        if self.feed_forward is not None:
+            named += [(self.feed_forward_norm, f"{p}.{n['feed_forward_norm']}"),
+                      (self.feed_forward, f"{p}.{n['feed_forward']}")]
+        return named
+
+    def parts(self):
+        return [part for part, _ in self._named()]
+
+    def expected_tensors(self, prefix: str = "") -> Dict[str, ExpectedTensor]:
+        out: Dict[str, ExpectedTensor] = {}
+        for part, name in self._named():
+            out.update(part.expected_tensors(name))
+        S = self.streams
+        for name in self.weights:
+            out.update({f"{self.prefix}.{name}.in": ExpectedTensor((S,)),
+                        f"{self.prefix}.{name}.out": ExpectedTensor((S,)),
+                        f"{self.prefix}.{name}.mix": ExpectedTensor((S, S))})
+        return out
+
+    def load(self, prefix: str, fetch: Fetch) -> None:
+        for part, name in self._named():
+            part.load(name, fetch)
+        for name in self.weights:
+            self.weights[name] = tuple(
+                fetch(f"{self.prefix}.{name}.{what}").to(torch.float32).contiguous()
+                for what in ("in", "out", "mix"))
+
+    def cache_request(self):
+        return self.mixer.cache_request()
+
+    def first_weight(self):
+        return first_weight_of(self.mixer)
+
+    def forward(self, ctx, resid, delta, cache):
+        from ..kernels import ops
+        after_block = getattr(ctx, "reads_after_part", None)
+        ctx.residual_sink = None  # a product's epilogue has one residual to add to, not several
+        w_in, share, mix = self.weights[self.mixer_name]
+        ctx.reads_after_part = (after_block if self.feed_forward is None
+                                else first_weight_of(self.feed_forward))
+        x = self.mixer_norm.add_norm(resid.read(w_in), delta)
+        delta = ops.StreamDelta(self.mixer.forward(ctx, x, cache), mix, share)
+        if self.feed_forward is None:
+            return delta
+        w_in, share, mix = self.weights[self.feed_forward_name]
+        ctx.reads_after_part = after_block
+        x = self.feed_forward_norm.add_norm(resid.read(w_in), delta)
+        bias = None
+        if getattr(self.feed_forward, "defers_bias", False):
+            y, bias = self.feed_forward.forward(ctx, x, defer_bias=True)
+        else:
+            y = self.feed_forward.forward(ctx, x)
+        return ops.StreamDelta(y, mix, share, bias)
+
+
 def _as_float_rows(y):
     """A part's output as one float32 tensor (planes summed; 16-bit rows widened)."""
     from ..kernels import ops

@@ -2,7 +2,8 @@
 it is the reference's SwiGLU (src/models/llama/mlp.rs:49-58; SiLU is
 x / (1 + exp(-x)) in 32-bit, src/nn/activation.rs:18-27); `activation =
 "gelu_tanh"` makes it 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
-gate and up are one fused product. `dense_mlp` is the form without a gate.
+gate and up are one fused product. `clamped_glu` clamps both halves and has biases;
+`dense_mlp` is the form without a gate.
 """
 from __future__ import annotations
 
@@ -14,6 +15,7 @@ from ..kernels import ops
 from ..weights.loader import ExpectedTensor
 from .base import Fetch, Part, register_feed_forward
 from .linear import Linear, matmul_nt
+from .products import product_f32, product_planes
 
 
 @register_feed_forward("swiglu")
@@ -71,6 +73,73 @@ class SwiGLU(Part):
         return self.down.forward(hidden, out_dtype=self.out_dtype, allow_planes=True,
                                  then_reads=getattr(ctx, "reads_after_part", None),
                                  residual=getattr(ctx, "residual_sink", None))
+
+
+@register_feed_forward("clamped_glu")
+class ClampedGLU(Part):
+    """The gated feed-forward with clamped halves and (`bias`) biases on all projections:
+
+        g = min(W_gate h + b, limit);  u = clamp(W_up h + b, -limit, limit)
+        y = W_down (g * sigmoid(alpha g) * (u + shift)) + b
+
+    The biases in front of the activation join the 32-bit sums; the one behind `down` joins
+    the rows here, or (`defer_bias`) is handed out for whoever adds the rows to the stream."""
+    replay_safe = True
+    defers_bias = True
+
+    def __init__(self, hidden_size: int, intermediate_size: int, limit: float,
+                 alpha: float = 1.702, shift: float = 1.0, bias: bool = True,
+                 names=("gate", "up", "down"), suffix: str = "", bias_suffix: str = ".b", *,
+                 dtype: torch.dtype, device: torch.device):
+        if not limit > 0.0:
+            raise ValueError(f"limit {limit} must be positive")
+        self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
+        self.limit, self.alpha, self.shift = float(limit), float(alpha), float(shift)
+        self.biased = bool(bias)
+        self.dtype, self.device = dtype, device
+        self.names, self.suffix, self.bias_suffix = tuple(names), suffix, bias_suffix
+        self.gate_up = self.gate_up_bias = self.down_bias = None
+        self.down = Linear(intermediate_size, [(self.names[2], hidden_size)], dtype=dtype,
+                           device=device, suffix=suffix)
+
+    def expected_tensors(self, prefix: str) -> Dict[str, ExpectedTensor]:
+        I, H = self.intermediate_size, self.hidden_size
+        gate, up, down = self.names
+        out = {f"{prefix}.{gate}{self.suffix}": ExpectedTensor((I, H)),
+               f"{prefix}.{up}{self.suffix}": ExpectedTensor((I, H)),
+               **self.down.expected_tensors(prefix)}
+        if self.biased:
+            out.update({f"{prefix}.{name}{self.bias_suffix}": ExpectedTensor((n,))
+                        for name, n in ((gate, I), (up, I), (down, H))})
+        return out
+
+    def load(self, prefix: str, fetch: Fetch) -> None:
+        gate, up, down = self.names
+        f = lambda n: fetch(f"{prefix}.{n}")
+        # rows interleaved as in `swiglu`: a product tile holds matching gate / up pairs
+        self.gate_up = torch.stack([f(gate + self.suffix), f(up + self.suffix)], 1).reshape(
+            2 * self.intermediate_size, self.hidden_size).contiguous()
+        self.down.load(prefix, fetch)
+        if self.biased:
+            b = lambda n: f(n + self.bias_suffix).to(torch.float32)
+            self.gate_up_bias = torch.stack([b(gate), b(up)], 1).reshape(-1).contiguous()
+            self.down_bias = b(down).contiguous()
+
+    def first_weight(self):
+        return self.gate_up
+
+    def forward(self, ctx, x, defer_bias: bool = False):
+        x = ops.plain(x)
+        hidden = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
+        ops.glu_clamped(product_f32(x, self.gate_up), self.gate_up_bias, hidden, self.limit,
+                        self.alpha, self.shift)
+        y = product_planes(hidden, self.down.weight,
+                           then_reads=getattr(ctx, "reads_after_part", None))
+        if defer_bias:
+            return y, self.down_bias
+        if isinstance(y, ops.Planes):
+            y = y.sum(torch.float32)
+        return y if self.down_bias is None else ops.add_row_vector(y, self.down_bias)
 
 
 UNARY_ACTIVATIONS = ("relu2",)

@@ -1,6 +1,6 @@
 """A feed-forward of routed experts.
 
-    z = W_router h (+ b)   (32-bit). Two scoring rules:
+    z = W_router h (+ b)   (32-bit). Three scoring rules:
     "softmax_chosen": the `top` experts with the largest z are chosen (the lower index
         among equals) and weighted by the softmax over the chosen z only
     "sigmoid": s = sigmoid(z); the choice goes by c = s (+ a learnt correction per expert,
@@ -9,6 +9,10 @@
         of the `keep` best groups can be chosen; the `top` largest c are chosen and weighted
         by s itself or (`normalise`) by s / (the chosen experts' sum of s + `sum_floor`),
         times `weight_scale`
+    "softmax": as "sigmoid" with s = softmax(z) over all of the router's outputs
+    `group_best` = 1: a group's score is its largest c alone
+    `identity` > 0: the router's last outputs are identity experts behind the `experts`: they
+        take part in scores, groups and choice, have no tensors, and their output is h
     expert:  g = min(W_gate h, limit);  u = clamp(W_up h, -limit, limit)
              y = W_down (g * sigmoid(alpha g) * (u + shift))
              (limit = infinity, alpha = 1, shift = 0:  W_down (silu(g) * u))
@@ -45,24 +49,28 @@ class RoutedExperts(Part):
                  groups: int = 1, keep: int = 1, router_bias: bool = True, shared_ff: int = 0,
                  shared_name: str = "shared", choice_correction: bool = False,
                  correction_name: str = "correction", normalise: bool = False,
-                 sum_floor: float = 0.0, weight_scale: float = 1.0, *, dtype: torch.dtype,
+                 sum_floor: float = 0.0, weight_scale: float = 1.0, identity: int = 0,
+                 group_best: int = 2, *, dtype: torch.dtype,
                  device: torch.device):
-        if not 1 <= top <= min(experts, 32) or experts > 256:
-            raise ValueError(f"{top} of {experts} experts: the router takes up to 256 experts and "
+        outputs = experts + identity  # of the router
+        if not 1 <= top <= min(outputs, 32) or outputs > 256 or identity < 0:
+            raise ValueError(f"{top} of {outputs} experts: the router takes up to 256 experts and "
                              f"chooses up to 32")
         if score not in ops.MOE_SCORES:
             raise ValueError(f"scoring rule {score!r}; known: {sorted(ops.MOE_SCORES)}")
-        if groups < 1 or experts % groups or not 1 <= keep <= groups or \
-                keep * (experts // groups) < top or (groups > 1 and score != "sigmoid"):
-            raise ValueError(f"{experts} experts in {groups} groups, {keep} kept, {top} chosen "
-                             f"(groups need the sigmoid scores)")
+        own_scores = score != "softmax_chosen"
+        if groups < 1 or outputs % groups or not 1 <= keep <= groups or \
+                keep * (outputs // groups) < top or (groups > 1 and not own_scores):
+            raise ValueError(f"{outputs} experts in {groups} groups, {keep} kept, {top} chosen "
+                             f"(groups need sigmoid or softmax scores)")
+        self.outputs, self.identity, self.group_best = outputs, int(identity), int(group_best)
         self.width, self.ff, self.experts, self.top = width, ff, experts, top
         self.limit, self.alpha, self.shift = float(limit), float(alpha), float(shift)
         self.score, self.groups, self.keep = score, int(groups), int(keep)
         self.has_router_bias = bool(router_bias)
-        if (choice_correction or normalise or weight_scale != 1.0) and score != "sigmoid":
+        if (choice_correction or normalise or weight_scale != 1.0) and not own_scores:
             raise ValueError("a correction of the choice, shares of the chosen scores' sum and "
-                             "a constant on the weights need the sigmoid scores")
+                             "a constant on the weights need sigmoid or softmax scores")
         self.has_correction, self.correction_name = bool(choice_correction), correction_name
         self.normalise, self.sum_floor = bool(normalise), float(sum_floor)
         self.weight_scale = float(weight_scale)
@@ -76,11 +84,11 @@ class RoutedExperts(Part):
                                  names=("gate", "up", "down"), suffix="", activation="silu")
 
     def expected_tensors(self, prefix: str) -> Dict[str, ExpectedTensor]:
-        out = {f"{prefix}.router": ExpectedTensor((self.experts, self.width))}
+        out = {f"{prefix}.router": ExpectedTensor((self.outputs, self.width))}
         if self.has_router_bias:
-            out[f"{prefix}.router.b"] = ExpectedTensor((self.experts,))
+            out[f"{prefix}.router.b"] = ExpectedTensor((self.outputs,))
         if self.has_correction:
-            out[f"{prefix}.{self.correction_name}"] = ExpectedTensor((self.experts,))
+            out[f"{prefix}.{self.correction_name}"] = ExpectedTensor((self.outputs,))
         if self.shared is not None:
             out.update(self.shared.expected_tensors(f"{prefix}.{self.shared_name}"))
         for e in range(self.experts):
@@ -117,10 +125,13 @@ class RoutedExperts(Part):
         weights = torch.empty((T, self.top), dtype=torch.float32, device=x.device)
         rule = dict(score=self.score, groups=self.groups, keep=self.keep,
                     correction=self.correction, normalise=self.normalise,
-                    sum_floor=self.sum_floor, weight_scale=self.weight_scale)
+                    sum_floor=self.sum_floor, weight_scale=self.weight_scale,
+                    group_best=self.group_best)
+        own = ops.plain(x) if self.identity else None  # what an identity expert gives
         grouped = ops.moe_grouped_fits(self.width) and ops.moe_grouped_fits(self.ff)
         if grouped:  # the choice, and the pairs sorted by expert
-            order = ops.moe_route_sorted(z, self.router_bias, self.top, chosen, weights, **rule)
+            order = ops.moe_route_sorted(z, self.router_bias, self.top, chosen, weights,
+                                         experts=self.experts, **rule)
         else:
             ops.moe_route(z, self.router_bias, self.top, chosen, weights, **rule)
         # the shared expert's rows join the sum where the chosen experts' rows are combined
@@ -150,7 +161,7 @@ class RoutedExperts(Part):
             act = ops.moe_grouped(x, self.gate_up, order, True, self.limit, self.alpha,
                                   by_token=True, shift=self.shift)
             y = ops.moe_grouped(act, self.down, order, False)
-        return ops.moe_combine(y, order, weights, out, addend=shared)
+        return ops.moe_combine(y, order, weights, out, addend=shared, identity=own)
 
     # From this many tokens on the experts' products run on the tcgen05 products: as one
     # grouped launch a product where the sizes allow it; else, in a step that is launched

@@ -59,11 +59,15 @@ class RMSNorm(Part):
     def add_norm(self, resid: torch.Tensor, delta, out: Optional[torch.Tensor] = None):
         """resid += delta (a tensor, split-K `ops.Planes`, an `ops.ScaledDelta`, an
         `ops.PostNormed` whose norm is applied on the way, or None); returns norm(resid) in the activation dtype. A delta that a projection made
-        with this norm's `sink` comes back as an `ops.RowScaled`."""
+        with this norm's `sink` comes back as an `ops.RowScaled`. `resid` may be an
+        `ops.StreamRead` (with an `ops.StreamDelta` or None): what is normalised is then a
+        weighted sum of several streams."""
         if isinstance(delta, ops.NormPending):
             return ops.add_rmsnorm(resid, delta, self.weight, self.eps, None)
         if out is None:
             out = torch.empty(resid.shape, dtype=self.dtype, device=resid.device)
+        if isinstance(resid, ops.StreamRead):  # several streams, mixed in the same pass
+            return ops.stream_mix_norm(resid, delta, self.weight, self.eps, out)
         if isinstance(delta, ops.PostNormed):
             if delta.eps == self.eps:
                 return ops.post_norm_add(resid, delta, self.weight, self.eps, out)
