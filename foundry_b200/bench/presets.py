@@ -146,7 +146,27 @@ def _tokovik(layers, width, heads, kv_heads, dim, ff, vocab, window=1024, state=
                        for _ in range(layers)]}
 
 
+def _nemasun(layers, width, heads, kv_heads, dim, ff, vocab, window=1024, keep_first=4, streams=2,
+             experts=16, identity=4, top=2) -> Dict:
+    """A Nemasun stack of real layer sizes: attention in a window of `window` positions that
+    keeps `keep_first` tokens, with a distance table of 32 rows up to 512 positions; dense and
+    routed feed-forwards alternating (an expert and the shared expert a quarter as wide as the
+    dense one; four groups of experts, identity experts among them, of which two are kept)."""
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+             "bias_max": 512, "bias_rows": 32, "mask": {"size": window, "keep_first": keep_first}}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    routed = {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 4},
+              "router": {"experts": experts, "identity": identity, "top": top,
+                         "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Nemasun", "vocab": vocab, "width": width, "streams": streams,
+            "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": routed if i % 2 else dense}
+                       for i in range(layers)]}
+
+
 PRESETS: Dict[str, Dict] = {
+    "nemasun-1b-layers": _nemasun(6, 2048, 32, 8, 64, 8192, 32000),
+    "nemasun-3b-layers": _nemasun(6, 3072, 24, 8, 128, 8192, 32000),
     "tokovik-1b-layers": _tokovik(6, 2048, 32, 8, 64, 8192, 32000),
     "tokovik-3b-layers": _tokovik(6, 3072, 24, 8, 128, 8192, 32000),
     "kutepel-1b-layers": _kutepel(6, 2048, 32, 8, 64, 8192, 32000, 256),

@@ -103,7 +103,8 @@ class KVGroup:
         if views is None:  # the views never change: made once per entry
             block = self.storage[self.index_of[entry]]
             if self.request.row_scales:
-                rows = block[..., :PAGE * self.request.head_dim].unflatten(-1, (PAGE, -1))
+                d = self.request.head_dim
+                rows = block.as_strided((*block.shape[:2], PAGE, d), (*block.stride()[:2], d, 1))
                 views = self._views[entry] = (rows, rows)
             elif self.keys_only:
                 views = self._views[entry] = (block, block)

@@ -140,7 +140,23 @@ struct AttnParams {
   int window, keep_first, sink;
   float steep;
   const float* sink_logits;
+  // Single tokens in the form with shared rows (attn_decode_kernel's ONE): a key's factor,
+  // float32 [pages][Kh][64] with these strides; a bias by distance, float32
+  // [A][table_last + 1] or null; float32 gate rows [tokens][A * D] or null.
+  const float* key_scale;
+  long long ks_page, ks_head;
+  const float* table;
+  int table_last;
+  const float* gate;
+  long long gate_stride;
 };
+
+// A head's finished output element on its way out: times the sigmoid of its gate where there is one.
+__device__ __forceinline__ void store_head(const AttnParams& p, int token, int column, float v) {
+  if (p.gate != nullptr)
+    v = v / (1.0f + __expf(-__ldcg(p.gate + (long long)token * p.gate_stride + column)));
+  p.out[(long long)token * p.out_stride + column] = __float2bfloat16_rn(v);
+}
 
 // --------------------------------------------------------------------- prefill
 // EXT: the masked form (window with kept first tokens, distance bias, sink); pages
@@ -392,8 +408,7 @@ __device__ void merge_if_last(const AttnParams& p, int seq, int kvh, int token, 
       }
       M = Mn;
     }
-    p.out[(long long)token * p.out_stride + (long long)(kvh * G + row) * D + d] =
-        __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+    store_head(p, token, (kvh * G + row) * D + d, L > 0.f ? acc / L : 0.f);
   }
   if (threadIdx.x == 0) p.counters[seq * p.Kh + kvh] = 0;
 }
@@ -461,8 +476,7 @@ __device__ void merge_in_cluster(const AttnParams& p, const float* cO, const flo
       p.ws_o[(slot * 16 + row) * D + d] = acc;
       if (d == 0) { p.ws_ml[slot * 32 + 2 * row] = M; p.ws_ml[slot * 32 + 2 * row + 1] = L; }
     } else {
-      p.out[(long long)token * p.out_stride + (long long)(kvh * G + row) * D + d] =
-          __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+      store_head(p, token, (kvh * G + row) * D + d, L > 0.f ? acc / L : 0.f);
     }
   }
   cluster_sync_all();  // peers may have been reading this CTA's memory until here
@@ -474,7 +488,12 @@ __device__ void merge_in_cluster(const AttnParams& p, const float* cO, const flo
 // O^T = V^T P^T, half the instructions of the 16-query-row form, of whose rows
 // a grouping of 3 or 4 uses a quarter. P^T reaches the second product's operand
 // layout by a transposition inside the warp (movmatrix).
-template <int D, int ST, bool CLUSTER, bool NARROW>
+//
+// ONE: a token has one cached row a head, its value, and that row times a factor (a float32
+// beside it) is its key: one page buffer serves both products, a score is multiplied by its
+// key's factor and gains a bias by distance, and kept first tokens' pages are walked in front
+// of the window's.
+template <int D, int ST, bool CLUSTER, bool NARROW, bool ONE>
 __global__ void __launch_bounds__(THREADS)
 attn_decode_kernel(const AttnParams p) {
   constexpr int KT = D / 16, NT = D / 8;
@@ -484,7 +503,8 @@ attn_decode_kernel(const AttnParams p) {
   // else to hide that latency behind; more buffers mean fewer CTAs per SM.
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);  // [16][D]
   __nv_bfloat16* sK = sQ + 16 * D;                              // [ST][64][D]
-  __nv_bfloat16* sV = sK + ST * 64 * D;                         // [ST][64][D]
+  __nv_bfloat16* sV = ONE ? sK : sK + ST * 64 * D;              // [ST][64][D]
+  __shared__ __align__(16) float sS[ONE ? ST * 64 : 4];         // ONE: the pages' key factors
   const int seq = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
   const int G = p.A / p.Kh;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -498,9 +518,14 @@ attn_decode_kernel(const AttnParams p) {
   const int n_pages = (kv_len + FB_PAGE - 1) / FB_PAGE;
   const int lo = p.window > 0 ? max(0, kv_len - p.window) : 0;  // the token's first visible key
   const int first = lo / FB_PAGE;
-  const int per = (n_pages - first + p.splits - 1) / p.splits;  // a range: 1/splits of the pages
-  const int pg0 = first + split * per;
-  const int pg1 = min(n_pages, pg0 + per);
+  // the pages walked: those of the kept first tokens in front of the window's, then the window's;
+  // the j-th of them is page_at(j)
+  const int kept = ONE ? min((p.keep_first + FB_PAGE - 1) / FB_PAGE, first) : 0;
+  const int walked = kept + n_pages - first;
+  auto page_at = [&](int j) { return ONE && j < kept ? j : first + j - kept; };
+  const int per = (walked + p.splits - 1) / p.splits;  // a range: 1/splits of the pages
+  const int pg0 = split * per;
+  const int pg1 = min(walked, pg0 + per);
   const int fresh = max(kv_len - (p.cu_tokens[seq + 1] - token), 0) / FB_PAGE;
 
   // without clusters every CTA's result is a part of its own
@@ -538,19 +563,25 @@ attn_decode_kernel(const AttnParams p) {
       const int r = warp * 16 + id / CH, c = id % CH;
       const int so = buffer * 64 * D + Swz<D>::off(r, c * 8);
       cp_async16(smem_u32(sK + so), kbase + off + r * D + c * 8, true);
-      cp_async16(smem_u32(sV + so), vbase + off + r * D + c * 8, true);
+      if (!ONE) cp_async16(smem_u32(sV + so), vbase + off + r * D + c * 8, true);
     }
+    if (ONE && lane < 4)
+      cp_async16(smem_u32(sS + buffer * 64 + warp * 16 + lane * 4),
+                 p.key_scale + (long long)page * p.ks_page + (long long)kvh * p.ks_head +
+                     warp * 16 + lane * 4, true);
   };
   // old pages of the first ST - 1 go out now; they complete with the first group
 #pragma unroll
   for (int ahead = 0; ahead < ST - 1; ++ahead)
-    if (pg0 + ahead < min(pg1, fresh)) load_rows(ahead, pages[pg0 + ahead]);
+    if (pg0 + ahead < pg1 && page_at(pg0 + ahead) < fresh)
+      load_rows(ahead, pages[page_at(pg0 + ahead)]);
   fb_pdl_wait();
   // rows 0..G-1 of the tile are this kv head's query heads, consecutive in q
   load_tile<D>(sQ, p.q + (long long)token * p.q_stride + (long long)(kvh * G) * D, D, 16, G);
 #pragma unroll
   for (int ahead = 0; ahead < ST - 1; ++ahead) {
-    if (pg0 + ahead < pg1 && pg0 + ahead >= fresh) load_rows(ahead, pages[pg0 + ahead]);
+    if (pg0 + ahead < pg1 && page_at(pg0 + ahead) >= fresh)
+      load_rows(ahead, pages[page_at(pg0 + ahead)]);
     cp_async_commit();  // one group per page, empty when there is no page
   }
 
@@ -564,7 +595,7 @@ attn_decode_kernel(const AttnParams p) {
   // wide: rows g, g + 8; narrow: queries 2t, 2t + 1 (the same in all lanes of a t)
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 
-  int next_page = pg0 + ST - 1 < pg1 ? pages[pg0 + ST - 1] : 0;
+  int next_page = pg0 + ST - 1 < pg1 ? pages[page_at(pg0 + ST - 1)] : 0;
   for (int pg = pg0; pg < pg1; ++pg) {
     const int st = (pg - pg0) % ST;
     __syncwarp();  // every lane has read the rows that the refill overwrites
@@ -572,7 +603,21 @@ attn_decode_kernel(const AttnParams p) {
     // order, and a page-table read in front of the copies would hold up the whole
     // iteration for a trip to L2.
     const int refill_page = next_page;
-    if (pg + ST < pg1) next_page = pages[pg + ST];
+    if (pg + ST < pg1) next_page = pages[page_at(pg + ST)];
+    const int key0 = page_at(pg) * FB_PAGE + warp * 16;  // this warp's 16 keys of the page
+    // the biases of this lane's four (narrow) or eight (wide) scores, asked for before the wait
+    constexpr int NB = NARROW ? 4 : 8;
+    float by_distance[ONE ? NB : 1];
+    if constexpr (ONE) {
+#pragma unroll
+      for (int e = 0; e < NB; ++e) {
+        const int key = NARROW ? key0 + g + (e >> 1) * 8 : key0 + (e >> 2) * 8 + 2 * t + (e & 1);
+        const int query = min(NARROW ? 2 * t + (e & 1) : g + ((e >> 1) & 1) * 8, G - 1);
+        const int away = min(max(kv_len - 1 - key, 0), p.table_last);
+        by_distance[e] = p.table == nullptr ? 0.f
+            : __ldg(p.table + (size_t)(kvh * G + query) * (p.table_last + 1) + away) * LOG2E;
+      }
+    }
     // The buffer that the previous iteration finished with is refilled once this
     // page's score products have been issued: a warp issues in order, and the
     // copies' address arithmetic then runs while the tensor cores work instead of
@@ -607,8 +652,7 @@ attn_decode_kernel(const AttnParams p) {
           ldsm_x4(qf[k], smem_u32(sQ + Swz<D>::off(lane & 15, k * 16 + (lane >> 4) * 8)));
       }
     }
-    const int key0 = pg * FB_PAGE + warp * 16;  // this warp's 16 keys of the page
-    if (key0 < kv_len && key0 + 16 > lo) {
+    if (key0 < kv_len && (key0 + 16 > lo || (ONE && key0 < p.keep_first))) {
       const __nv_bfloat16* tK = sK + st * 64 * D;
       const __nv_bfloat16* tV = sV + st * 64 * D;
       if constexpr (NARROW) {
@@ -634,8 +678,10 @@ attn_decode_kernel(const AttnParams p) {
 #pragma unroll
           for (int i = 1; i < NS; ++i) v += sp[i][e];
           v *= p.scale_log2;
+          if constexpr (ONE)
+            v = fmaf(v, sS[st * 64 + warp * 16 + g + (e >> 1) * 8], by_distance[e]);
           const int key = key0 + g + (e >> 1) * 8;
-          if (key >= kv_len || key < lo) v = -INFINITY;
+          if (key >= kv_len || (key < lo && (!ONE || key >= p.keep_first))) v = -INFINITY;
           s[e] = v;
           mx[e & 1] = fmaxf(mx[e & 1], v);
         }
@@ -697,8 +743,10 @@ attn_decode_kernel(const AttnParams p) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float v = s[n][e] * p.scale_log2;
+            if constexpr (ONE)
+              v = fmaf(v, sS[st * 64 + warp * 16 + n * 8 + 2 * t + (e & 1)], by_distance[n * 4 + e]);
             const int key = key0 + n * 8 + 2 * t + (e & 1);
-            if (key >= kv_len || key < lo) v = -INFINITY;
+            if (key >= kv_len || (key < lo && (!ONE || key >= p.keep_first))) v = -INFINITY;
             s[n][e] = v;
             mx[e >> 1] = fmaxf(mx[e >> 1], v);
           }
@@ -820,8 +868,7 @@ attn_decode_kernel(const AttnParams p) {
       ws_o[row * D + d] = acc;
       if (d == 0) { ws_ml[2 * row] = M; ws_ml[2 * row + 1] = L; }
     } else {
-      p.out[(long long)token * p.out_stride + (long long)(kvh * G + row) * D + d] =
-          __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+      store_head(p, token, (kvh * G + row) * D + d, L > 0.f ? acc / L : 0.f);
     }
   }
   if (CLUSTER) merge_in_cluster<D>(p, cO, cM, cL, seq, kvh, token, G);
@@ -841,38 +888,38 @@ int launch_prefill(const AttnParams& p, int q_blocks, cudaStream_t stream) {
   return fb_check_launch("attention_prefill");
 }
 
-template <int D, int ST, bool CLUSTER, bool NARROW>
+template <int D, int ST, bool CLUSTER, bool NARROW, bool ONE>
 int launch_decode_as(const AttnParams& p, cudaStream_t stream) {
-  int bytes = (16 + 2 * ST * 64) * D * 2;
+  int bytes = (16 + (ONE ? 1 : 2) * ST * 64) * D * 2;
   // the merge reuses the page buffers: four warps' outputs, their (max, sum),
   // and the CTA's own partial result for its cluster
   const int merge = 16 * D * 2 + (4 * 16 * (D + 8) + 128 + 16 * D + 32) * 4;
   if (merge > bytes) bytes = merge;
   static bool configured[64] = {};
   if (fb_first_use_on_device(configured)) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<D, ST, CLUSTER, NARROW>,
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<D, ST, CLUSTER, NARROW, ONE>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) return fb_fail(2, "attention_decode: %s", cudaGetErrorString(e));
   }
   const dim3 grid(p.n_seqs, p.Kh, p.splits);
   if (CLUSTER)
-    fb_launch_cluster(attn_decode_kernel<D, ST, CLUSTER, NARROW>, grid, dim3(THREADS), bytes, stream,
+    fb_launch_cluster(attn_decode_kernel<D, ST, CLUSTER, NARROW, ONE>, grid, dim3(THREADS), bytes, stream,
                       (unsigned)p.cluster, p);
   else
-    fb_launch(attn_decode_kernel<D, ST, CLUSTER, NARROW>, grid, dim3(THREADS), bytes, stream, p);
+    fb_launch(attn_decode_kernel<D, ST, CLUSTER, NARROW, ONE>, grid, dim3(THREADS), bytes, stream, p);
   return fb_check_launch("attention_decode");
 }
 
 // Several CTAs per (sequence, kv head) merge inside clusters of p.cluster, and
 // what is left (all of them when p.cluster is 1) through the workspace.
-template <int D, int ST>
+template <int D, int ST, bool ONE = false>
 int launch_decode(const AttnParams& p, cudaStream_t stream) {
   const bool narrow = p.A / p.Kh <= 8;
   if (p.cluster > 1)
-    return narrow ? launch_decode_as<D, ST, true, true>(p, stream)
-                  : launch_decode_as<D, ST, true, false>(p, stream);
-  return narrow ? launch_decode_as<D, ST, false, true>(p, stream)
-                : launch_decode_as<D, ST, false, false>(p, stream);
+    return narrow ? launch_decode_as<D, ST, true, true, ONE>(p, stream)
+                  : launch_decode_as<D, ST, true, false, ONE>(p, stream);
+  return narrow ? launch_decode_as<D, ST, false, true, ONE>(p, stream)
+                : launch_decode_as<D, ST, false, false, ONE>(p, stream);
 }
 
 int check_common(const char* what, int n_seqs, int A, int Kh, int D, long long q_stride,
@@ -1014,6 +1061,60 @@ FB_API int fb_attention_decode(const void* q, long long q_stride, void* out, lon
     case 32: return launch_decode<32, 3>(p, stream);
     case 64: return launch_decode<64, 3>(p, stream);
     default: return launch_decode<128, 3>(p, stream);
+  }
+}
+
+// Single tokens over shared rows (see attn_decode_kernel's ONE): as fb_attention_decode, with
+// `rows` [n_pages, Kh, 64, D] whose heads lie row_head and whose pages page_stride elements
+// apart, their float32 factors, kept first tokens, `table` float32 [A, table_last + 1] or null,
+// and `gate` float32 rows or null.
+FB_API int fb_attention_decode_shared(const void* q, long long q_stride, void* out,
+                                      long long out_stride, const int* cu_tokens,
+                                      const int* kv_lens, const int* page_table, int max_pages,
+                                      const void* rows, long long page_stride, long long row_head,
+                                      const float* key_scale, long long ks_page, long long ks_head,
+                                      int n_seqs, int A, int Kh, int D, float scale, int window,
+                                      int keep_first, const float* table, int table_last,
+                                      const float* gate, long long gate_stride, int splits,
+                                      int cluster, float* ws_o, float* ws_ml, int* counters,
+                                      const void* next, long long next_bytes, int trigger_next,
+                                      cudaStream_t stream) {
+  FB_REQUIRE(next_bytes >= 0 && next_bytes % 16 == 0 && ((uintptr_t)next % 16) == 0,
+             "attention_decode_shared: the prefetch range must be 16-byte aligned");
+  int rc = check_common("attention_decode_shared", n_seqs, A, Kh, D, q_stride, out_stride, q, rows,
+                        rows, page_stride, row_head);
+  if (rc) return rc;
+  FB_REQUIRE(splits >= 1 && splits <= 65535 && window >= 0 && keep_first >= 0,
+             "attention_decode_shared: bad split count %d or mask", splits);
+  FB_REQUIRE(key_scale != nullptr && ((uintptr_t)key_scale % 16) == 0 && ks_page % 4 == 0 &&
+             ks_head % 4 == 0, "attention_decode_shared: the factors must keep 16-byte alignment");
+  FB_REQUIRE(table == nullptr || table_last >= 0, "attention_decode_shared: bad table");
+  if (cluster < 1) cluster = 1;
+  FB_REQUIRE(cluster <= MAX_CLUSTER && splits % cluster == 0,
+             "attention_decode_shared: clusters of %d do not divide %d splits (or exceed %d)",
+             cluster, splits, MAX_CLUSTER);
+  const int parts = splits / cluster;
+  FB_REQUIRE(parts == 1 || (ws_o && ws_ml && counters && ((uintptr_t)ws_ml % 8) == 0),
+             "attention_decode_shared: %d partial results per pair need workspaces and counters", parts);
+  AttnParams p{};
+  p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride;
+  p.out = (__nv_bfloat16*)out; p.out_stride = out_stride;
+  p.cu_tokens = cu_tokens; p.kv_lens = kv_lens; p.page_table = page_table; p.max_pages = max_pages;
+  p.k_cache = p.v_cache = (const __nv_bfloat16*)rows;
+  p.page_stride = page_stride; p.head_stride = row_head;
+  p.n_seqs = n_seqs; p.A = A; p.Kh = Kh; p.scale_log2 = scale * LOG2E;
+  p.splits = splits; p.cluster = cluster; p.parts = parts;
+  p.ws_o = ws_o; p.ws_ml = ws_ml; p.counters = counters;
+  p.next = next; p.next_bytes = next_bytes; p.trigger_next = trigger_next ? 1 : 0;
+  p.window = window; p.keep_first = window > 0 ? keep_first : 0;
+  p.key_scale = key_scale; p.ks_page = ks_page; p.ks_head = ks_head;
+  p.table = table; p.table_last = table == nullptr ? 0 : table_last;
+  p.gate = gate; p.gate_stride = gate_stride;
+  switch (D) {
+    case 16: return launch_decode<16, 4, true>(p, stream);
+    case 32: return launch_decode<32, 4, true>(p, stream);
+    case 64: return launch_decode<64, 4, true>(p, stream);
+    default: return launch_decode<128, 4, true>(p, stream);
   }
 }
 

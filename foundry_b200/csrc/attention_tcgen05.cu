@@ -40,6 +40,13 @@
 // a window, position i sees j iff 0 <= i - j < window: the block walks the pages from the one
 // that holds its first query's first key on, and masks by row at both edges.
 //
+// The form with shared rows (ONE): a token has one cached row a head, its value, and that row
+// times a factor (a float32 beside it, the row's reciprocal root mean square) is its key. One
+// ring of pages then serves both products. The softmax multiplies a score by its key's factor
+// and adds a learnt bias by distance from a table in shared memory; the window may keep the
+// first tokens, whose pages are walked in front of it; and the heads' outputs may be
+// multiplied by the sigmoid of a gate before they are rounded.
+//
 // Shared memory (96 KB at head size 128) and tensor memory (256 columns) are
 // sized so that two CTAs share an SM: the second CTA's warps fill the gaps that
 // a row's long dependent chain leaves on the schedulers and the tensor pipe.
@@ -75,7 +82,21 @@ struct FaParams {
   // term exp(sink_logits[head]) that has no key and no value: it starts the running
   // maximum and the sum.
   const float* sink_logits;
+  // The form with shared rows only. keep_first: tokens that every position sees.
+  int keep_first;
+  // float32 [A, table_pitch] or null: head a's bias in powers of two for the distance n lies at
+  // a * table_pitch + TABLE_FRONT + n, up to the distance table_last (every further one has that
+  // of table_last), with TABLE_FRONT and TABLE_BACK entries in front and behind that a page's
+  // masked keys may touch.
+  const float* table;
+  int table_last, table_pitch;
+  const float* key_scale;           // [pages][Kh][64] with these strides
+  long long ks_page, ks_head;
+  const float* gate;                // float32 rows, A * DV elements, or null
+  long long gate_stride;
 };
+constexpr int TABLE_FRONT = 192;  // a query row may lie 127 in front of a page, a key 63 into it
+constexpr int TABLE_BACK = 96;    // a warp's rows span 32, a page 64 keys
 
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
@@ -84,23 +105,32 @@ __device__ __forceinline__ float fast_exp2(float x) {
 }
 
 // KS, VS: 64-element (128-byte) blocks along a key row and a value row
-template <int KS, int VS>
+template <int KS, int VS, bool ONE>
 struct FaSmem {
   static constexpr int Q_BYTES = BQ * KS * 128;
   static constexpr int K_BYTES = FB_PAGE * KS * 128;       // one K page of one head
   static constexpr int V_BYTES = FB_PAGE * VS * 128;       // one V page of one head
-  static constexpr int USED = Q_BYTES + ST * (K_BYTES + V_BYTES) + 256;
+  static constexpr int RING = ONE ? 4 : ST;  // stages of a ring (ONE: of the only one)
+  static constexpr int V_RING = ONE ? 0 : ST;
+  static constexpr int TILES = Q_BYTES + RING * K_BYTES + V_RING * V_BYTES;
+  static constexpr int BARS = 256;
+  static constexpr int SCALES = ONE ? 4 * 64 * 4 : 0;  // a page's key factors, one copy a warp
+  static constexpr int USED = TILES + BARS + SCALES;
+  static constexpr int LIMIT = (233472 - 2 * 1024) / 2;
+  static constexpr int TABLE_ROOM = (LIMIT - USED) / 4;  // floats left for a distance table
   // never three CTAs on an SM: they would need more tensor memory than it has
-  static constexpr int BYTES = USED > 77 * 1024 ? USED : 77 * 1024;
-  static_assert(BYTES <= (233472 - 2 * 1024) / 2, "two CTAs must fit an SM");
+  static constexpr int LEAST = 77 * 1024;
+  static constexpr int BYTES = USED > LEAST ? USED : LEAST;
+  static_assert(BYTES <= LIMIT, "two CTAs must fit an SM");
 };
 
-template <int KS, int VS>
+template <int KS, int VS, bool ONE>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                        const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const FaParams p) {
-  using Smem = FaSmem<KS, VS>;
+  using Smem = FaSmem<KS, VS, ONE>;
+  constexpr int RING = Smem::RING;
   constexpr int Q_SUB = BQ * 128;              // bytes of one query sub-tile
   constexpr int KV_SUB = FB_PAGE * 128;        // bytes of one K or V sub-tile
   constexpr int TMEM_COLS = 256;               // 2 x 64 score columns + VS * 64 output columns
@@ -109,13 +139,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
   uint8_t* base = smem_raw;
   uint8_t* sQ = base;
   uint8_t* sK = sQ + Smem::Q_BYTES;                      // [ST][KS][64 keys][64]
-  uint8_t* sV = sK + ST * Smem::K_BYTES;                 // [ST][VS][64 keys][64]
-  uint64_t* bars = (uint64_t*)(sV + ST * Smem::V_BYTES);
+  uint8_t* sV = ONE ? sK : sK + ST * Smem::K_BYTES;      // [ST][VS][64 keys][64]
+  uint64_t* bars = (uint64_t*)(base + Smem::TILES);
   uint64_t* q_full = bars;
-  uint64_t* k_full = bars + 1;         // [ST]
-  uint64_t* v_full = k_full + ST;      // [ST]
-  uint64_t* k_empty = v_full + ST;     // [ST]
-  uint64_t* v_empty = k_empty + ST;    // [ST]
+  uint64_t* k_full = bars + 1;         // [RING]
+  uint64_t* v_full = k_full + RING;    // [ST]
+  uint64_t* k_empty = v_full + ST;     // [RING]
+  uint64_t* v_empty = k_empty + RING;  // [ST]
   uint64_t* s_full = v_empty + ST;     // [2]: the scores of a page are in buffer b
   uint64_t* p_full = s_full + 2;       // [2]: its probabilities have replaced them
   uint64_t* pv_done = p_full + 2;      // completes once per P.V product
@@ -123,6 +153,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
   uint32_t* tmem_slot = (uint32_t*)(o_final + 1);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
   int* s_info = (int*)(tmem_slot + 2);
+  float* s_scale = (float*)(base + Smem::TILES + Smem::BARS);  // [4 warps][64] (ONE)
+  float* s_table = s_scale + 4 * 64;                           // (ONE, where the table fits)
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -138,10 +170,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     s_info[0] = s < p.n_seqs ? s : -1;
     s_info[1] = b;
     mbar_init(q_full, 1);
-    for (int i = 0; i < ST; ++i) {
-      mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1);
-      mbar_init(&v_full[i], 1); mbar_init(&v_empty[i], 1);
-    }
+    for (int i = 0; i < RING; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
+    for (int i = 0; i < ST; ++i) { mbar_init(&v_full[i], 1); mbar_init(&v_empty[i], 1); }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&s_full[i], 1);
       mbar_init(&p_full[i], 4);  // one arrival per softmax warp
@@ -167,21 +197,28 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                  : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
+  const int head = blockIdx.x, kvh = head / (p.A / p.Kh);
+  const bool table_here = ONE && p.table != nullptr && p.table_pitch <= Smem::TABLE_ROOM;
+  if (table_here)  // (constant data: no wait for the kernel in front)
+    for (int i = threadIdx.x; i < p.table_pitch; i += THREADS)
+      s_table[i] = p.table[(size_t)head * p.table_pitch + i];
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
 
   const int row0 = s_info[1] * BQ;
-  const int head = blockIdx.x, kvh = head / (p.A / p.Kh);
   const int tok0 = p.cu_tokens[seq], q_len = p.cu_tokens[seq + 1] - tok0;
   const int kv_len = p.kv_lens[seq];
   const int pos0 = kv_len - q_len + row0;  // position of this block's first query
   const int rows_valid = min(BQ, q_len - row0);
-  // the pages the block walks; j counts from the first of them
+  // the pages the block walks: those of the kept first tokens that lie in front of the
+  // window's, then from the first row's window on; the j-th of them is page_at(j)
   const int first_page = p.window > 0 ? max(0, pos0 - p.window + 1) / FB_PAGE : 0;
-  const int n_pages = (pos0 + rows_valid - 1) / FB_PAGE + 1 - first_page;
-  const int* pages = p.page_table + (size_t)seq * p.max_pages + first_page;
+  const int kept = ONE ? min((p.keep_first + FB_PAGE - 1) / FB_PAGE, first_page) : 0;
+  const int n_pages = kept + (pos0 + rows_valid - 1) / FB_PAGE + 1 - first_page;
+  const int* pages = p.page_table + (size_t)seq * p.max_pages;
+  auto page_at = [&](int j) { return ONE && j < kept ? j : first_page + j - kept; };
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA producer
@@ -192,15 +229,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       for (int sb = 0; sb < KS; ++sb)
         tma_load_2d(sQ + sb * Q_SUB, &map_q, q_full, head * p.D + sb * 64, tok0 + row0);
       for (int j = 0; j < n_pages; ++j) {
-        const int s = j % ST;
-        const uint32_t parity = (uint32_t)((j / ST) & 1) ^ 1u;
-        const int page = pages[j];
+        const int s = j % RING;
+        const uint32_t parity = (uint32_t)((j / RING) & 1) ^ 1u;
+        const int page = pages[page_at(j)];
         if (!mbar_wait(&k_empty[s], parity, abort_flag, 11, j)) break;
         mbar_expect_tx(&k_full[s], Smem::K_BYTES);
 #pragma unroll
         for (int sb = 0; sb < KS; ++sb)
           tma_load_3d(sK + s * Smem::K_BYTES + sb * KV_SUB, &map_k, &k_full[s], sb * 64,
-                      kvh * FB_PAGE, page);
+                      ONE ? 0 : kvh * FB_PAGE, ONE ? page * p.Kh + kvh : page);
+        if (ONE) continue;
         if (!mbar_wait(&v_empty[s], parity, abort_flag, 10, j)) break;
         mbar_expect_tx(&v_full[s], Smem::V_BYTES);
 #pragma unroll
@@ -219,8 +257,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         if (j < n_pages) {
           // S[j & 1] = Q K_j^T. The buffer held P of page j - 2, whose product was
           // issued in the previous iteration: the tensor pipe runs them in order.
-          const int s = j % ST, b = j & 1;
-          ok = mbar_wait(&k_full[s], (uint32_t)((j / ST) & 1), abort_flag, 13, j);
+          const int s = j % RING, b = j & 1;
+          ok = mbar_wait(&k_full[s], (uint32_t)((j / RING) & 1), abort_flag, 13, j);
           if (!ok) break;
           tc_fence_after();
           const uint32_t q_addr = smem_u32(sQ);
@@ -232,13 +270,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
               umma(tmem_base + (uint32_t)(b * FB_PAGE), make_desc(q_addr + sb * Q_SUB + k * 32),
                    make_desc(k_addr + sb * KV_SUB + k * 32), idesc_qk, (sb | k) != 0 ? 1u : 0u);
           tc_commit(&s_full[b]);
-          tc_commit(&k_empty[s]);
+          if (!ONE) tc_commit(&k_empty[s]);
         }
         if (j >= 1) {
           // O += P_{j-1} V_{j-1}, one page behind the scores; P from tensor memory
-          const int jj = j - 1, s = jj % ST, b = jj & 1;
+          const int jj = j - 1, s = jj % (ONE ? RING : ST), b = jj & 1;
           ok = mbar_wait(&p_full[b], (uint32_t)((jj >> 1) & 1), abort_flag, 15, jj) &&
-               mbar_wait(&v_full[s], (uint32_t)((jj / ST) & 1), abort_flag, 9, jj);
+               (ONE || mbar_wait(&v_full[s], (uint32_t)((jj / ST) & 1), abort_flag, 9, jj));
           if (!ok) break;
           tc_fence_after();
           const uint32_t v_addr = smem_u32(sV + s * Smem::V_BYTES);
@@ -247,7 +285,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
             umma_a_tmem(tmem_base + O_COL, tmem_base + (uint32_t)(b * FB_PAGE + k * 8),
                         make_desc_mn(v_addr + k * 16 * 128, KV_SUB), idesc_pv,
                         (jj | k) != 0 ? 1u : 0u);
-          tc_commit(&v_empty[s]);
+          tc_commit(ONE ? &k_empty[s] : &v_empty[s]);
           tc_commit(pv_done);
           if (jj == n_pages - 1) tc_commit(o_final);
         }
@@ -263,8 +301,28 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     if (p.sink_logits != nullptr) { m_ref = p.sink_logits[head] * LOG2E; l = 1.f; }
     bool ok = true;
     fb_pdl_wait();
+    // ONE: a page's key factors go to the warp's own copy, read a page ahead
+    float* my_scale = s_scale + quarter * 64;
+    const float* ks_base = ONE ? p.key_scale + (long long)kvh * p.ks_head : nullptr;
+    float ks0 = 0.f, ks1 = 0.f;
+    if (ONE) {
+      const float* src = ks_base + (long long)pages[page_at(0)] * p.ks_page;
+      ks0 = __ldcg(src + lane);
+      ks1 = __ldcg(src + 32 + lane);
+    }
     for (int j = 0; j < n_pages && ok; ++j) {
       const int b = j & 1;
+      if (ONE) {
+        __syncwarp();  // the page before has been read by every lane
+        my_scale[lane] = ks0 * p.scale_log2;
+        my_scale[32 + lane] = ks1 * p.scale_log2;
+        __syncwarp();
+        if (j + 1 < n_pages) {
+          const float* src = ks_base + (long long)pages[page_at(j + 1)] * p.ks_page;
+          ks0 = __ldcg(src + lane);
+          ks1 = __ldcg(src + 32 + lane);
+        }
+      }
       ok = mbar_wait(&s_full[b], (uint32_t)((j >> 1) & 1), abort_flag, 16, j);
       if (!ok) break;
       tc_fence_after();
@@ -281,7 +339,46 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         }
       }
 
-      const int key0 = (first_page + j) * FB_PAGE;
+      const int key0 = page_at(j) * FB_PAGE;
+      if (ONE) {
+        // score times the key's factor, plus the bias of its distance, in powers of two
+        const float4* factor = reinterpret_cast<const float4*>(my_scale);
+        const int nearest = pos0 + quarter * 32 - (key0 + FB_PAGE - 1);  // of the warp's distances
+        if (p.table == nullptr || nearest >= p.table_last) {
+          const float flat = p.table == nullptr ? 0.f
+              : (table_here ? s_table : p.table + (size_t)head * p.table_pitch)[TABLE_FRONT + p.table_last];
+#pragma unroll
+          for (int e4 = 0; e4 < FB_PAGE / 4; ++e4) {
+            const float4 f = factor[e4];
+            sc[4 * e4] = fmaf(sc[4 * e4], f.x, flat);
+            sc[4 * e4 + 1] = fmaf(sc[4 * e4 + 1], f.y, flat);
+            sc[4 * e4 + 2] = fmaf(sc[4 * e4 + 2], f.z, flat);
+            sc[4 * e4 + 3] = fmaf(sc[4 * e4 + 3], f.w, flat);
+          }
+        } else if (table_here) {
+          // (a row without tokens keeps to the table, too: its position is one of the block's)
+          const float* at = s_table + TABLE_FRONT + (qpos - key0);
+#pragma unroll
+          for (int e4 = 0; e4 < FB_PAGE / 4; ++e4) {
+            const float4 f = factor[e4];
+            sc[4 * e4] = fmaf(sc[4 * e4], f.x, at[-4 * e4]);
+            sc[4 * e4 + 1] = fmaf(sc[4 * e4 + 1], f.y, at[-4 * e4 - 1]);
+            sc[4 * e4 + 2] = fmaf(sc[4 * e4 + 2], f.z, at[-4 * e4 - 2]);
+            sc[4 * e4 + 3] = fmaf(sc[4 * e4 + 3], f.w, at[-4 * e4 - 3]);
+          }
+        } else {  // a table longer than shared memory has room for
+          const float* at = p.table + (size_t)head * p.table_pitch + TABLE_FRONT + (qpos - key0);
+#pragma unroll
+          for (int e4 = 0; e4 < FB_PAGE / 4; ++e4) {
+            const float4 f = factor[e4];
+            sc[4 * e4] = fmaf(sc[4 * e4], f.x, __ldg(at - 4 * e4));
+            sc[4 * e4 + 1] = fmaf(sc[4 * e4 + 1], f.y, __ldg(at - 4 * e4 - 1));
+            sc[4 * e4 + 2] = fmaf(sc[4 * e4 + 2], f.z, __ldg(at - 4 * e4 - 2));
+            sc[4 * e4 + 3] = fmaf(sc[4 * e4 + 3], f.w, __ldg(at - 4 * e4 - 3));
+          }
+        }
+      }
+      const float to_log2 = ONE ? 1.0f : p.scale_log2;
       const bool diagonal = key0 + FB_PAGE - 1 > pos0 + quarter * 32;  // some key may be masked
       if (diagonal) {
 #pragma unroll
@@ -291,9 +388,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       // some key may lie behind some row's window (rows of the warp reach 31 further)
       if (p.window > 0 && key0 <= pos0 + quarter * 32 + 31 - p.window) {
         const int behind = qpos - p.window - key0;  // keys of the page up to this one are behind it
+        const int held = ONE ? p.keep_first - key0 : 0;  // keys of the page in front of this one stay
 #pragma unroll
         for (int e = 0; e < FB_PAGE; ++e)
-          if (e <= behind) sc[e] = -INFINITY;
+          if (e <= behind && (!ONE || e >= held)) sc[e] = -INFINITY;
       }
       // the row maximum of the raw scores, by four independent chains; the scale is
       // positive, so it can be applied to the maximum afterwards
@@ -305,7 +403,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         mx4[2] = fmaxf(mx4[2], sc[e + 2]);
         mx4[3] = fmaxf(mx4[3], sc[e + 3]);
       }
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * to_log2;
       const bool grow = mx > m_ref + RESCALE_STEP;  // also the first page (m_ref = -inf)
       if (__any_sync(0xffffffffu, grow)) {
         const float corr = grow ? exp2f(m_ref - mx) : 1.0f;  // 0 on the row's first page
@@ -340,8 +438,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       for (int c = 0; c < 32; ++c) {
         // 2^(s * scale - m_ref): one multiply-add and one ex2; the result is at most 2^8
         // and is rounded to bfloat16 next, so the approximate ex2 costs no accuracy
-        const float p0 = fast_exp2(fmaf(sc[2 * c], p.scale_log2, neg_ref));
-        const float p1 = fast_exp2(fmaf(sc[2 * c + 1], p.scale_log2, neg_ref));
+        const float p0 = fast_exp2(fmaf(sc[2 * c], to_log2, neg_ref));
+        const float p1 = fast_exp2(fmaf(sc[2 * c + 1], to_log2, neg_ref));
         sum4[c & 1] += p0;
         sum4[2 + (c & 1)] += p1;
         const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
@@ -370,6 +468,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
           for (int e = 0; e < 32; e += 8) {
             if (c + e >= p.DV) break;  // (whole pieces: DV is a multiple of 8)
+            if (ONE && p.gate != nullptr) {
+              const float* g = p.gate + (long long)(tok0 + row0 + row) * p.gate_stride +
+                               (long long)head * p.DV + c + e;
+              const float4 a = __ldcg(reinterpret_cast<const float4*>(g));
+              const float4 d = __ldcg(reinterpret_cast<const float4*>(g + 4));
+              const float z[8] = {a.x, a.y, a.z, a.w, d.x, d.y, d.z, d.w};
+#pragma unroll
+              for (int q = 0; q < 8; ++q)
+                r[e + q] = __float_as_uint(__uint_as_float(r[e + q]) / (1.0f + __expf(-z[q])));
+            }
             uint4 pk;
             __nv_bfloat162 h0 = __floats2bfloat162_rn(__uint_as_float(r[e]) * inv, __uint_as_float(r[e + 1]) * inv);
             __nv_bfloat162 h1 = __floats2bfloat162_rn(__uint_as_float(r[e + 2]) * inv, __uint_as_float(r[e + 3]) * inv);
@@ -431,18 +539,23 @@ int make_map(CUtensorMap* map, const void* ptr, int rank, const long long* dims,
   return 0;
 }
 
-template <int KS, int VS>
+template <int KS, int VS, bool ONE = false>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FaParams& p,
            int q_blocks, cudaStream_t stream) {
+  using Smem = FaSmem<KS, VS, ONE>;
+  int bytes = Smem::BYTES;
+  if (ONE && p.table != nullptr && p.table_pitch <= Smem::TABLE_ROOM &&
+      Smem::USED + p.table_pitch * 4 > bytes)
+    bytes = Smem::USED + p.table_pitch * 4;
   static bool configured[64] = {};
   if (fb_first_use_on_device(configured)) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<KS, VS>,
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<KS, VS, ONE>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         FaSmem<KS, VS>::BYTES);
+                                         ONE ? Smem::LIMIT : Smem::BYTES);
     if (e != cudaSuccess) return fb_fail(2, "attention_tc: %s", cudaGetErrorString(e));
   }
-  fb_launch(attn_prefill_tc_kernel<KS, VS>, dim3(p.A, q_blocks), dim3(THREADS), FaSmem<KS, VS>::BYTES,
-            stream, mq, mk, mv, p);
+  fb_launch(attn_prefill_tc_kernel<KS, VS, ONE>, dim3(p.A, q_blocks), dim3(THREADS), bytes, stream,
+            mq, mk, mv, p);
   return fb_check_launch("attention_prefill_tc");
 }
 
@@ -488,7 +601,7 @@ FB_API int fb_attention_prefill_tc(const void* q, long long q_stride, int T, voi
     rc = make_map(&mv, v_cache, 3, vdims, vstrides, box);
     if (rc) return rc;
   }
-  FaParams p;
+  FaParams p{};
   p.out = (__nv_bfloat16*)out; p.out_stride = out_stride;
   p.cu_tokens = cu_tokens; p.kv_lens = kv_lens; p.page_table = page_table;
   p.max_pages = max_pages; p.n_seqs = n_seqs; p.A = A; p.Kh = Kh;
@@ -499,6 +612,62 @@ FB_API int fb_attention_prefill_tc(const void* q, long long q_stride, int T, voi
                                : launch<1, 2>(mq, mk, mv, p, q_blocks, stream);
   return DV <= 64 ? launch<2, 1>(mq, mk, mv, p, q_blocks, stream)
                   : launch<2, 2>(mq, mk, mv, p, q_blocks, stream);
+}
+
+// The form with shared rows (see the file's notes): `rows` are one cache entry's
+// [n_pages, Kh, 64, D] with heads `row_head` elements apart and pages Kh * row_head apart,
+// `key_scale` their float32 factors. `table`: see FaParams (null: no bias). `gate`: null or
+// float32 rows of A * D elements, 16-byte aligned.
+FB_API int fb_attention_prefill_shared(const void* q, long long q_stride, int T, void* out,
+                                       long long out_stride, const int* cu_tokens,
+                                       const int* kv_lens, const int* page_table, int max_pages,
+                                       const void* rows, long long row_head,
+                                       const float* key_scale, long long ks_page,
+                                       long long ks_head, int n_pages, int n_seqs, int q_blocks,
+                                       int A, int Kh, int D, int window, int keep_first,
+                                       float scale, const float* table, int table_last,
+                                       int table_pitch, const float* gate, long long gate_stride,
+                                       cudaStream_t stream) {
+  FB_REQUIRE(D > 0 && D <= 128 && D % 8 == 0 && window >= 0 && keep_first >= 0,
+             "attention_prefill_shared: head size %d is not built (a multiple of 8 up to 128)", D);
+  FB_REQUIRE(n_seqs > 0 && A > 0 && Kh > 0 && A % Kh == 0 && T > 0 && n_pages > 0,
+             "attention_prefill_shared: bad sizes");
+  FB_REQUIRE(row_head >= (long long)FB_PAGE * D && row_head % 8 == 0 && key_scale != nullptr,
+             "attention_prefill_shared: heads %lld elements apart", row_head);
+  FB_REQUIRE(table == nullptr || (table_last >= 0 &&
+             table_pitch >= TABLE_FRONT + table_last + 1 + TABLE_BACK),
+             "attention_prefill_shared: a table of %d entries a head for distances up to %d",
+             table_pitch, table_last);
+  FB_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && ((uintptr_t)q % 16) == 0 &&
+                 ((uintptr_t)out % 16) == 0 && ((uintptr_t)rows % 16) == 0 &&
+                 ((uintptr_t)gate % 16) == 0 && gate_stride % 4 == 0,
+             "attention_prefill_shared: pointers and strides must keep 16-byte alignment");
+  if (q_blocks <= 0) return 0;
+  bind_status_mirror(stream);
+  CUtensorMap mq, mk;
+  {
+    const long long dims[2] = {(long long)A * D, T}, strides[1] = {q_stride};
+    const int box[2] = {64, BQ};
+    int rc = make_map(&mq, q, 2, dims, strides, box);
+    if (rc) return rc;
+  }
+  {
+    const int box[3] = {64, FB_PAGE, 1};
+    const long long dims[3] = {D, FB_PAGE, (long long)Kh * n_pages}, strides[2] = {D, row_head};
+    int rc = make_map(&mk, rows, 3, dims, strides, box);
+    if (rc) return rc;
+  }
+  FaParams p{};
+  p.out = (__nv_bfloat16*)out; p.out_stride = out_stride;
+  p.cu_tokens = cu_tokens; p.kv_lens = kv_lens; p.page_table = page_table;
+  p.max_pages = max_pages; p.n_seqs = n_seqs; p.A = A; p.Kh = Kh;
+  p.D = D; p.DV = D; p.window = window; p.keep_first = window > 0 ? keep_first : 0;
+  p.scale_log2 = scale * LOG2E;
+  p.table = table; p.table_last = table_last; p.table_pitch = table_pitch;
+  p.key_scale = key_scale; p.ks_page = ks_page; p.ks_head = ks_head;
+  p.gate = gate; p.gate_stride = gate_stride;
+  if (D <= 64) return launch<1, 1, true>(mq, mk, mk, p, q_blocks, stream);
+  return launch<2, 2, true>(mq, mk, mk, p, q_blocks, stream);
 }
 
 // As fb_gemm_tc_status, for the attention kernel of this file.

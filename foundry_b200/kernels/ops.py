@@ -157,6 +157,15 @@ _SIGNATURES = {
                           c_void_p, c_void_p, c_void_p, c_ll, c_ll, c_ll, c_ll, c_ll, c_ll, c_ll,
                           c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                           c_float, c_void_p, c_float, c_float, c_float, c_void_p],
+    "fb_attention_prefill_shared": [c_void_p, c_ll, c_int, c_void_p, c_ll, c_void_p, c_void_p,
+                                    c_void_p, c_int, c_void_p, c_ll, c_void_p, c_ll, c_ll, c_int,
+                                    c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                                    c_void_p, c_int, c_int, c_void_p, c_ll, c_void_p],
+    "fb_attention_decode_shared": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
+                                   c_int, c_void_p, c_ll, c_ll, c_void_p, c_ll, c_ll, c_int, c_int,
+                                   c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p,
+                                   c_ll, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_ll,
+                                   c_int, c_void_p],
     "fb_attention_prefill_masked": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
                                     c_int, c_void_p, c_void_p, c_ll, c_ll, c_int, c_int, c_int,
                                     c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_void_p,
@@ -2182,18 +2191,102 @@ def attention_sink(ctx, q: torch.Tensor, out: torch.Tensor, page_table, k_cache,
     return out
 
 
+# room around a distance table's entries for keys that a page's mask takes out
+# (TABLE_FRONT and TABLE_BACK in csrc/attention_tcgen05.cu)
+DISTANCE_FRONT, DISTANCE_BACK = 192, 96
+LOG2E = 1.4426950408889634
+
+
+class DistanceBias:
+    """A bias by distance: float32 `flat` [H, n], head h's for the distances 0 .. n - 1 (every
+    further one has the last entry's); `padded`: the same in powers of two with room on both
+    sides, as the prompt kernel reads it."""
+
+    def __init__(self, flat: torch.Tensor):
+        self.flat = flat.to(torch.float32).contiguous()
+        H, n = self.flat.shape
+        pitch = (DISTANCE_FRONT + n + DISTANCE_BACK + 3) // 4 * 4
+        self.padded = torch.zeros((H, pitch), dtype=torch.float32, device=flat.device)
+        self.padded[:, DISTANCE_FRONT:DISTANCE_FRONT + n] = self.flat * LOG2E
+        self.padded[:, DISTANCE_FRONT + n:] = self.flat[:, -1:] * LOG2E
+
+    @property
+    def last(self) -> int:
+        return self.flat.shape[1] - 1
+
+
+SHARED_ROWS_TC = _os.environ.get("FOUNDRY_B200_SHARED_ROWS_TC", "1") != "0"
+
+
 def attention_shared_rows(ctx, q: torch.Tensor, out: torch.Tensor, page_table, rows, scales, H: int,
                           G: int, dim: int, scale: float, window: int = 0, keep_first: int = 0,
-                          dist_bias: Optional[torch.Tensor] = None,
+                          dist_bias: Optional[DistanceBias] = None,
                           gate: Optional[torch.Tensor] = None,
                           then_reads: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Softmax attention whose values are its keys before their norm: a token has ONE cached
     row a head (`rows` [pages, G, PAGE, dim]), read as the value and, times its factor
     (`scales` [pages, G, PAGE], the reciprocal root mean square), as the key. Position i sees
-    j <= i where i - j < window or j < keep_first (window 0: all); `dist_bias` and `gate` as
-    in `attention_sink`."""
+    j <= i where i - j < window or j < keep_first (window 0: all); `dist_bias` by distance;
+    `gate` as in `attention_sink`. bfloat16: prompts whose head size is a multiple of 8 up to
+    128 run on tcgen05, single tokens of a size that the split-range kernel has there;
+    everything else on the CUDA cores."""
+    T = q.shape[0]
+    if (SHARED_ROWS_TC and q.dtype == torch.bfloat16 and T > 0 and dim % 8 == 0 and dim <= 128
+            and _tc_attention_ok(q, out) and (gate is None or (
+                gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0))):
+        if rows.stride(0) != G * rows.stride(1) or tuple(rows.shape[1:]) != (G, PAGE, dim) \
+                or rows.stride(2) != dim or tuple(scales.shape) != (rows.shape[0], G, PAGE):
+            raise KernelError(f"attention_shared_rows: rows {tuple(rows.shape)} strides "
+                              f"{rows.stride()}, factors {tuple(scales.shape)}")
+        if gate is not None and tuple(gate.shape) != (T, H * dim):
+            raise KernelError(f"attention_shared_rows: a gate of {tuple(gate.shape)}")
+        if dist_bias is not None and dist_bias.flat.shape[0] != H:
+            raise KernelError(f"attention_shared_rows: a bias of {dist_bias.flat.shape[0]} heads")
+        f32 = lambda t, n: 0 if t is None else _dev(t, n, torch.float32, contiguous=False)
+        step = (_dev(ctx.cu_tokens, "cu_tokens", torch.int32),
+                _dev(ctx.kv_lens, "kv_lens", torch.int32),
+                _dev(page_table, "page_table", torch.int32), page_table.shape[1])
+        head = (_dev(q, "q", torch.bfloat16, contiguous=False), _rows(q, "q"))
+        to = (_dev(out, "out", torch.bfloat16, contiguous=False), _rows(out, "out"))
+        gated = (f32(gate, "gate"), 0 if gate is None else _rows(gate, "gate"))
+        last = 0 if dist_bias is None else dist_bias.last
+        factors = (f32(scales, "scales"), *scales.stride()[:2])
+        if not ctx.is_decode:
+            if ctx.cu_tokens_host is None:  # a replayed step: the bucket's bound
+                blocks = (ctx.query_blocks_bound + 1) // 2 + ctx.n_seqs
+            else:
+                cu = ctx.cu_tokens_host
+                blocks = sum((cu[i + 1] - cu[i] + 127) // 128 for i in range(ctx.n_seqs))
+            _call("fb_attention_prefill_shared", *head, T, *to, *step, rows.data_ptr(),
+                  rows.stride(1), *factors, rows.shape[0], ctx.kv_lens.numel(), blocks, H, G, dim,
+                  int(window), int(keep_first), float(scale),
+                  f32(None if dist_bias is None else dist_bias.padded, "dist_bias"), last,
+                  0 if dist_bias is None else dist_bias.padded.shape[1], *gated, _stream())
+            return out
+        if dim in FAST_HEAD_DIMS and H // G <= 16:
+            pages = (ctx.max_kv_len + PAGE - 1) // PAGE
+            if window:
+                pages = min(pages, (window + PAGE - 2) // PAGE + 1 + (keep_first + PAGE - 1) // PAGE)
+            splits, _ = decode_plan(ctx.n_seqs * G, pages, dim,
+                                    getattr(ctx, "unequal_lengths", False) and not window)
+            n = ctx.kv_lens.numel()
+            cluster = max(c for c in range(1, DECODE_CLUSTER_MAX + 1) if splits % c == 0) \
+                if DECODE_CLUSTER else 1
+            parts = splits // cluster
+            ws = (0, 0, 0)
+            if parts > 1:
+                ws_o = torch.empty(n * G * parts * 16 * dim, dtype=torch.float32, device=q.device)
+                ws_ml = torch.empty(n * G * parts * 32, dtype=torch.float32, device=q.device)
+                ws = (ws_o.data_ptr(), ws_ml.data_ptr(), _arrival_counters(q.device, n * G).data_ptr())
+            _call("fb_attention_decode_shared", *head, *to, *step, rows.data_ptr(), rows.stride(0),
+                  rows.stride(1), *factors, n, H, G, dim, float(scale), int(window),
+                  int(keep_first), f32(None if dist_bias is None else dist_bias.flat, "dist_bias"),
+                  last, *gated, splits, cluster, *ws, *_prefetch_range(then_reads),
+                  1 if n > SKINNY_ROWS else 0, _stream())
+            return out
     return attention_sink(ctx, q, out, page_table, rows, rows, H, G, dim, dim, scale, window=window,
-                          keep_first=keep_first, values_in_keys=True, dist_bias=dist_bias,
+                          keep_first=keep_first, values_in_keys=True,
+                          dist_bias=None if dist_bias is None else dist_bias.flat,
                           key_scales=scales, gate=gate)
 
 

@@ -19,7 +19,9 @@ bias is one read. Every constant is a parameter. Tensor names under the mixer's 
 `q k g o`, `q.norm k.norm`, `rel`.
 
 The cache keeps every row of a sequence (kept tokens stay readable for ever); the kernels
-walk the kept prefix and the window only.
+walk the kept prefix and the window only. In bfloat16 prompts run on tcgen05 (one ring of
+pages for both products, the table in shared memory, the gate in the epilogue) and single
+tokens on the split-range tensor-core kernel; float32 and other sizes on the CUDA cores.
 """
 from __future__ import annotations
 
@@ -93,7 +95,7 @@ class SharedRowAttention(Part):
                         * fetch(f"{prefix}.k.norm").to(torch.float32)).contiguous()
         table = fetch(f"{prefix}.rel").to(torch.float32)
         rows = torch.tensor(self.buckets, dtype=torch.long, device=table.device)
-        self.dist_bias = table[rows].t().contiguous()  # [H, bias_max + 1]
+        self.dist_bias = ops.DistanceBias(table[rows].t())  # by distance, 0 .. bias_max
 
     def cache_request(self) -> KVRequest:
         return KVRequest(self.kv_heads, self.dim, None, 0, row_scales=True)

@@ -159,6 +159,44 @@ def test_attention_in_two_cuttings(sizes, dtype):
             assert rel_error(g, w) < bound(dtype), (sizes, cuts)
 
 
+@pytest.mark.parametrize("last", [33, 120, 2000, 9000])
+@pytest.mark.parametrize("mask", [(37, 0), (64, 64), (150, 5), (300, 130), (1000, 1), (None, 0)])
+@pytest.mark.parametrize("sizes", [(64, 4, 2), (128, 2, 1), (96, 3, 1), (40, 2, 2)])
+def test_prompts_and_single_tokens_on_the_tensor_cores(sizes, mask, last):
+    """bfloat16 steps on the tensor cores against the CUDA-core kernel on the same rows:
+    windows that end inside a block of queries and inside a page, kept tokens of less and more
+    than a page, distance tables that fit shared memory and one that does not, portions that
+    begin in the middle of a page; and the kernels counted, so that nothing stands in."""
+    from foundry_b200.kernels import ops
+    d, heads, kv_heads = sizes
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": d, "vdim": d, "scale": d ** -0.5,
+         "bias_max": last}
+    if mask[0]:
+        m["mask"] = {"size": mask[0], "keep_first": mask[1]}
+    W, eps = 64, 1e-5
+    weights = tiny.random_weights(tiny.mixer_shapes("a", m, W, 32), seed=d)
+    part = mixer_part(m, W, eps, 32, weights, torch.bfloat16)
+    cache = new_cache(part, 2048, 3, torch.bfloat16)
+    torch.manual_seed(d)
+    xs = [torch.randn(n, W).to(torch.bfloat16).float() for n in (533, 70, 129)]
+    results = {}
+    for tc in (True, False):
+        ops.SHARED_ROWS_TC = tc
+        try:
+            for cuts in ([[533], [70], [129]], [[100, 133, 2, 297, 1], [5, 63, 1, 1], [64, 65]],
+                         [[520] + [1] * 13, [60] + [1] * 10, [116] + [1] * 13]):
+                got, counts = counted(lambda: run_mixer(part, cache, xs, cuts, torch.bfloat16))
+                assert (counts.get("attention_prefill_shared", 0) > 0) == tc, counts
+                assert (counts.get("attention_decode_shared", 0) > 0) == (
+                    tc and d in ops.FAST_HEAD_DIMS and len(cuts[0]) > 1), counts
+                results[tc, len(cuts[0])] = got
+        finally:
+            ops.SHARED_ROWS_TC = True
+    for cut in (1, 5, 14):
+        for g, w in zip(results[True, cut], results[False, cut]):
+            assert rel_error(g, w) < 0.75 * bound(torch.bfloat16), cut
+
+
 def crafted_attention(W, d, window, kept, heads, kv_heads):
     """An attention made so that a query that carries input 1 matches only a key that carries
     input 2: that score is about 20, every other key's about +-1. Keys are values, so what
