@@ -141,12 +141,12 @@ struct AttnParams {
   float steep;
   const float* sink_logits;
   // Single tokens in the form with shared rows (attn_decode_kernel's ONE): a key's factor,
-  // float32 [pages][Kh][64] with these strides; a bias by distance, float32
-  // [A][table_last + 1] or null; float32 gate rows [tokens][A * D] or null.
+  // float32 [pages][Kh][64] with these strides; a bias by distance in powers of two, float32
+  // [A][table_pitch], of which distances 0 .. table_last are read, or null; float32 gate rows [tokens][A * D] or null.
   const float* key_scale;
   long long ks_page, ks_head;
   const float* table;
-  int table_last;
+  int table_last, table_pitch;
   const float* gate;
   long long gate_stride;
 };
@@ -615,7 +615,7 @@ attn_decode_kernel(const AttnParams p) {
         const int query = min(NARROW ? 2 * t + (e & 1) : g + ((e >> 1) & 1) * 8, G - 1);
         const int away = min(max(kv_len - 1 - key, 0), p.table_last);
         by_distance[e] = p.table == nullptr ? 0.f
-            : __ldg(p.table + (size_t)(kvh * G + query) * (p.table_last + 1) + away) * LOG2E;
+            : __ldg(p.table + (size_t)(kvh * G + query) * p.table_pitch + away);
       }
     }
     // The buffer that the previous iteration finished with is refilled once this
@@ -1066,7 +1066,7 @@ FB_API int fb_attention_decode(const void* q, long long q_stride, void* out, lon
 
 // Single tokens over shared rows (see attn_decode_kernel's ONE): as fb_attention_decode, with
 // `rows` [n_pages, Kh, 64, D] whose heads lie row_head and whose pages page_stride elements
-// apart, their float32 factors, kept first tokens, `table` float32 [A, table_last + 1] or null,
+// apart, their float32 factors, kept first tokens, `table` as in AttnParams or null,
 // and `gate` float32 rows or null.
 FB_API int fb_attention_decode_shared(const void* q, long long q_stride, void* out,
                                       long long out_stride, const int* cu_tokens,
@@ -1075,7 +1075,7 @@ FB_API int fb_attention_decode_shared(const void* q, long long q_stride, void* o
                                       const float* key_scale, long long ks_page, long long ks_head,
                                       int n_seqs, int A, int Kh, int D, float scale, int window,
                                       int keep_first, const float* table, int table_last,
-                                      const float* gate, long long gate_stride, int splits,
+                                      int table_pitch, const float* gate, long long gate_stride, int splits,
                                       int cluster, float* ws_o, float* ws_ml, int* counters,
                                       const void* next, long long next_bytes, int trigger_next,
                                       cudaStream_t stream) {
@@ -1088,7 +1088,8 @@ FB_API int fb_attention_decode_shared(const void* q, long long q_stride, void* o
              "attention_decode_shared: bad split count %d or mask", splits);
   FB_REQUIRE(key_scale != nullptr && ((uintptr_t)key_scale % 16) == 0 && ks_page % 4 == 0 &&
              ks_head % 4 == 0, "attention_decode_shared: the factors must keep 16-byte alignment");
-  FB_REQUIRE(table == nullptr || table_last >= 0, "attention_decode_shared: bad table");
+  FB_REQUIRE(table == nullptr || (table_last >= 0 && table_pitch > table_last),
+             "attention_decode_shared: bad table");
   if (cluster < 1) cluster = 1;
   FB_REQUIRE(cluster <= MAX_CLUSTER && splits % cluster == 0,
              "attention_decode_shared: clusters of %d do not divide %d splits (or exceed %d)",
@@ -1108,7 +1109,7 @@ FB_API int fb_attention_decode_shared(const void* q, long long q_stride, void* o
   p.next = next; p.next_bytes = next_bytes; p.trigger_next = trigger_next ? 1 : 0;
   p.window = window; p.keep_first = window > 0 ? keep_first : 0;
   p.key_scale = key_scale; p.ks_page = ks_page; p.ks_head = ks_head;
-  p.table = table; p.table_last = table == nullptr ? 0 : table_last;
+  p.table = table; p.table_last = table == nullptr ? 0 : table_last; p.table_pitch = table_pitch;
   p.gate = gate; p.gate_stride = gate_stride;
   switch (D) {
     case 16: return launch_decode<16, 4, true>(p, stream);

@@ -310,6 +310,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       ks0 = __ldcg(src + lane);
       ks1 = __ldcg(src + 32 + lane);
     }
+    // (a warp issues in order: the page number behind the next factors is read a page earlier)
+    int page_ahead = ONE && n_pages > 1 ? pages[page_at(1)] : 0;
     for (int j = 0; j < n_pages && ok; ++j) {
       const int b = j & 1;
       if (ONE) {
@@ -318,9 +320,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         my_scale[32 + lane] = ks1 * p.scale_log2;
         __syncwarp();
         if (j + 1 < n_pages) {
-          const float* src = ks_base + (long long)pages[page_at(j + 1)] * p.ks_page;
+          const float* src = ks_base + (long long)page_ahead * p.ks_page;
           ks0 = __ldcg(src + lane);
           ks1 = __ldcg(src + 32 + lane);
+          if (j + 2 < n_pages) page_ahead = pages[page_at(j + 2)];
         }
       }
       ok = mbar_wait(&s_full[b], (uint32_t)((j >> 1) & 1), abort_flag, 16, j);

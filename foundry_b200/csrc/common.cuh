@@ -187,6 +187,17 @@ __device__ __forceinline__ float fb_glu_act(float g, int act) {
   return g / (1.0f + __expf(-z));
 }
 
+// A gated feed-forward with clamped halves: g = min(gate + b, limit), u = clamp(up + b, -limit,
+// limit), g * sigmoid(alpha g) * (u + shift); `bias` (float32, a weight row each) or null.
+struct FbGluClamp {
+  float limit, alpha, shift;
+  const float* bias;
+};
+__device__ __forceinline__ float fb_glu_clamped(const FbGluClamp& r, float gate, float up) {
+  const float g = fminf(gate, r.limit), u = fminf(fmaxf(up, -r.limit), r.limit);
+  return g / (1.0f + __expf(-r.alpha * g)) * (u + r.shift);
+}
+
 __device__ __forceinline__ float fb_warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -92,6 +92,7 @@ struct RowsParams {
   int out_f32;
   int epilogue;
   int glu_act;          // epilogue 1: the gate's activation (0 SiLU, 1 GELU in its tanh form)
+  FbGluClamp clamp;     // epilogue 4: as 1 with clamped halves and biases by weight row
   int vector_ok;        // the epilogue's rows are aligned for 16- and 8-byte accesses
   RowsScale scale;
   RowsSink sink;
@@ -312,6 +313,11 @@ gemm_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
       if (rotated) { freq[0] = rw.inv_freq[el >> 1]; freq[1] = rw.inv_freq[(el >> 1) + 1]; }
     }
     float gamma[4] = {0.f, 0.f, 0.f, 0.f};
+    float pair_bias[4] = {0.f, 0.f, 0.f, 0.f};
+    if (epi == 4 && p.clamp.bias != nullptr) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q) if (q < live) pair_bias[q] = __ldg(p.clamp.bias + f0 + q);
+    }
     if (epi == 2) {
 #pragma unroll
       for (int q = 0; q < 4; ++q) if (q < live) gamma[q] = p.sink.gamma[f0 + q];
@@ -400,11 +406,15 @@ gemm_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
               for (int q = 0; q < 4; ++q) if (q < live) dst[q] = __float2bfloat16_rn(val[q]);
             }
           }
-        } else if (epi == 1) {
+        } else if (epi == 1 || epi == 4) {
           // (gate, up) pairs: two results per lane
           __nv_bfloat16* dst = (__nv_bfloat16*)p.out + (long long)j * p.ldo + (f0 >> 1);
-          const float h0 = fb_glu_act(val[0], p.glu_act) * val[1];
-          const float h1 = fb_glu_act(val[2], p.glu_act) * val[3];
+          const float h0 = epi == 4
+              ? fb_glu_clamped(p.clamp, val[0] + pair_bias[0], val[1] + pair_bias[1])
+              : fb_glu_act(val[0], p.glu_act) * val[1];
+          const float h1 = epi == 4
+              ? fb_glu_clamped(p.clamp, val[2] + pair_bias[2], val[3] + pair_bias[3])
+              : fb_glu_act(val[2], p.glu_act) * val[3];
           if (vec) {
             const __nv_bfloat162 pk = __floats2bfloat162_rn(h0, h1);
             *reinterpret_cast<__nv_bfloat162*>(dst) = pk;
@@ -513,6 +523,7 @@ int launch_rows(const CUtensorMap& mw, const CUtensorMap& mx, const RowsParams& 
     case 0: return launch_rows_as<NB, 0>(mw, mx, p, tiles, stream);
     case 1: return launch_rows_as<NB, 1>(mw, mx, p, tiles, stream);
     case 2: return launch_rows_as<NB, 2>(mw, mx, p, tiles, stream);
+    case 4: return launch_rows_as<NB, 4>(mw, mx, p, tiles, stream);
     default: return launch_rows_as<NB, 3>(mw, mx, p, tiles, stream);
   }
 }
@@ -552,6 +563,7 @@ FB_API int fb_gemm_rows(const void* x, long long ldx, int M, const void* w, long
                         int max_pages, const float* inv_freq, int rotary_dim, void* q_out,
                         long long q_stride, void* k_cache, void* v_cache, long long page_stride,
                         long long head_stride, int ring_pages, int A, int Kh, int D, int splits,
+                        float glu_limit, float glu_alpha, float glu_shift, const float* glu_bias,
                         cudaStream_t stream) {
   FB_REQUIRE(M > 0 && M <= 256 && N > 0 && K > 0, "gemm_rows: bad sizes %d x %d x %d", M, N, K);
   FB_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && ((uintptr_t)x % 16) == 0 &&
@@ -561,9 +573,15 @@ FB_API int fb_gemm_rows(const void* x, long long ldx, int M, const void* w, long
   // epilogue 4: as 1 with the tanh form of GELU on the gate
   const int glu_act = epilogue == 4 ? 1 : 0;
   if (epilogue == 4) epilogue = 1;
-  FB_REQUIRE(epilogue >= 0 && epilogue <= 3, "gemm_rows: unknown epilogue %d", epilogue);
+  FB_REQUIRE((epilogue >= 0 && epilogue <= 3) || epilogue == 6, "gemm_rows: unknown epilogue %d",
+             epilogue);
   RowsParams p{};
   p.glu_act = glu_act;
+  if (epilogue == 6) {  // as 1 with clamped halves and biases (glu_*; glu_bias null: none)
+    FB_REQUIRE(glu_limit > 0.f, "gemm_rows: the clamped epilogue needs a positive limit");
+    epilogue = 4;
+    p.clamp = FbGluClamp{glu_limit, glu_alpha, glu_shift, glu_bias};
+  }
   p.M = M; p.N = N; p.K = K;
   const int tiles = (N + BM - 1) / BM;
   p.kblocks = (K + BK - 1) / BK;
@@ -577,7 +595,7 @@ FB_API int fb_gemm_rows(const void* x, long long ldx, int M, const void* w, long
   p.scale = RowsScale{scale_ss, scale_count, scale_stride,
                       scale_dim > 0 ? 1.0f / (float)scale_dim : 0.f, scale_eps};
   const int NB = M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
-  if (epilogue <= 1) {
+  if (epilogue <= 1 || epilogue == 4) {
     FB_REQUIRE(out != nullptr && (epilogue == 0 || (!out_f32 && N % 2 == 0)),
                "gemm_rows: the SiLU-mul epilogue writes bfloat16 pairs");
     p.vector_ok = ldo % 4 == 0 && ((uintptr_t)out % 16) == 0;

@@ -129,13 +129,15 @@ struct SecondProduct {
 struct NoSecond {};
 template <bool PAIR> struct PairArg { using type = NoSecond; };
 template <> struct PairArg<true> { using type = SecondProduct; };
-template <bool SINK> struct SinkArg { using type = NoSink; };
-template <> struct SinkArg<true> { using type = ResidualSink; };
 // what a kernel instance ends with
 constexpr int MODE_PLAIN = 0;  // store, or SiLU(gate) * up
 constexpr int MODE_ROPE = 1;   // rotate and write queries, keys, values
 constexpr int MODE_SINK = 2;   // add into the residual rows in front of a norm
 constexpr int MODE_PAIR = 3;   // store; the grid holds two products
+constexpr int MODE_CLAMP = 4;  // (gate, up) pairs with clamped halves and biases
+template <int MODE> struct EndArg { using type = NoSink; };
+template <> struct EndArg<MODE_SINK> { using type = ResidualSink; };
+template <> struct EndArg<MODE_CLAMP> { using type = FbGluClamp; };
 
 // NT: token tiles of 8 (1 or 2). WARPS: warps per CTA, each with a K range.
 // UNROLL: chunks whose loads are in flight together.
@@ -155,7 +157,7 @@ gemm_skinny_kernel(const __nv_bfloat16* x, long long ldx,
                    int late_trigger, int early_from,
                    const typename RopeArg<MODE == MODE_ROPE>::type rw,
                    const RowScale scale,
-                   const typename SinkArg<MODE == MODE_SINK>::type sink,
+                   const typename EndArg<MODE>::type sink,
                    const typename PairArg<MODE == MODE_PAIR>::type second) {
   constexpr bool ROPE = MODE == MODE_ROPE, SINK = MODE == MODE_SINK;
   __shared__ float red[WARPS][16][8 * NT + 1];
@@ -457,6 +459,22 @@ gemm_skinny_kernel(const __nv_bfloat16* x, long long ldx,
         if (row == 0 && tok < T) sink.ss_out[(size_t)blockIdx.x * sink.ss_stride + tok] = sq;
       }
     }
+  } else if constexpr (MODE == MODE_CLAMP) {
+    for (int idx = threadIdx.x; idx < 8 * T; idx += WARPS * 32) {
+      const int p = idx & 7, tok = idx >> 3;
+      const int row = n0 + 2 * p;
+      if (row + 1 >= N) continue;
+      float gate = 0.f, up = 0.f, b0 = 0.f, b1 = 0.f;
+      if (sink.bias != nullptr) { b0 = __ldg(sink.bias + row); b1 = __ldg(sink.bias + row + 1); }
+#pragma unroll
+      for (int wi = 0; wi < WARPS; ++wi) {
+        gate += red[wi][2 * p][tok];
+        up += red[wi][2 * p + 1][tok];
+      }
+      const float rs = row_scale(tok);
+      out_h[(size_t)tok * ldo + (row >> 1)] =
+          __float2bfloat16_rn(fb_glu_clamped(sink, gate * rs + b0, up * rs + b1));
+    }
   } else {
     if (epilogue == 0 || epilogue == 5) {
       for (int idx = threadIdx.x; idx < 16 * T; idx += WARPS * 32) {
@@ -511,14 +529,14 @@ int launch_skinny(const void* x, long long ldx, const void* w, long long ldw, vo
                   long long next_bytes, int ksplit, long long plane_stride, int warps,
                   int late_trigger, const RopeWrite& rw, const RowScale& scale,
                   const ResidualSink& sink, cudaStream_t stream,
-                  SecondProduct second = SecondProduct{}) {
+                  SecondProduct second = SecondProduct{}, const FbGluClamp& clamp = FbGluClamp{}) {
   FB_REQUIRE(next_bytes >= 0 && next_bytes % 16 == 0 && ((uintptr_t)next % 16) == 0,
              "gemm_skinny: the prefetch range must be 16-byte aligned and a multiple of 16 bytes");
   FB_REQUIRE(T > 0 && T <= 16 && N > 0 && K > 0, "gemm_skinny: bad sizes T=%d N=%d K=%d", T, N, K);
   FB_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && ((uintptr_t)x % 16) == 0 &&
                  ((uintptr_t)w % 16) == 0,
              "gemm_skinny: K, the row strides and the pointers must keep 16-byte alignment");
-  FB_REQUIRE((epilogue != 1 && epilogue != 4) || (!out_f32 && N % 2 == 0),
+  FB_REQUIRE((epilogue != 1 && epilogue != 4 && epilogue != 6) || (!out_f32 && N % 2 == 0),
              "gemm_skinny: the SiLU-mul epilogue needs a bf16 output and an even row count");
   FB_REQUIRE(ksplit >= 1 && ksplit <= 64 && (ksplit == 1 || (out_f32 && epilogue == 0 &&
                                                              plane_stride >= (long long)T * ldo)),
@@ -562,6 +580,7 @@ int launch_skinny(const void* x, long long ldx, const void* w, long long ldw, vo
   do {                                                                           \
     if (epilogue == 2) FB_SKINNY_R(NT, W, U, MODE_ROPE, rw, NoSink{}, NoSecond{});            \
     else if (epilogue == 3) FB_SKINNY_R(NT, W, U, MODE_SINK, NoRope{}, sink, NoSecond{});     \
+    else if (epilogue == 6) FB_SKINNY_R(NT, W, U, MODE_CLAMP, NoRope{}, clamp, NoSecond{});   \
     else if (second.w != nullptr) FB_SKINNY_R(NT, W, U, MODE_PAIR, NoRope{}, NoSink{}, second); \
     else FB_SKINNY_R(NT, W, U, MODE_PLAIN, NoRope{}, NoSink{}, NoSecond{});                   \
   } while (0)
@@ -603,15 +622,19 @@ FB_API int fb_gemm_skinny(const void* x, long long ldx, const void* w, long long
                           const void* next, long long next_bytes, int ksplit,
                           long long plane_stride, int warps, const float* scale_ss,
                           int scale_count, int scale_stride, int scale_dim, float scale_eps,
+                          float glu_limit, float glu_alpha, float glu_shift, const float* glu_bias,
                           cudaStream_t stream) {
   // epilogue 4: as 1 with the tanh form of GELU on the gate
   // epilogue 5: as 0 with out = max(out, 0)^2
-  FB_REQUIRE(epilogue == 0 || epilogue == 1 || epilogue == 4 || epilogue == 5,
+  // epilogue 6: as 1 with clamped halves and biases (glu_*; glu_bias null: none)
+  FB_REQUIRE(epilogue == 0 || epilogue == 1 || (epilogue >= 4 && epilogue <= 6),
              "gemm_skinny: epilogue %d", epilogue);
+  FB_REQUIRE(epilogue != 6 || glu_limit > 0.f, "gemm_skinny: the clamped epilogue needs a positive limit");
   const RowScale scale{scale_ss, scale_count, scale_stride,
                        scale_dim > 0 ? 1.0f / (float)scale_dim : 0.f, scale_eps};
   return launch_skinny(x, ldx, w, ldw, out, ldo, out_f32, T, N, K, epilogue, next, next_bytes,
-                       ksplit, plane_stride, warps, 1, RopeWrite{}, scale, ResidualSink{}, stream);
+                       ksplit, plane_stride, warps, 1, RopeWrite{}, scale, ResidualSink{}, stream,
+                       SecondProduct{}, FbGluClamp{glu_limit, glu_alpha, glu_shift, glu_bias});
 }
 
 // Two products of the same T tokens in one launch, float32 out: out1 = x1 w1^T ([T, N1]) and

@@ -991,7 +991,8 @@ FB_API int fb_gemm_tc(const void* a, long long lda, int rows_a, const void* b, l
                       int share_min_kblocks, const float* scale_ss, int scale_count,
                       int scale_stride, int scale_dim, float scale_eps, float* resid,
                       long long ldr, const float* gamma, void* xg, long long ldxg, float* ss_out,
-                      int ss_stride, cudaStream_t stream) {
+                      int ss_stride, float glu_limit, float glu_alpha, float glu_shift,
+                      const float* glu_bias, cudaStream_t stream) {
   FB_REQUIRE(rows_a > 0 && rows_b > 0 && K > 0, "gemm_tc: bad sizes %d x %d x %d", rows_a, rows_b, K);
   FB_REQUIRE(K % 8 == 0 && lda % 8 == 0 && ldb % 8 == 0,
              "gemm_tc: K and the row strides must be multiples of 8 elements (16 bytes), got K=%d "
@@ -1000,8 +1001,11 @@ FB_API int fb_gemm_tc(const void* a, long long lda, int rows_a, const void* b, l
              "gemm_tc: operands must start on 16-byte boundaries");
   FB_REQUIRE(splits >= 1 && (splits == 1 || out_f32), "gemm_tc: split-K needs a float32 output");
   // epilogue 4: as 1 with the tanh form of GELU on the gate
-  const int glu_act = epilogue == 4 ? 1 : 0;
-  if (epilogue == 4) epilogue = 1;
+  // epilogue 6: as 1 with clamped halves and biases (glu_*; glu_bias null: none)
+  const int glu_act = epilogue == 4 ? 1 : epilogue == 6 ? 2 : 0;
+  if (epilogue == 4 || epilogue == 6) epilogue = 1;
+  FB_REQUIRE(glu_act != 2 || (glu_limit > 0.f && ((uintptr_t)glu_bias % 16) == 0),
+             "gemm_tc: the clamped epilogue needs a positive limit and aligned biases");
   FB_REQUIRE(epilogue == 0 || epilogue == 2 ||
                  (epilogue == 1 && splits == 1 && !out_f32 && (stride_a == 1 || stride_b == 1)),
              "gemm_tc: the SiLU-mul epilogue needs one split, a bf16 output and features on a "
@@ -1020,6 +1024,7 @@ FB_API int fb_gemm_tc(const void* a, long long lda, int rows_a, const void* b, l
   p.kblocks_per_split = (total_kb + splits - 1) / splits;
   p.stride_a = stride_a; p.stride_b = stride_b; p.split_stride = split_stride;
   p.out = out; p.out_f32 = out_f32; p.epilogue = epilogue; p.glu_act = glu_act;
+  p.clamp = FbGluClamp{glu_limit, glu_alpha, glu_shift, glu_bias};
   p.constant_operand = constant_operand;
   p.full_tiles = 0; p.tail_splits = 1; p.tail_kblocks = total_kb; p.partial = nullptr;
   p.tail_counters = nullptr;

@@ -56,7 +56,9 @@ struct FbGemmParams {
   void* out;
   int out_f32;                // 1: float32 output, 0: bfloat16
   int constant_operand;       // 1: A holds constants (weights), 2: B does, 0: neither
-  int glu_act;                // epilogue 1: the gate's activation (0 SiLU, 1 GELU in its tanh form)
+  int glu_act;                // epilogue 1: the gate's activation (0 SiLU, 1 GELU in its tanh form,
+                              // 2: `clamp`, with biases by weight row)
+  FbGluClamp clamp;
   int epilogue;               // 0: store D; 1: act(gate) * up over interleaved feature pairs;
                               // 2: residual add in front of a norm (`rows`)
                               // 3: rotation and cache write of a q/k/v projection (`rope`)
@@ -84,6 +86,44 @@ constexpr int UMMA_K = 16;         // K of one tcgen05.mma for 16-bit inputs
 constexpr int THREADS = 192;       // 6 warps
 using GemmParams = FbGemmParams;
 
+// Epilogue 1 with clamped halves, feature pairs in this thread's registers (`base`: where the
+// first result goes).
+template <int CHUNK>
+__device__ __forceinline__ void store_clamped(const GemmParams& p, const float (&v)[CHUNK],
+                                              long long base, long long j0, __nv_bfloat16* out_h) {
+  const bool whole = j0 + CHUNK <= p.rows_b && (base % 8) == 0;
+#pragma unroll
+  for (int e = 0; e < CHUNK; e += 16) {  // 8 results = 16 bytes per store
+    float r8[8];
+#pragma unroll
+    for (int q = 0; q < 8; q += 2) {
+      float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (p.clamp.bias != nullptr && j0 + e + 2 * q + 3 < p.rows_b)
+        b = __ldg(reinterpret_cast<const float4*>(p.clamp.bias + j0 + e + 2 * q));
+      else if (p.clamp.bias != nullptr && j0 + e + 2 * q + 1 < p.rows_b)
+        b = make_float4(__ldg(p.clamp.bias + j0 + e + 2 * q), __ldg(p.clamp.bias + j0 + e + 2 * q + 1), 0.f, 0.f);
+      r8[q] = fb_glu_clamped(p.clamp, v[e + 2 * q] + b.x, v[e + 2 * q + 1] + b.y);
+      r8[q + 1] = fb_glu_clamped(p.clamp, v[e + 2 * q + 2] + b.z, v[e + 2 * q + 3] + b.w);
+    }
+    if (whole) {
+      uint4 pk;
+      __nv_bfloat162 h0 = __floats2bfloat162_rn(r8[0], r8[1]);
+      __nv_bfloat162 h1 = __floats2bfloat162_rn(r8[2], r8[3]);
+      __nv_bfloat162 h2 = __floats2bfloat162_rn(r8[4], r8[5]);
+      __nv_bfloat162 h3 = __floats2bfloat162_rn(r8[6], r8[7]);
+      pk.x = *reinterpret_cast<uint32_t*>(&h0);
+      pk.y = *reinterpret_cast<uint32_t*>(&h1);
+      pk.z = *reinterpret_cast<uint32_t*>(&h2);
+      pk.w = *reinterpret_cast<uint32_t*>(&h3);
+      *reinterpret_cast<uint4*>(out_h + base + (e >> 1)) = pk;
+    } else {
+#pragma unroll
+      for (int q = 0; q < 8; ++q)
+        if (j0 + e + 2 * q + 1 < p.rows_b) out_h[base + (e >> 1) + q] = __float2bfloat16_rn(r8[q]);
+    }
+  }
+}
+
 // Stores CHUNK consecutive accumulator columns (j0 .. j0 + CHUNK) of row
 // i_global, in the layout and with the epilogue the parameters name.
 template <int CHUNK>
@@ -97,7 +137,9 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&v
       // features run along j: pairs sit in this thread's registers
       if (i_global < p.rows_a) {
         const long long base = i_global * p.stride_a + (j0 >> 1);
-        if (j0 + CHUNK <= p.rows_b && (base % 8) == 0) {
+        if (p.glu_act == 2) {
+          store_clamped<CHUNK>(p, v, base, j0, out_h);
+        } else if (j0 + CHUNK <= p.rows_b && (base % 8) == 0) {
 #pragma unroll
           for (int e = 0; e < CHUNK; e += 16) {  // 8 results = 16 bytes per store
             float r8[8];
@@ -135,8 +177,15 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&v
         const float other = __shfl_xor_sync(0xffffffffu, v[e], 1);
         if ((lane & 1) == 0 && i_global + 1 < p.rows_a && j0 + e < p.rows_b) {
           const float gate = v[e];
-          out_h[(i_global >> 1) + (j0 + e) * p.stride_b] =
-              __float2bfloat16_rn(fb_glu_act(gate, p.glu_act) * other);
+          float h;
+          if (p.glu_act == 2) {
+            const float* b = p.clamp.bias;
+            h = fb_glu_clamped(p.clamp, gate + (b != nullptr ? __ldg(b + i_global) : 0.f),
+                               other + (b != nullptr ? __ldg(b + i_global + 1) : 0.f));
+          } else {
+            h = fb_glu_act(gate, p.glu_act) * other;
+          }
+          out_h[(i_global >> 1) + (j0 + e) * p.stride_b] = __float2bfloat16_rn(h);
         }
       }
     }

@@ -59,7 +59,7 @@ _SIGNATURES = {
     "fb_gemm_tc": [c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_void_p, c_ll, c_ll, c_int,
                    c_int, c_int, c_ll, c_int, c_int, c_int, c_void_p, c_ll, c_void_p, c_int,
                    c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_ll, c_void_p,
-                   c_void_p, c_ll, c_void_p, c_int, c_void_p],
+                   c_void_p, c_ll, c_void_p, c_int, c_float, c_float, c_float, c_void_p, c_void_p],
     "fb_gemm_tc_rope": [c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_ll,
                         c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p,
                         c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_ll,
@@ -72,7 +72,7 @@ _SIGNATURES = {
                             c_void_p],
     "fb_gemm_skinny": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int,
                        c_int, c_void_p, c_ll, c_int, c_ll, c_int, c_void_p, c_int, c_int, c_int,
-                       c_float, c_void_p],
+                       c_float, c_float, c_float, c_float, c_void_p, c_void_p],
     "fb_gemm_skinny_residual": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_void_p,
                                 c_ll, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_float, c_void_p,
                                 c_ll, c_int, c_void_p],
@@ -98,7 +98,7 @@ _SIGNATURES = {
                      c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_ll, c_void_p,
                      c_void_p, c_ll, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                      c_void_p, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_ll, c_int, c_int,
-                     c_int, c_int, c_int, c_void_p],
+                     c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_void_p],
     "fb_gemm_rows_status": [c_void_p],
     "fb_row_scales": [c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "fb_select_tokens": [c_void_p, c_ll, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -163,7 +163,7 @@ _SIGNATURES = {
                                     c_void_p, c_int, c_int, c_void_p, c_ll, c_void_p],
     "fb_attention_decode_shared": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
                                    c_int, c_void_p, c_ll, c_ll, c_void_p, c_ll, c_ll, c_int, c_int,
-                                   c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p,
+                                   c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
                                    c_ll, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_ll,
                                    c_int, c_void_p],
     "fb_attention_prefill_masked": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
@@ -531,7 +531,22 @@ def add_rmsnorm(resid: torch.Tensor, delta, weight: torch.Tensor, eps: float,
 
 GLU_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
 # the products' epilogue code for act(gate) * up over (gate, up) row pairs
-GLU_EPILOGUE = {"silu": 1, "gelu_tanh": 4}
+GLU_EPILOGUE = {"silu": 1, "gelu_tanh": 4, "clamped": 6}
+
+
+class GluClamp:
+    """The rule of the "clamped" activation: g = min(gate + b, limit), u = clamp(up + b,
+    +-limit), g sigmoid(alpha g) (u + shift); `bias` float32 by (interleaved) weight row, or None."""
+
+    def __init__(self, limit: float, alpha: float, shift: float, bias: Optional[torch.Tensor] = None):
+        self.limit, self.alpha, self.shift, self.bias = float(limit), float(alpha), float(shift), bias
+
+    def args(self):
+        return (self.limit, self.alpha, self.shift,
+                0 if self.bias is None else _dev(self.bias, "bias", torch.float32))
+
+
+_NO_CLAMP = (0.0, 0.0, 0.0, 0)
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False,
@@ -777,7 +792,8 @@ def _pair_scratch(device):
 def gemm_tc(a, b: torch.Tensor, out: Optional[torch.Tensor], stride_a: int, stride_b: int,
             bn: int, splits: int = 1, split_stride: int = 0, epilogue: int = 0,
             constant_operand: int = 0, persistent: int = 0,
-            sink: Optional[ResidualSink] = None, sink_out=None) -> None:
+            sink: Optional[ResidualSink] = None, sink_out=None,
+            clamp: Optional[GluClamp] = None) -> None:
     """Tensor-core product D[i,j] = sum_k a[i,k] b[j,k] written to
     out[i*stride_a + j*stride_b (+ split*split_stride)]; see csrc/gemm_tcgen05.cu.
     With tokens as the rows of `a` (stride_b == 1, one split): `a` may be a
@@ -806,7 +822,7 @@ def gemm_tc(a, b: torch.Tensor, out: Optional[torch.Tensor], stride_a: int, stri
           _dev(out, "out", contiguous=False), stride_a, stride_b,
           1 if out.dtype == torch.float32 else 0, bn, splits, split_stride, epilogue,
           constant_operand, int(persistent), *scratch, PAIR_SHARE_MIN_KBLOCKS, *scale, *sink_args,
-          _stream(),
+          *(_NO_CLAMP if clamp is None else clamp.args()), _stream(),
           tag=("a{} b{} k{} tile{} splits{}", a.shape[0], b.shape[0], a.shape[1], bn, splits))
 
 
@@ -826,11 +842,11 @@ def _prefetch_range(then_reads: Optional[torch.Tensor]):
 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 0,
-                then_reads: Optional[torch.Tensor] = None, ksplit: int = 1,
-                warps: int = 0) -> torch.Tensor:
+                then_reads: Optional[torch.Tensor] = None, ksplit: int = 1, warps: int = 0,
+                clamp: Optional[GluClamp] = None) -> torch.Tensor:
     """Up to 16 token rows: the weight-streaming kernel (csrc/gemm_skinny.cu).
     epilogue 1: `w` rows are (gate, up) pairs and out is [M, N/2] = SiLU(gate)*up
-    (4: the tanh form of GELU instead); epilogue 5: out = max(x w^T, 0)^2.
+    (4: the tanh form of GELU instead; 6: the rule `clamp`); epilogue 5: out = max(x w^T, 0)^2.
     `then_reads`: the weights the step streams after this product; the kernel's
     blocks ask for their start to be brought into L2 as they finish.
     `ksplit` > 1: K is shared by that many CTAs per row group and `out` is
@@ -841,7 +857,7 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: i
     N = w.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_skinny takes bfloat16 operands")
-    want = (M, N // 2) if epilogue in (1, 4) else (M, N)
+    want = (M, N // 2) if epilogue in (1, 4, 6) else (M, N)
     if ksplit > 1:
         want = (ksplit, *want)
         if out.dtype != torch.float32 or not out.is_contiguous():
@@ -853,7 +869,7 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: i
           _rows(out, "out") if ksplit == 1 else N, 1 if out.dtype == torch.float32 else 0,
           M, N, K, epilogue,
           *_prefetch_range(then_reads), ksplit, M * N if ksplit > 1 else 0, warps, *scale,
-          _stream(), tag=("m{} k{} n{}", M, K, N))
+          *(_NO_CLAMP if clamp is None else clamp.args()), _stream(), tag=("m{} k{} n{}", M, K, N))
     return out
 
 
@@ -991,7 +1007,7 @@ def rows_usable(x, w) -> bool:
 
 
 def _gemm_rows(x, w, epilogue: int, out=None, sink: Optional[ResidualSink] = None,
-               sink_out=None, rope=None) -> None:
+               sink_out=None, rope=None, clamp: Optional[GluClamp] = None) -> None:
     """The launcher's face; `x` may be a `RowScaled`."""
     scale = _NO_SCALE
     if isinstance(x, RowScaled):
@@ -1013,13 +1029,14 @@ def _gemm_rows(x, w, epilogue: int, out=None, sink: Optional[ResidualSink] = Non
         rope_args = rope
     _call("fb_gemm_rows", _dev(x, "x", torch.bfloat16, contiguous=False), _rows(x, "x"), M,
           _dev(w, "w", torch.bfloat16, contiguous=False), _rows(w, "w"), N, K, *out_args, epilogue,
-          *scale, *sink_args, *rope_args, ROWS_SPLITS, _stream(),
+          *scale, *sink_args, *rope_args, ROWS_SPLITS,
+          *(_NO_CLAMP if clamp is None else clamp.args()), _stream(),
           tag=("m{} k{} n{} e{}", M, K, N, epilogue))
 
 
 def gemm_rows(x, w: torch.Tensor, out: Optional[torch.Tensor] = None,
               out_dtype: Optional[torch.dtype] = None, silu_mul: bool = False,
-              act: str = "silu") -> torch.Tensor:
+              act: str = "silu", clamp: Optional[GluClamp] = None) -> torch.Tensor:
     """out[M, N] = x[M, K] @ w[N, K]^T for 17 to 256 token rows (any count up to
     256 works); with `silu_mul` the weight rows are (gate, up) pairs and out is
     [M, N / 2] = act(gate) * up. `x` may be a `RowScaled`."""
@@ -1029,7 +1046,7 @@ def gemm_rows(x, w: torch.Tensor, out: Optional[torch.Tensor] = None,
                           device=w.device)
     if tuple(out.shape) != (M, N // 2 if silu_mul else N) or out.stride(1) != 1:
         raise KernelError(f"gemm_rows: out is {tuple(out.shape)} for x {tuple(x.shape)}, w {tuple(w.shape)}")
-    _gemm_rows(x, w, GLU_EPILOGUE[act] if silu_mul else 0, out=out)
+    _gemm_rows(x, w, GLU_EPILOGUE[act] if silu_mul else 0, out=out, clamp=clamp)
     return out
 
 
@@ -1443,9 +1460,11 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
 
 
 def gemm_bf16_silu_mul(x: torch.Tensor, w_pairs: torch.Tensor, out: torch.Tensor,
-                       then_reads: Optional[torch.Tensor] = None, act: str = "silu") -> torch.Tensor:
+                       then_reads: Optional[torch.Tensor] = None, act: str = "silu",
+                       clamp: Optional[GluClamp] = None) -> torch.Tensor:
     """out[M, I] = act(x @ gate^T) * (x @ up^T) with `w_pairs` [2I, K] holding
-    gate i in row 2i and up i in row 2i+1; the activation ("silu", "gelu_tanh")
+    gate i in row 2i and up i in row 2i+1; the activation ("silu", "gelu_tanh", or
+    "clamped" with the rule `clamp`)
     runs in the product's epilogue, so the [M, 2I] intermediate never reaches memory."""
     M, K = x.shape
     two_i = w_pairs.shape[0]
@@ -1456,21 +1475,25 @@ def gemm_bf16_silu_mul(x: torch.Tensor, w_pairs: torch.Tensor, out: torch.Tensor
     epilogue = GLU_EPILOGUE[act]
     usable = _tc_usable(x.values if isinstance(x, RowScaled) else x, w_pairs, out)
     if usable and rows_usable(x, w_pairs):
-        return gemm_rows(x, w_pairs, out, silu_mul=True, act=act)
+        return gemm_rows(x, w_pairs, out, silu_mul=True, act=act, clamp=clamp)
     if not usable:
         x = plain(x)
-        tmp = torch.empty((M, two_i), dtype=torch.bfloat16, device=x.device)
+        tmp = torch.empty((M, two_i), device=x.device,
+                          dtype=torch.bfloat16 if clamp is None else torch.float32)
         gemm_simt(x, w_pairs, tmp)
+        if clamp is not None:
+            return glu_clamped(tmp, clamp.bias, out, clamp.limit, clamp.alpha, clamp.shift)
         return silu_mul(tmp, out, interleaved=True, act=act)
     if M <= SKINNY_ROWS:
         return gemm_skinny(x, w_pairs, out, epilogue=epilogue, then_reads=then_reads,
-                           warps=skinny_plan(two_i, K, False)[1])
+                           warps=skinny_plan(two_i, K, False)[1], clamp=clamp)
     if M > 128:
         bn, form = prompt_plan(M, two_i)
         gemm_tc(x, w_pairs, out, out.stride(0), 1, bn, epilogue=epilogue, constant_operand=2,
-                persistent=form)
+                persistent=form, clamp=clamp)
     else:
-        gemm_tc(x, w_pairs, out, out.stride(0), 1, 128, epilogue=epilogue, constant_operand=2)
+        gemm_tc(x, w_pairs, out, out.stride(0), 1, 128, epilogue=epilogue, constant_operand=2,
+                clamp=clamp)
     return out
 
 
@@ -2280,8 +2303,9 @@ def attention_shared_rows(ctx, q: torch.Tensor, out: torch.Tensor, page_table, r
                 ws = (ws_o.data_ptr(), ws_ml.data_ptr(), _arrival_counters(q.device, n * G).data_ptr())
             _call("fb_attention_decode_shared", *head, *to, *step, rows.data_ptr(), rows.stride(0),
                   rows.stride(1), *factors, n, H, G, dim, float(scale), int(window),
-                  int(keep_first), f32(None if dist_bias is None else dist_bias.flat, "dist_bias"),
-                  last, *gated, splits, cluster, *ws, *_prefetch_range(then_reads),
+                  int(keep_first), 0 if dist_bias is None else dist_bias.padded.data_ptr()
+                  + 4 * DISTANCE_FRONT, last, 0 if dist_bias is None else dist_bias.padded.shape[1],
+                  *gated, splits, cluster, *ws, *_prefetch_range(then_reads),
                   1 if n > SKINNY_ROWS else 0, _stream())
             return out
     return attention_sink(ctx, q, out, page_table, rows, rows, H, G, dim, dim, scale, window=window,

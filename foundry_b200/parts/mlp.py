@@ -85,6 +85,7 @@ class ClampedGLU(Part):
     The biases in front of the activation join the 32-bit sums; the one behind `down` joins
     the rows here, or (`defer_bias`) is handed out for whoever adds the rows to the stream."""
     replay_safe = True
+    accepts_row_scaled = True  # the gate/up product applies a deferred norm's row scale
     defers_bias = True
 
     def __init__(self, hidden_size: int, intermediate_size: int, limit: float,
@@ -124,15 +125,19 @@ class ClampedGLU(Part):
             b = lambda n: f(n + self.bias_suffix).to(torch.float32)
             self.gate_up_bias = torch.stack([b(gate), b(up)], 1).reshape(-1).contiguous()
             self.down_bias = b(down).contiguous()
+        self.rule = ops.GluClamp(self.limit, self.alpha, self.shift, self.gate_up_bias)
 
     def first_weight(self):
         return self.gate_up
 
     def forward(self, ctx, x, defer_bias: bool = False):
-        x = ops.plain(x)
         hidden = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
-        ops.glu_clamped(product_f32(x, self.gate_up), self.gate_up_bias, hidden, self.limit,
-                        self.alpha, self.shift)
+        if x.dtype == torch.bfloat16 and self.gate_up.dtype == torch.bfloat16:
+            ops.gemm_bf16_silu_mul(x, self.gate_up, hidden, then_reads=self.down.weight,
+                                   act="clamped", clamp=self.rule)  # in the product's epilogue
+        else:
+            ops.glu_clamped(product_f32(ops.plain(x), self.gate_up), self.gate_up_bias, hidden,
+                            self.limit, self.alpha, self.shift)
         y = product_planes(hidden, self.down.weight,
                            then_reads=getattr(ctx, "reads_after_part", None))
         if defer_bias:
