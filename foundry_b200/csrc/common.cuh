@@ -195,7 +195,7 @@ struct FbGluClamp {
 };
 __device__ __forceinline__ float fb_glu_clamped(const FbGluClamp& r, float gate, float up) {
   const float g = fminf(gate, r.limit), u = fminf(fmaxf(up, -r.limit), r.limit);
-  return g / (1.0f + __expf(-r.alpha * g)) * (u + r.shift);
+  return __fdividef(g * (u + r.shift), 1.0f + __expf(-r.alpha * g));
 }
 
 __device__ __forceinline__ float fb_warp_sum(float v) {

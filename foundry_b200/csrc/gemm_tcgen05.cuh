@@ -91,21 +91,25 @@ using GemmParams = FbGemmParams;
 template <int CHUNK>
 __device__ __forceinline__ void store_clamped(const GemmParams& p, const float (&v)[CHUNK],
                                               long long base, long long j0, __nv_bfloat16* out_h) {
-  const bool whole = j0 + CHUNK <= p.rows_b && (base % 8) == 0;
+  const float* bias = p.clamp.bias;
+  if (j0 + CHUNK <= p.rows_b && (base % 8) == 0) {
+    float b[CHUNK];  // all of the chunk's biases asked for before the first is needed
+    if (bias != nullptr) {
 #pragma unroll
-  for (int e = 0; e < CHUNK; e += 16) {  // 8 results = 16 bytes per store
-    float r8[8];
+      for (int e = 0; e < CHUNK; e += 4) {
+        const float4 b4 = __ldg(reinterpret_cast<const float4*>(bias + j0 + e));
+        b[e] = b4.x; b[e + 1] = b4.y; b[e + 2] = b4.z; b[e + 3] = b4.w;
+      }
+    } else {
 #pragma unroll
-    for (int q = 0; q < 8; q += 2) {
-      float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (p.clamp.bias != nullptr && j0 + e + 2 * q + 3 < p.rows_b)
-        b = __ldg(reinterpret_cast<const float4*>(p.clamp.bias + j0 + e + 2 * q));
-      else if (p.clamp.bias != nullptr && j0 + e + 2 * q + 1 < p.rows_b)
-        b = make_float4(__ldg(p.clamp.bias + j0 + e + 2 * q), __ldg(p.clamp.bias + j0 + e + 2 * q + 1), 0.f, 0.f);
-      r8[q] = fb_glu_clamped(p.clamp, v[e + 2 * q] + b.x, v[e + 2 * q + 1] + b.y);
-      r8[q + 1] = fb_glu_clamped(p.clamp, v[e + 2 * q + 2] + b.z, v[e + 2 * q + 3] + b.w);
+      for (int e = 0; e < CHUNK; ++e) b[e] = 0.f;
     }
-    if (whole) {
+#pragma unroll
+    for (int e = 0; e < CHUNK; e += 16) {  // 8 results = 16 bytes per store
+      float r8[8];
+#pragma unroll
+      for (int q = 0; q < 8; ++q)
+        r8[q] = fb_glu_clamped(p.clamp, v[e + 2 * q] + b[e + 2 * q], v[e + 2 * q + 1] + b[e + 2 * q + 1]);
       uint4 pk;
       __nv_bfloat162 h0 = __floats2bfloat162_rn(r8[0], r8[1]);
       __nv_bfloat162 h1 = __floats2bfloat162_rn(r8[2], r8[3]);
@@ -116,11 +120,18 @@ __device__ __forceinline__ void store_clamped(const GemmParams& p, const float (
       pk.z = *reinterpret_cast<uint32_t*>(&h2);
       pk.w = *reinterpret_cast<uint32_t*>(&h3);
       *reinterpret_cast<uint4*>(out_h + base + (e >> 1)) = pk;
-    } else {
-#pragma unroll
-      for (int q = 0; q < 8; ++q)
-        if (j0 + e + 2 * q + 1 < p.rows_b) out_h[base + (e >> 1) + q] = __float2bfloat16_rn(r8[q]);
     }
+    return;
+  }
+#pragma unroll 1
+  for (int e = 0; e < CHUNK; e += 2) {
+    if (j0 + e + 1 >= p.rows_b) break;
+    float g = 0.f, u = 0.f;
+#pragma unroll
+    for (int c = 0; c < CHUNK; c += 2)  // (registers have no runtime index)
+      if (c == e) { g = v[c]; u = v[c + 1]; }
+    if (bias != nullptr) { g += __ldg(bias + j0 + e); u += __ldg(bias + j0 + e + 1); }
+    out_h[base + (e >> 1)] = __float2bfloat16_rn(fb_glu_clamped(p.clamp, g, u));
   }
 }
 
