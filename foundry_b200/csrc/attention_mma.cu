@@ -152,9 +152,12 @@ struct AttnParams {
 };
 
 // A head's finished output element on its way out: times the sigmoid of its gate where there is one.
-__device__ __forceinline__ void store_head(const AttnParams& p, int token, int column, float v) {
-  if (p.gate != nullptr)
-    v = v / (1.0f + __expf(-__ldcg(p.gate + (long long)token * p.gate_stride + column)));
+__device__ __forceinline__ float head_gate(const AttnParams& p, int token, int column) {
+  return p.gate != nullptr ? __ldcg(p.gate + (long long)token * p.gate_stride + column) : 0.f;
+}
+__device__ __forceinline__ void store_head(const AttnParams& p, int token, int column, float v,
+                                           float gate) {
+  if (p.gate != nullptr) v = v / (1.0f + __expf(-gate));
   p.out[(long long)token * p.out_stride + column] = __float2bfloat16_rn(v);
 }
 
@@ -381,6 +384,7 @@ __device__ void merge_if_last(const AttnParams& p, int seq, int kvh, int token, 
   const size_t base = (size_t)(seq * p.Kh + kvh) * p.parts;
   for (int idx = threadIdx.x; idx < G * D; idx += THREADS) {
     const int row = idx / D, d = idx - row * D;
+    const float gate = head_gate(p, token, kvh * G * D + idx);
     // four parts at a time, their twelve loads on the way together
     float M = -INFINITY, L = 0.f, acc = 0.f;
     for (int s0 = 0; s0 < p.parts; s0 += 4) {
@@ -408,7 +412,7 @@ __device__ void merge_if_last(const AttnParams& p, int seq, int kvh, int token, 
       }
       M = Mn;
     }
-    store_head(p, token, (kvh * G + row) * D + d, L > 0.f ? acc / L : 0.f);
+    store_head(p, token, kvh * G * D + idx, L > 0.f ? acc / L : 0.f, gate);
   }
   if (threadIdx.x == 0) p.counters[seq * p.Kh + kvh] = 0;
 }
@@ -442,13 +446,16 @@ __device__ void merge_in_cluster(const AttnParams& p, const float* cO, const flo
                                  const float* cL, int seq, int kvh, int token, int G) {
   unsigned rank;
   asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(rank));
-  __syncthreads();
-  cluster_sync_all();
   const int S = p.cluster;
   const int total = G * D, share = (total + S - 1) / S;
   const int end = min(total, (int)(rank + 1) * share);
+  // (a thread's first gate is on its way while the cluster meets)
+  const int mine = rank * share + threadIdx.x;
+  float gate = mine < end ? head_gate(p, token, kvh * G * D + mine) : 0.f;
+  __syncthreads();
+  cluster_sync_all();
   const size_t slot = (size_t)(seq * p.Kh + kvh) * p.parts + blockIdx.z / S;
-  for (int idx = rank * share + threadIdx.x; idx < end; idx += THREADS) {
+  for (int idx = mine; idx < end; idx += THREADS) {
     const int row = idx / D, d = idx - row * D;
     float ms[MAX_CLUSTER], ls[MAX_CLUSTER], os[MAX_CLUSTER];
 #pragma unroll
@@ -476,7 +483,8 @@ __device__ void merge_in_cluster(const AttnParams& p, const float* cO, const flo
       p.ws_o[(slot * 16 + row) * D + d] = acc;
       if (d == 0) { p.ws_ml[slot * 32 + 2 * row] = M; p.ws_ml[slot * 32 + 2 * row + 1] = L; }
     } else {
-      store_head(p, token, (kvh * G + row) * D + d, L > 0.f ? acc / L : 0.f);
+      store_head(p, token, kvh * G * D + idx, L > 0.f ? acc / L : 0.f, gate);
+      if (idx + THREADS < end) gate = head_gate(p, token, kvh * G * D + idx + THREADS);
     }
   }
   cluster_sync_all();  // peers may have been reading this CTA's memory until here
@@ -570,6 +578,22 @@ attn_decode_kernel(const AttnParams p) {
                  p.key_scale + (long long)page * p.ks_page + (long long)kvh * p.ks_head +
                      warp * 16 + lane * 4, true);
   };
+  // ONE: the biases of this lane's four (narrow) or eight (wide) scores of a page (constant data)
+  constexpr int NB = NARROW ? 4 : 8;
+  float by_next[ONE ? NB : 1];
+  auto ask_biases = [&](int j) {
+    const int first_key = page_at(j) * FB_PAGE + warp * 16;
+#pragma unroll
+    for (int e = 0; e < (ONE ? NB : 0); ++e) {
+      const int key = NARROW ? first_key + g + (e >> 1) * 8
+                             : first_key + (e >> 2) * 8 + 2 * t + (e & 1);
+      const int query = min(NARROW ? 2 * t + (e & 1) : g + ((e >> 1) & 1) * 8, G - 1);
+      const int away = min(max(kv_len - 1 - key, 0), p.table_last);
+      by_next[e] = p.table == nullptr ? 0.f
+          : __ldg(p.table + (size_t)(kvh * G + query) * p.table_pitch + away);
+    }
+  };
+  if (ONE) ask_biases(pg0);
   // old pages of the first ST - 1 go out now; they complete with the first group
 #pragma unroll
   for (int ahead = 0; ahead < ST - 1; ++ahead)
@@ -605,18 +629,12 @@ attn_decode_kernel(const AttnParams p) {
     const int refill_page = next_page;
     if (pg + ST < pg1) next_page = pages[page_at(pg + ST)];
     const int key0 = page_at(pg) * FB_PAGE + warp * 16;  // this warp's 16 keys of the page
-    // the biases of this lane's four (narrow) or eight (wide) scores, asked for before the wait
-    constexpr int NB = NARROW ? 4 : 8;
+    // this page's biases were asked for a page ago; the next page's are asked for now
     float by_distance[ONE ? NB : 1];
     if constexpr (ONE) {
 #pragma unroll
-      for (int e = 0; e < NB; ++e) {
-        const int key = NARROW ? key0 + g + (e >> 1) * 8 : key0 + (e >> 2) * 8 + 2 * t + (e & 1);
-        const int query = min(NARROW ? 2 * t + (e & 1) : g + ((e >> 1) & 1) * 8, G - 1);
-        const int away = min(max(kv_len - 1 - key, 0), p.table_last);
-        by_distance[e] = p.table == nullptr ? 0.f
-            : __ldg(p.table + (size_t)(kvh * G + query) * p.table_pitch + away);
-      }
+      for (int e = 0; e < NB; ++e) by_distance[e] = by_next[e];
+      if (pg + 1 < pg1) ask_biases(pg + 1);
     }
     // The buffer that the previous iteration finished with is refilled once this
     // page's score products have been issued: a warp issues in order, and the
@@ -868,7 +886,8 @@ attn_decode_kernel(const AttnParams p) {
       ws_o[row * D + d] = acc;
       if (d == 0) { ws_ml[2 * row] = M; ws_ml[2 * row + 1] = L; }
     } else {
-      store_head(p, token, (kvh * G + row) * D + d, L > 0.f ? acc / L : 0.f);
+      store_head(p, token, kvh * G * D + idx, L > 0.f ? acc / L : 0.f,
+                 head_gate(p, token, kvh * G * D + idx));
     }
   }
   if (CLUSTER) merge_in_cluster<D>(p, cO, cM, cL, seq, kvh, token, G);

@@ -104,6 +104,29 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// Two 32-bit multiply-adds or sums in one instruction: (a, b) <- (a x + p, b y + q); (a, b) + c.
+__device__ __forceinline__ void fma2(float& a, float& b, float x, float y, float p, float q) {
+  asm("{\n\t.reg .b64 u, v, w;\n\tmov.b64 u, {%0, %1};\n\tmov.b64 v, {%2, %3};\n\t"
+      "mov.b64 w, {%4, %5};\n\tfma.rn.f32x2 u, u, v, w;\n\tmov.b64 {%0, %1}, u;\n\t}"
+      : "+f"(a), "+f"(b)
+      : "f"(x), "f"(y), "f"(p), "f"(q));
+}
+__device__ __forceinline__ void add2(float& a, float& b, float c) {
+  asm("{\n\t.reg .b64 u, v;\n\tmov.b64 u, {%0, %1};\n\tmov.b64 v, {%2, %2};\n\t"
+      "add.rn.f32x2 u, u, v;\n\tmov.b64 {%0, %1}, u;\n\t}"
+      : "+f"(a), "+f"(b)
+      : "f"(c));
+}
+
+// 32 bytes at a time (a whole sector), for data that a kernel in front wrote
+__device__ __forceinline__ void load_f32x8(const float* p, float* v) {
+  asm volatile("ld.global.v8.f32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];"
+               : "=f"(v[0]), "=f"(v[1]), "=f"(v[2]), "=f"(v[3]), "=f"(v[4]), "=f"(v[5]),
+                 "=f"(v[6]), "=f"(v[7])
+               : "l"(p)
+               : "memory");
+}
+
 // KS, VS: 64-element (128-byte) blocks along a key row and a value row
 template <int KS, int VS, bool ONE>
 struct FaSmem {
@@ -353,10 +376,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
           for (int e4 = 0; e4 < FB_PAGE / 4; ++e4) {
             const float4 f = factor[e4];
-            sc[4 * e4] = fmaf(sc[4 * e4], f.x, flat);
-            sc[4 * e4 + 1] = fmaf(sc[4 * e4 + 1], f.y, flat);
-            sc[4 * e4 + 2] = fmaf(sc[4 * e4 + 2], f.z, flat);
-            sc[4 * e4 + 3] = fmaf(sc[4 * e4 + 3], f.w, flat);
+            fma2(sc[4 * e4], sc[4 * e4 + 1], f.x, f.y, flat, flat);
+            fma2(sc[4 * e4 + 2], sc[4 * e4 + 3], f.z, f.w, flat, flat);
           }
         } else if (table_here) {
           // (a row without tokens keeps to the table, too: its position is one of the block's)
@@ -364,20 +385,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
           for (int e4 = 0; e4 < FB_PAGE / 4; ++e4) {
             const float4 f = factor[e4];
-            sc[4 * e4] = fmaf(sc[4 * e4], f.x, at[-4 * e4]);
-            sc[4 * e4 + 1] = fmaf(sc[4 * e4 + 1], f.y, at[-4 * e4 - 1]);
-            sc[4 * e4 + 2] = fmaf(sc[4 * e4 + 2], f.z, at[-4 * e4 - 2]);
-            sc[4 * e4 + 3] = fmaf(sc[4 * e4 + 3], f.w, at[-4 * e4 - 3]);
+            fma2(sc[4 * e4], sc[4 * e4 + 1], f.x, f.y, at[-4 * e4], at[-4 * e4 - 1]);
+            fma2(sc[4 * e4 + 2], sc[4 * e4 + 3], f.z, f.w, at[-4 * e4 - 2],
+                 at[-4 * e4 - 3]);
           }
         } else {  // a table longer than shared memory has room for
           const float* at = p.table + (size_t)head * p.table_pitch + TABLE_FRONT + (qpos - key0);
 #pragma unroll
           for (int e4 = 0; e4 < FB_PAGE / 4; ++e4) {
             const float4 f = factor[e4];
-            sc[4 * e4] = fmaf(sc[4 * e4], f.x, __ldg(at - 4 * e4));
-            sc[4 * e4 + 1] = fmaf(sc[4 * e4 + 1], f.y, __ldg(at - 4 * e4 - 1));
-            sc[4 * e4 + 2] = fmaf(sc[4 * e4 + 2], f.z, __ldg(at - 4 * e4 - 2));
-            sc[4 * e4 + 3] = fmaf(sc[4 * e4 + 3], f.w, __ldg(at - 4 * e4 - 3));
+            fma2(sc[4 * e4], sc[4 * e4 + 1], f.x, f.y, __ldg(at - 4 * e4), __ldg(at - 4 * e4 - 1));
+            fma2(sc[4 * e4 + 2], sc[4 * e4 + 3], f.z, f.w, __ldg(at - 4 * e4 - 2),
+                 __ldg(at - 4 * e4 - 3));
           }
         }
       }
@@ -441,8 +460,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       for (int c = 0; c < 32; ++c) {
         // 2^(s * scale - m_ref): one multiply-add and one ex2; the result is at most 2^8
         // and is rounded to bfloat16 next, so the approximate ex2 costs no accuracy
-        const float p0 = fast_exp2(fmaf(sc[2 * c], to_log2, neg_ref));
-        const float p1 = fast_exp2(fmaf(sc[2 * c + 1], to_log2, neg_ref));
+        if (ONE) {
+          add2(sc[2 * c], sc[2 * c + 1], neg_ref);
+        } else {
+          sc[2 * c] = fmaf(sc[2 * c], to_log2, neg_ref);
+          sc[2 * c + 1] = fmaf(sc[2 * c + 1], to_log2, neg_ref);
+        }
+        const float p0 = fast_exp2(sc[2 * c]);
+        const float p1 = fast_exp2(sc[2 * c + 1]);
         sum4[c & 1] += p0;
         sum4[2 + (c & 1)] += p1;
         const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
@@ -455,7 +480,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_full[b]);
     }
-    // O / l
+    // O / l (ONE: times the sigmoid of the gate, whose next 32 columns are asked for while this
+    // thread works on these)
+    const float* gate_row = (ONE && p.gate != nullptr && row < rows_valid)
+        ? p.gate + (long long)(tok0 + row0 + row) * p.gate_stride + (long long)head * p.DV : nullptr;
+    float gate[ONE ? 32 : 1];
+    auto ask_gate = [&](int c) {
+#pragma unroll
+      for (int e = 0; e < (ONE ? 32 : 0); e += 8)
+        if (gate_row != nullptr && c + e < p.DV) load_f32x8(gate_row + c + e, gate + e);
+    };
+    ask_gate(0);
     if (ok) ok = mbar_wait(o_final, 0, abort_flag, 19, n_pages);
     if (ok) {
       tc_fence_after();
@@ -467,20 +502,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         uint32_t r[32];
         tmem_ld32(tmem_base + lane_base + O_COL + (uint32_t)c, r);
         tmem_ld_wait();
+        if (ONE && gate_row != nullptr) {
+#pragma unroll
+          for (int e = 0; e < (ONE ? 32 : 0); ++e)
+            r[e] = __float_as_uint(__fdividef(__uint_as_float(r[e]), 1.0f + __expf(-gate[e])));
+          ask_gate(c + 32);
+        }
         if (row < rows_valid) {
 #pragma unroll
           for (int e = 0; e < 32; e += 8) {
             if (c + e >= p.DV) break;  // (whole pieces: DV is a multiple of 8)
-            if (ONE && p.gate != nullptr) {
-              const float* g = p.gate + (long long)(tok0 + row0 + row) * p.gate_stride +
-                               (long long)head * p.DV + c + e;
-              const float4 a = __ldcg(reinterpret_cast<const float4*>(g));
-              const float4 d = __ldcg(reinterpret_cast<const float4*>(g + 4));
-              const float z[8] = {a.x, a.y, a.z, a.w, d.x, d.y, d.z, d.w};
-#pragma unroll
-              for (int q = 0; q < 8; ++q)
-                r[e + q] = __float_as_uint(__uint_as_float(r[e + q]) / (1.0f + __expf(-z[q])));
-            }
             uint4 pk;
             __nv_bfloat162 h0 = __floats2bfloat162_rn(__uint_as_float(r[e]) * inv, __uint_as_float(r[e + 1]) * inv);
             __nv_bfloat162 h1 = __floats2bfloat162_rn(__uint_as_float(r[e + 2]) * inv, __uint_as_float(r[e + 3]) * inv);
@@ -620,7 +651,7 @@ FB_API int fb_attention_prefill_tc(const void* q, long long q_stride, int T, voi
 // The form with shared rows (see the file's notes): `rows` are one cache entry's
 // [n_pages, Kh, 64, D] with heads `row_head` elements apart and pages Kh * row_head apart,
 // `key_scale` their float32 factors. `table`: see FaParams (null: no bias). `gate`: null or
-// float32 rows of A * D elements, 16-byte aligned.
+// float32 rows of A * D elements, 32-byte aligned.
 FB_API int fb_attention_prefill_shared(const void* q, long long q_stride, int T, void* out,
                                        long long out_stride, const int* cu_tokens,
                                        const int* kv_lens, const int* page_table, int max_pages,
@@ -643,8 +674,9 @@ FB_API int fb_attention_prefill_shared(const void* q, long long q_stride, int T,
              table_pitch, table_last);
   FB_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && ((uintptr_t)q % 16) == 0 &&
                  ((uintptr_t)out % 16) == 0 && ((uintptr_t)rows % 16) == 0 &&
-                 ((uintptr_t)gate % 16) == 0 && gate_stride % 4 == 0,
-             "attention_prefill_shared: pointers and strides must keep 16-byte alignment");
+                 ((uintptr_t)gate % 32) == 0 && gate_stride % 8 == 0,
+             "attention_prefill_shared: pointers and strides must keep 16-byte (the gate: 32-byte) "
+             "alignment");
   if (q_blocks <= 0) return 0;
   bind_status_mirror(stream);
   CUtensorMap mq, mk;

@@ -2256,7 +2256,7 @@ def attention_shared_rows(ctx, q: torch.Tensor, out: torch.Tensor, page_table, r
     T = q.shape[0]
     if (SHARED_ROWS_TC and q.dtype == torch.bfloat16 and T > 0 and dim % 8 == 0 and dim <= 128
             and _tc_attention_ok(q, out) and (gate is None or (
-                gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0))):
+                gate.stride(0) % 8 == 0 and gate.data_ptr() % 32 == 0))):
         if rows.stride(0) != G * rows.stride(1) or tuple(rows.shape[1:]) != (G, PAGE, dim) \
                 or rows.stride(2) != dim or tuple(scales.shape) != (rows.shape[0], G, PAGE):
             raise KernelError(f"attention_shared_rows: rows {tuple(rows.shape)} strides "
