@@ -76,6 +76,13 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// 2^x where the result is at most a few hundred and goes into a 16-bit operand and a sum
+__device__ __forceinline__ float approx_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float REFERENCE_STEP = 8.0f;  // shared rows: the softmax's reference moves by 2^8 at least
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&h);
@@ -581,16 +588,29 @@ attn_decode_kernel(const AttnParams p) {
   // ONE: the biases of this lane's four (narrow) or eight (wide) scores of a page (constant data)
   constexpr int NB = NARROW ? 4 : 8;
   float by_next[ONE ? NB : 1];
-  auto ask_biases = [&](int j) {
-    const int first_key = page_at(j) * FB_PAGE + warp * 16;
+  // (entries of the lane's two queries, then of the key's distance: one address a score)
+  const float* bias_of[2] = {nullptr, nullptr};
+  if (ONE && p.table != nullptr) {
 #pragma unroll
-    for (int e = 0; e < (ONE ? NB : 0); ++e) {
-      const int key = NARROW ? first_key + g + (e >> 1) * 8
-                             : first_key + (e >> 2) * 8 + 2 * t + (e & 1);
-      const int query = min(NARROW ? 2 * t + (e & 1) : g + ((e >> 1) & 1) * 8, G - 1);
-      const int away = min(max(kv_len - 1 - key, 0), p.table_last);
-      by_next[e] = p.table == nullptr ? 0.f
-          : __ldg(p.table + (size_t)(kvh * G + query) * p.table_pitch + away);
+    for (int r = 0; r < 2; ++r)
+      bias_of[r] = p.table + (size_t)(kvh * G + min(NARROW ? 2 * t + r : g + 8 * r, G - 1)) * p.table_pitch;
+  }
+  auto ask_biases = [&](int j) {
+    const int away0 = kv_len - 1 - (page_at(j) * FB_PAGE + warp * 16);
+    auto entry = [&](int k) { return min(max(away0 - k, 0), p.table_last); };
+    if constexpr (!ONE) return;
+    if (p.table == nullptr) {
+#pragma unroll
+      for (int e = 0; e < (ONE ? NB : 0); ++e) by_next[e] = 0.f;
+    } else if (NARROW) {
+      const int n0 = entry(g), n1 = entry(g + 8);
+#pragma unroll
+      for (int e = 0; e < (ONE ? NB : 0); ++e) by_next[e] = __ldg(bias_of[e & 1] + (e < 2 ? n0 : n1));
+    } else {
+      const int n4[4] = {entry(2 * t), entry(2 * t + 1), entry(8 + 2 * t), entry(9 + 2 * t)};
+#pragma unroll
+      for (int e = 0; e < (ONE ? NB : 0); ++e)
+        by_next[e] = __ldg(bias_of[(e >> 1) & 1] + n4[(e >> 2) * 2 + (e & 1)]);
     }
   };
   if (ONE) ask_biases(pg0);
@@ -703,19 +723,27 @@ attn_decode_kernel(const AttnParams p) {
           s[e] = v;
           mx[e & 1] = fmaxf(mx[e & 1], v);
         }
+        // ONE: the reference only moves when a score has outgrown it by 2^8 (a vote in place of
+        // the shuffles, and nothing to rescale)
+        const bool moves = !ONE || __any_sync(0xffffffffu, mx[0] > m[0] + REFERENCE_STEP ||
+                                                              mx[1] > m[1] + REFERENCE_STEP);
+        float corr[2] = {1.f, 1.f}, sum[2] = {0.f, 0.f};
+        if (moves) {
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 4));
-          mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 8));
-          mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 16));
+          for (int r = 0; r < 2; ++r) {
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 4));
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 8));
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 16));
+          }
+          // one of the warp's keys is visible, so mx is finite
+#pragma unroll
+          for (int r = 0; r < 2; ++r) corr[r] = exp2f(m[r] - mx[r]);
+        } else {
+          mx[0] = m[0]; mx[1] = m[1];
         }
-        // one of the warp's keys is visible, so mx is finite
-        float corr[2], sum[2] = {0.f, 0.f};
-#pragma unroll
-        for (int r = 0; r < 2; ++r) corr[r] = exp2f(m[r] - mx[r]);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float pv = exp2f(s[e] - mx[e & 1]);
+          const float pv = ONE ? approx_exp2(s[e] - mx[e & 1]) : exp2f(s[e] - mx[e & 1]);
           s[e] = pv;
           sum[e & 1] += pv;
         }
@@ -726,10 +754,12 @@ attn_decode_kernel(const AttnParams p) {
           l[r] = l[r] * corr[r] + sum[r];
           m[r] = mx[r];
         }
+        if (moves) {
 #pragma unroll
-        for (int n = 0; n < OT; ++n) {
-          o[n][0] *= corr[0]; o[n][1] *= corr[1];
-          o[n][2] *= corr[0]; o[n][3] *= corr[1];
+          for (int n = 0; n < OT; ++n) {
+            o[n][0] *= corr[0]; o[n][1] *= corr[1];
+            o[n][2] *= corr[0]; o[n][3] *= corr[1];
+          }
         }
         // P^T as the B operand: (keys 2t, 2t + 1 and 2t + 8, 2t + 9; query g)
         const uint32_t b0 = movmatrix_trans(pack_bf16(s[0], s[1]));
@@ -769,19 +799,25 @@ attn_decode_kernel(const AttnParams p) {
             mx[e >> 1] = fmaxf(mx[e >> 1], v);
           }
         }
+        const bool moves = !ONE || __any_sync(0xffffffffu, mx[0] > m[0] + REFERENCE_STEP ||
+                                                              mx[1] > m[1] + REFERENCE_STEP);
+        float corr[2] = {1.f, 1.f}, sum[2] = {0.f, 0.f};
+        if (moves) {
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-          mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+          for (int r = 0; r < 2; ++r) {
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+          }
+#pragma unroll
+          for (int r = 0; r < 2; ++r) corr[r] = exp2f(m[r] - mx[r]);
+        } else {
+          mx[0] = m[0]; mx[1] = m[1];
         }
-        float corr[2], sum[2] = {0.f, 0.f};
-#pragma unroll
-        for (int r = 0; r < 2; ++r) corr[r] = exp2f(m[r] - mx[r]);
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            const float pv = exp2f(s[n][e] - mx[e >> 1]);
+            const float pv = ONE ? approx_exp2(s[n][e] - mx[e >> 1]) : exp2f(s[n][e] - mx[e >> 1]);
             s[n][e] = pv;
             sum[e >> 1] += pv;
           }
@@ -791,10 +827,12 @@ attn_decode_kernel(const AttnParams p) {
           l[r] = l[r] * corr[r] + sum[r];
           m[r] = mx[r];
         }
+        if (moves) {
 #pragma unroll
-        for (int n = 0; n < NT; ++n) {
-          o[n][0] *= corr[0]; o[n][1] *= corr[0];
-          o[n][2] *= corr[1]; o[n][3] *= corr[1];
+          for (int n = 0; n < NT; ++n) {
+            o[n][0] *= corr[0]; o[n][1] *= corr[0];
+            o[n][2] *= corr[1]; o[n][3] *= corr[1];
+          }
         }
         uint32_t a[4];
         a[0] = pack_bf16(s[0][0], s[0][1]);
