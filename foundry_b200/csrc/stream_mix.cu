@@ -225,17 +225,14 @@ FB_API int fb_stream_mix_norm(const float* x, long long token_stride, long long 
                    whole16(w) && whole16(out) && token_stride % 4 == 0 && plane_stride % 4 == 0;
   const int yd = y != nullptr ? y_dtype : FB_F32;
   // (the block width decides the order of a row's sums, so it depends on W alone)
-  const int pieces = (W + 3) / 4;
-  const int items = pieces <= 1024 ? 1 : 2;
-  const int threads = ((pieces + items - 1) / items + 31) / 32 * 32;
+  const int threads = ((W + 3) / 4 + 63) / 64 * 32;  // two pieces each
   if (vec && S <= 4 && threads <= 1024) {
-#define FB_STREAM(SM_, I_)                                                                       \
-  fb_launch(stream_mix_norm_kernel<TY, TO, SM_, I_>, dim3(T), dim3(threads), 0, stream, p, (TO*)out)
     FB_DISPATCH_DTYPE(yd, TY, FB_DISPATCH_DTYPE(out_dtype, TO, {
-      if (S <= 2) { if (items == 1) FB_STREAM(2, 1); else FB_STREAM(2, 2); }
-      else { if (items == 1) FB_STREAM(4, 1); else FB_STREAM(4, 2); }
+      if (S <= 2)
+        fb_launch(stream_mix_norm_kernel<TY, TO, 2, 2>, dim3(T), dim3(threads), 0, stream, p, (TO*)out);
+      else
+        fb_launch(stream_mix_norm_kernel<TY, TO, 4, 2>, dim3(T), dim3(threads), 0, stream, p, (TO*)out);
     }));
-#undef FB_STREAM
     return fb_check_launch("stream_mix_norm");
   }
   const size_t smem = (size_t)W * 4;
