@@ -31,6 +31,8 @@ Optional, any part
     `ctx.*_host`, which are None in a replayed step). Short prompt steps of a
     model whose parts all say so are captured once per bucket and replayed
     (engine/prompt.py); otherwise they are launched one by one.
+    defers_bias = True (a feed-forward): forward(ctx, x, defer_bias=True) returns (rows,
+    bias) for a block that adds the bias where it adds the rows to the stream.
     first_weight() -> the weight tensor its forward streams first, or None.
     `ctx.reads_after_part` holds the first weight of whatever runs after the
     part being called (the block sets it for its mixer and feed-forward, the

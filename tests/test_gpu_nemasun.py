@@ -127,12 +127,12 @@ OTHER_SIZES = [
     (2, 2, 128, 128, 0, 20, 11),
     (8, 2, 32, 77, 65, 16, 40),
     (3, 1, 72, None, 0, 30, 1000),
-    (16, 1, 128, 200, 64, 32, 120),
+    (16, 1, 128, 200, 64, 26, 110),
     (20, 1, 16, 1, 3, 8, 9),
     (2, 1, 264, 90, 5, 12, 50),
     (5, 5, 13, 65, 128, 24, 70),
     (32, 4, 64, 1000, 4, 64, 4096),
-    (6, 3, 96, 96, 6, 32, 120),
+    (6, 3, 104, 80, 7, 28, 90),
 ]
 
 
@@ -159,9 +159,9 @@ def test_attention_in_two_cuttings(sizes, dtype):
             assert rel_error(g, w) < bound(dtype), (sizes, cuts)
 
 
-@pytest.mark.parametrize("last", [33, 120, 2000, 9000])
+@pytest.mark.parametrize("last", [33, 110, 2000, 9000])
 @pytest.mark.parametrize("mask", [(37, 0), (64, 64), (150, 5), (300, 130), (1000, 1), (None, 0)])
-@pytest.mark.parametrize("sizes", [(64, 4, 2), (128, 2, 1), (96, 3, 1), (40, 2, 2)])
+@pytest.mark.parametrize("sizes", [(64, 4, 2), (128, 2, 1), (88, 3, 1), (40, 2, 2)])
 def test_prompts_and_single_tokens_on_the_tensor_cores(sizes, mask, last):
     """bfloat16 steps on the tensor cores against the CUDA-core kernel on the same rows:
     windows that end inside a block of queries and inside a page, kept tokens of less and more
@@ -317,7 +317,7 @@ def test_clamped_feed_forward(sizes, dtype):
         assert rel_error((rows_of(y).float() + bias).cpu(), want) < bound(dtype), T
 
 
-MOE = [(64, 32, 8, 2, 4, (2, 1), 128), (80, 56, 6, 2, 3, (4, 2), 40), (36, 12, 4, 4, 4, None, None),
+MOE = [(64, 32, 9, 3, 4, (2, 1), 120), (80, 56, 6, 2, 3, (4, 2), 40), (36, 12, 4, 4, 4, None, None),
        (128, 64, 12, 0, 5, (3, 2), 64), (256, 96, 100, 28, 8, (16, 4), 96), (64, 64, 1, 1, 1, None, None),
        (64, 30, 5, 1, 2, (6, 5), None)]
 

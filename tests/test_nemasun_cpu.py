@@ -112,7 +112,7 @@ def test_weights_of_a_part_that_is_not_there_may_lie_in_the_file():
     assert not hit("l0.norm2") and not hit("l2.hc1.mix") and not hit("l2.norm1")
 
 
-@pytest.mark.parametrize("rows, last", [(16, 40), (8, 9), (30, 128), (32, 120), (20, 11), (6, 300),
+@pytest.mark.parametrize("rows, last", [(16, 40), (8, 9), (30, 128), (32, 130), (20, 11), (6, 300),
                                         (2, 5), (64, 4096), (24, 70)])
 def test_distance_buckets(rows, last):
     from foundry_b200.parts.shared_row_attention import distance_buckets
